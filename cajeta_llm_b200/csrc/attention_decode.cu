@@ -329,7 +329,7 @@ __global__ void __launch_bounds__(TC_THREADS, TC_BLOCKS) decode_attention_tc_ker
     const __nv_bfloat16* __restrict__ vplane, const int* __restrict__ positions, const int* __restrict__ row_req,
     const int* __restrict__ table, int table_stride, int page_tokens, int n_heads, int n_kv, int head_batches,
     int window, float scale, float* __restrict__ part_acc, float* __restrict__ part_ml, int* __restrict__ counters,
-    int max_splits, int merge_later, float softcap, const float* __restrict__ head_gate, int gate_ld) {
+    int max_splits, int merge_later, float softcap, const float* __restrict__ head_gate, int gate_ld, float sink) {
     cj::release_successor();
     constexpr int COLS = HD / 8;
     extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -490,7 +490,10 @@ __global__ void __launch_bounds__(TC_THREADS, TC_BLOCKS) decode_attention_tc_ker
         }
         const int h = h0 + row;
         if (n_splits == 1) {
-            float inv = 1.0f / l;
+            float m = smax[0][row];
+#pragma unroll
+            for (int w = 1; w < TC_WARPS; ++w) m = fmaxf(m, smax[w][row]);
+            float inv = 1.0f / (l + expf(sink - m));          // the key without a value; sink = -inf: none
             if (head_gate) inv *= 1.0f / (1.0f + expf(-head_gate[(size_t)t * gate_ld + h]));
             *(__nv_bfloat162*)(out + ((size_t)t * n_heads + h) * HD + 2 * d2) = __floats2bfloat162_rn(a.x * inv, a.y * inv);
         } else {
@@ -536,7 +539,7 @@ __global__ void __launch_bounds__(TC_THREADS, TC_BLOCKS) decode_attention_tc_ker
             a.x = fmaf(v.x, f, a.x);
             a.y = fmaf(v.y, f, a.y);
         }
-        float inv = 1.0f / L;
+        float inv = 1.0f / (L + expf(sink - M));
         if (head_gate) inv *= 1.0f / (1.0f + expf(-head_gate[(size_t)t * gate_ld + h]));
         *(__nv_bfloat162*)(out + ((size_t)t * n_heads + h) * HD + 2 * d2) = __floats2bfloat162_rn(a.x * inv, a.y * inv);
     }
@@ -549,7 +552,7 @@ template <int HD>
 __global__ void __launch_bounds__(128) decode_merge_kernel(
     __nv_bfloat16* __restrict__ out, const float* __restrict__ part_acc, const float* __restrict__ part_ml,
     const int* __restrict__ positions, int T, int n_heads, int window, int max_splits, const float* __restrict__ head_gate,
-    int gate_ld) {
+    int gate_ld, float sink) {
     cj::release_successor();
     const int lane = threadIdx.x & 31;
     const long long idx = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -579,7 +582,7 @@ __global__ void __launch_bounds__(128) decode_merge_kernel(
             a.x = fmaf(v.x, f, a.x);
             a.y = fmaf(v.y, f, a.y);
         }
-        float inv = gate / L;
+        float inv = gate / (L + expf(sink - M));
         *(__nv_bfloat162*)(out + (size_t)idx * HD + 2 * d2) = __floats2bfloat162_rn(a.x * inv, a.y * inv);
     }
 }
@@ -628,11 +631,12 @@ CJ_EXPORT int cj_decode_attention(const void* q, void* out, const void* kplane, 
 
 // The same on the tensor cores (chunks of 128 keys; up to 8 query heads of a kv head a block).
 // counters: int32 [T * n_heads] here (one per row, kv head and batch of 8 heads).
+// sink: a constant score of one more key that has no value, exp(sink) in the divisor alone; -infinity: none.
 CJ_EXPORT int cj_decode_attention_tc(const void* q, void* out, const void* kplane, const void* vplane, const int* positions,
                                      const int* row_req, const int* table, int table_stride, int page_tokens, int T,
                                      int n_heads, int n_kv, int hd, int window, float scale, int max_context,
                                      float* part_acc, float* part_ml, int* counters, int max_splits, int merge_later,
-                                     float softcap, const float* head_gate, int gate_ld, cudaStream_t stream) {
+                                     float softcap, const float* head_gate, int gate_ld, float sink, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (!q || !out || !kplane || !vplane || !positions || !row_req || !table || !part_acc || !part_ml || !counters) return CJ_ERR_ARG;
     if (n_heads <= 0 || n_kv <= 0 || n_heads % n_kv != 0 || page_tokens <= 0) return CJ_ERR_SIZE;
@@ -657,11 +661,11 @@ CJ_EXPORT int cj_decode_attention_tc(const void* q, void* out, const void* kplan
         cj::launch(decode_attention_tc_kernel<HD>, dim3(grid), dim3(TC_THREADS), smem, stream, (const __nv_bfloat16*)q, \
             (__nv_bfloat16*)out, (const __nv_bfloat16*)kplane, (const __nv_bfloat16*)vplane, positions, row_req, table, \
             table_stride, page_tokens, n_heads, n_kv, head_batches, window, scale, part_acc, part_ml, counters,        \
-            max_splits, merge_later && splits > 1 ? 1 : 0, softcap, head_gate, gate_ld);                               \
+            max_splits, merge_later && splits > 1 ? 1 : 0, softcap, head_gate, gate_ld, sink);                         \
         if (merge_later && splits > 1)                                                                                 \
             cj::launch(decode_merge_kernel<HD>, dim3((unsigned)(((long long)T * n_heads + 3) / 4)), dim3(128), 0, stream, \
                 (__nv_bfloat16*)out, (const float*)part_acc, (const float*)part_ml, positions, T, n_heads, window, max_splits, \
-                head_gate, gate_ld);                                                                                   \
+                head_gate, gate_ld, sink);                                                                             \
     }
     if (hd == 128) LAUNCH(128) else LAUNCH(64)
 #undef LAUNCH

@@ -3,8 +3,9 @@
 // and a single decoded token alike (every row carries its own position), any head size
 // up to 256, any group size, float32 or bfloat16 storage; all arithmetic is float32.
 // Values may have another size than keys (vd), a score may be capped,
-// s <- cap * tanh(s / cap), and a head's output may be multiplied by the sigmoid of a gate
-// value of its own (one float32 per row and head).
+// s <- cap * tanh(s / cap), a head's output may be multiplied by the sigmoid of a gate
+// value of its own (one float32 per row and head), and the softmax's divisor may hold exp(sink) for a constant
+// score `sink` of a key without a value (neither scaled nor capped; 0 adds one to the divisor).
 //
 // For head h, kv head = h / (heads / kv_heads); keys t in [from, p] with
 // from = p + 1 - w when w > 0 and p + 1 > w, else 0; s_t = (q . k_t) * scale; softmax
@@ -29,7 +30,7 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_kernel(
     const TQ* __restrict__ q, TO* __restrict__ out, const TC* __restrict__ kplane, const TC* __restrict__ vplane,
     const int* __restrict__ positions, const int* __restrict__ row_req, const int* __restrict__ table,
     int table_stride, int page_tokens, int n_heads, int n_kv, int hd, int vd, int window, float scale, float softcap,
-    const float* __restrict__ head_gate, int gate_ld) {
+    const float* __restrict__ head_gate, int gate_ld, float sink) {
     cj::after_predecessor();
     cj::release_successor();
     extern __shared__ float smem[];
@@ -98,11 +99,11 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_kernel(
         if (d < vd) acc_s[warp * vd + d] = acc[i];
     }
     __syncthreads();
-    float mx = m_s[0];
+    float mx = fmaxf(m_s[0], sink);         // sink = -inf: none, its term below is zero
 #pragma unroll
     for (int w = 1; w < WARPS; ++w) mx = fmaxf(mx, m_s[w]);
     float f[WARPS];
-    float lsum = 0.0f;
+    float lsum = expf(sink - mx);
 #pragma unroll
     for (int w = 0; w < WARPS; ++w) {
         f[w] = (m_s[w] == -INFINITY) ? 0.0f : expf(m_s[w] - mx);
@@ -259,10 +260,11 @@ CJ_EXPORT int cj_mixed_heads_attention(const void* q, void* out, int act_dtype, 
 
 // q [T, n_heads, hd], out [T, n_heads, vd] in the activation dtype; planes [pages, n_kv, page_tokens, hd | vd].
 // softcap 0: none.  head_gate: null, or float32 with row stride gate_ld whose entry [t, h] gates head h of row t.
+// sink: a constant score of one more key that has no value, exp(sink) in the divisor alone; -infinity: none.
 CJ_EXPORT int cj_paged_attention(const void* q, void* out, int act_dtype, const void* kplane, const void* vplane,
                                  int cache_dtype, const int* positions, const int* row_req, const int* table,
                                  int table_stride, int page_tokens, int T, int n_heads, int n_kv, int hd, int vd,
-                                 int window, float scale, float softcap, const float* head_gate, int gate_ld,
+                                 int window, float scale, float softcap, const float* head_gate, int gate_ld, float sink,
                                  cudaStream_t stream) {
     if (T <= 0) return 0;
     if (!q || !out || !kplane || !vplane || !positions || !row_req || !table) return CJ_ERR_ARG;
@@ -274,7 +276,7 @@ CJ_EXPORT int cj_paged_attention(const void* q, void* out, int act_dtype, const 
 #define LAUNCH(TQ, TC)                                                                                             \
     cj::launch(paged_attention_kernel<TQ, TC, TQ>, dim3(grid), dim3(WARPS * 32), smem, stream, (const TQ*)q, (TQ*)out, (const TC*)kplane, \
         (const TC*)vplane, positions, row_req, table, table_stride, page_tokens, n_heads, n_kv, hd, vd, window, scale, softcap, \
-        head_gate, gate_ld)
+        head_gate, gate_ld, sink)
     if (act_dtype == CJ_F32 && cache_dtype == CJ_F32) LAUNCH(float, float);
     else if (act_dtype == CJ_BF16 && cache_dtype == CJ_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);
     else return CJ_ERR_DTYPE;
@@ -295,6 +297,9 @@ CJ_EXPORT int cj_paged_attention(const void* q, void* out, int act_dtype, const 
 // that grows with the row's position p in steps of `every` tokens.
 // `whole`: the norm's statistic is taken over all heads of q (of k) at once, mean over n_heads * hd
 // (n_kv * hd) entries, and the weight has that many entries, a head reading its own stretch.
+// Flags (HP_*): UNIT_QK norms the heads of q and k without a weight (a rotation keeps a head's length, so with no
+// weight it is the same before the rotation or after it); UNIT_V divides every value by its root mean square over vd
+// before it is written; PAIRS rotates entry 2i with entry 2i + 1 instead of entry i with i + rot/2.
 // ---------------------------------------------------------------------------------
 __device__ __forceinline__ void store4(float* dst, float4 v) { *(float4*)dst = v; }
 __device__ __forceinline__ void store4(__nv_bfloat16* dst, float4 v) {
@@ -310,12 +315,14 @@ __device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(
 // One block per row (with few rows the row's heads are shared out over gridDim.y blocks): the row's cos
 // and sin are worked out once into shared memory, then a warp takes a head at a time.  Head sizes, rotary
 // parts and offsets that are multiples of four go four entries a lane (16-byte loads, 8- or 16-byte stores).
+constexpr int HP_WHOLE = 1, HP_UNIT_QK = 2, HP_UNIT_V = 4, HP_PAIRS = 8;
+
 template <typename TQ, typename TC>
 __global__ void __launch_bounds__(128) head_prepare_kernel(
     const float* __restrict__ x, int ld, int q_off, int k_off, int v_off, TQ* __restrict__ q_out, TC* __restrict__ kplane,
     TC* __restrict__ vplane, const int* __restrict__ positions, const int* __restrict__ row_req, const int* __restrict__ table,
     int table_stride, int page_tokens, int T, int n_heads, int n_kv, int hd, int vd, int rot, const float* __restrict__ inv_freq,
-    float magnitude, const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps, int write_kv, int whole,
+    float magnitude, const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps, int write_kv, int flags,
     float q_temp_coef, int q_temp_every) {
     cj::after_predecessor();
     cj::release_successor();
@@ -325,6 +332,8 @@ __global__ void __launch_bounds__(128) head_prepare_kernel(
     const int t = blockIdx.x;
     const int pos = positions[t];
     const int half = rot >> 1;
+    const bool whole = (flags & HP_WHOLE) != 0, unit_qk = (flags & HP_UNIT_QK) != 0, unit_v = (flags & HP_UNIT_V) != 0;
+    const bool pairs = (flags & HP_PAIRS) != 0;
     // a query's temperature grows with its position in steps of `every` tokens: 1 + coef ln(floor((p + 1) / every) + 1)
     const float q_temp = q_temp_coef != 0.0f ? 1.0f + q_temp_coef * logf((float)((pos + 1) / q_temp_every) + 1.0f) : 1.0f;
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
@@ -358,7 +367,7 @@ __global__ void __launch_bounds__(128) head_prepare_kernel(
         inv_whole[1] = 1.0f / sqrtf(sk / (float)(n_kv > 0 ? n_kv * hd : 1) + eps);
     }
     const int slots = n_heads + (write_kv && have_page ? n_kv : 0);
-    const bool vec = (hd % 4 == 0) && hd <= 256 && (half % 4 == 0) && (vd % 4 == 0) && ((ld | q_off | k_off | (v_off < 0 ? 0 : v_off)) % 4 == 0) &&
+    const bool vec = (hd % 4 == 0) && hd <= 256 && (half % (pairs ? 2 : 4) == 0) && (vd % 4 == 0) && vd <= 256 && ((ld | q_off | k_off | (v_off < 0 ? 0 : v_off)) % 4 == 0) &&
                      ((((uintptr_t)x) | ((uintptr_t)q_out) | ((uintptr_t)kplane) | ((uintptr_t)vplane) | ((uintptr_t)q_norm) |
                        ((uintptr_t)k_norm)) & 15) == 0;
     for (int slot = blockIdx.y * 4 + warp; slot < slots; slot += gridDim.y * 4) {
@@ -381,7 +390,7 @@ __global__ void __launch_bounds__(128) head_prepare_kernel(
         }
         if (nw && whole) {
             inv = inv_whole[is_q ? 0 : 1];
-        } else if (nw) {
+        } else if (nw || unit_qk) {
             float ss = 0.0f;
             if (vec) {
 #pragma unroll
@@ -403,7 +412,12 @@ __global__ void __launch_bounds__(128) head_prepare_kernel(
                 if (d >= hd) break;
                 float4 a = mul4(held[k], inv);
                 if (nw) a = mul4(a, *(const float4*)(nw + d));
-                if (d < rot) {
+                if (pairs && d < rot) {
+                    const int i = d >> 1;                    // entries d .. d + 3: pairs i and i + 1 (d and half are even in i)
+                    const float2 c = *(const float2*)(cs + i), sn = *(const float2*)(cs + half + i);
+                    a = make_float4(fmaf(-a.y, sn.x, a.x * c.x), fmaf(a.x, sn.x, a.y * c.x), fmaf(-a.w, sn.y, a.z * c.y),
+                                    fmaf(a.z, sn.y, a.w * c.y));
+                } else if (d < rot) {
                     const bool low = d < half;
                     const int i = low ? d : d - half, pd = low ? d + half : d - half;
                     float4 b = mul4(*(const float4*)(src + pd), inv);
@@ -418,7 +432,25 @@ __global__ void __launch_bounds__(128) head_prepare_kernel(
             }
             if (!is_q) {
                 const float* vs = v_off < 0 ? src : xrow + v_off + head * vd;
-                for (int d = lane * 4; d < vd; d += 128) store4(vplane + place * vd + d, *(const float4*)(vs + d));
+                float4 val[2];
+#pragma unroll
+                for (int k = 0; k < 2; ++k) {
+                    const int d = lane * 4 + k * 128;
+                    val[k] = d < vd ? *(const float4*)(vs + d) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                }
+                float vinv = 1.0f;
+                if (unit_v) {
+                    float ss = 0.0f;
+#pragma unroll
+                    for (int k = 0; k < 2; ++k)
+                        ss = fmaf(val[k].x, val[k].x, fmaf(val[k].y, val[k].y, fmaf(val[k].z, val[k].z, fmaf(val[k].w, val[k].w, ss))));
+                    vinv = 1.0f / sqrtf(warp_sum(ss) / (float)vd + eps);
+                }
+#pragma unroll
+                for (int k = 0; k < 2; ++k) {
+                    const int d = lane * 4 + k * 128;
+                    if (d < vd) store4(vplane + place * vd + d, mul4(val[k], vinv));
+                }
             }
             continue;
         }
@@ -426,16 +458,23 @@ __global__ void __launch_bounds__(128) head_prepare_kernel(
             float a = src[d] * inv * (nw ? nw[d] : 1.0f);
             float r = a;
             if (d < rot) {
-                const int i = d < half ? d : d - half, pd = d < half ? d + half : d - half;
+                const bool low = pairs ? (d & 1) == 0 : d < half;       // the pair's first entry
+                const int i = pairs ? d >> 1 : (low ? d : d - half), pd = pairs ? d ^ 1 : (low ? d + half : d - half);
                 const float b = src[pd] * inv * (nw ? nw[pd] : 1.0f);
-                r = d < half ? a * cs[i] - b * cs[half + i] : a * cs[i] + b * cs[half + i];
+                r = low ? a * cs[i] - b * cs[half + i] : a * cs[i] + b * cs[half + i];
             }
             if (is_q) q_out[((size_t)t * n_heads + head) * hd + d] = from_f32<TQ>(r);
             else kplane[place * hd + d] = from_f32<TC>(r);
         }
         if (!is_q) {
             const float* vs = v_off < 0 ? src : xrow + v_off + head * vd;
-            for (int d = lane; d < vd; d += 32) vplane[place * vd + d] = from_f32<TC>(vs[d]);
+            float vinv = 1.0f;
+            if (unit_v) {
+                float ss = 0.0f;
+                for (int d = lane; d < vd; d += 32) ss = fmaf(vs[d], vs[d], ss);
+                vinv = 1.0f / sqrtf(warp_sum(ss) / (float)vd + eps);
+            }
+            for (int d = lane; d < vd; d += 32) vplane[place * vd + d] = from_f32<TC>(vs[d] * vinv);
         }
     }
 }
@@ -444,13 +483,14 @@ CJ_EXPORT int cj_head_prepare(const float* x, int ld, int q_off, int k_off, int 
                               void* vplane, int cache_dtype, const int* positions, const int* row_req, const int* table,
                               int table_stride, int page_tokens, int T, int n_heads, int n_kv, int hd, int vd, int rotary_dim,
                               const float* inv_freq, float magnitude, const float* q_norm, const float* k_norm, float eps,
-                              int write_kv, int whole, float q_temp_coef, int q_temp_every, cudaStream_t stream) {
+                              int write_kv, int flags, float q_temp_coef, int q_temp_every, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (!x || !q_out || !positions || n_heads <= 0 || hd <= 0 || vd <= 0) return CJ_ERR_ARG;
     if (rotary_dim < 0 || rotary_dim > hd || (rotary_dim & 1)) return CJ_ERR_SIZE;
     if (rotary_dim > 0 && !inv_freq) return CJ_ERR_ARG;
     if (write_kv && (!kplane || !vplane || !row_req || !table || page_tokens <= 0 || n_kv <= 0)) return CJ_ERR_ARG;
     if (v_off < 0 && vd != hd) return CJ_ERR_SIZE;
+    if ((flags & HP_UNIT_QK) && (q_norm || k_norm || (flags & HP_WHOLE))) return CJ_ERR_ARG;
     if (q_temp_coef != 0.0f && q_temp_every < 1) return CJ_ERR_SIZE;
     // a warp a head; with few rows the heads of a row go over several blocks
     const int slots = n_heads + (write_kv ? n_kv : 0);
@@ -461,7 +501,7 @@ CJ_EXPORT int cj_head_prepare(const float* x, int ld, int q_off, int k_off, int 
 #define LAUNCH(TQ, TC)                                                                                                  \
     cj::launch(head_prepare_kernel<TQ, TC>, dim3(grid), dim3(128), smem, stream, x, ld, q_off, k_off, v_off, (TQ*)q_out,  \
         (TC*)kplane, (TC*)vplane, positions, row_req, table, table_stride, page_tokens, T, n_heads, n_kv, hd, vd,      \
-        rotary_dim, inv_freq, magnitude, q_norm, k_norm, eps, write_kv, whole, q_temp_coef, q_temp_every)
+        rotary_dim, inv_freq, magnitude, q_norm, k_norm, eps, write_kv, flags, q_temp_coef, q_temp_every)
     if (q_dtype == CJ_F32 && cache_dtype == CJ_F32) LAUNCH(float, float);
     else if (q_dtype == CJ_BF16 && cache_dtype == CJ_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);
     else return CJ_ERR_DTYPE;

@@ -7,8 +7,9 @@
 // Per row at position p: keys [from, p], from = p + 1 - w when a window is set and
 // exceeded, else 0; s = (q . k) * scale; softmax with the running maximum subtracted;
 // o = (sum e v) / (sum e)  (model/PagedKvCache.cajeta:374-470).  Optionally a score is capped,
-// s <- cap * tanh(s / cap) after the scale, and a head's output is multiplied by the sigmoid of a
-// gate value of its own (float32, one per row and head).  The reference's
+// s <- cap * tanh(s / cap) after the scale, a head's output is multiplied by the sigmoid of a
+// gate value of its own (float32, one per row and head), and the divisor also holds exp(sink) for a constant score
+// `sink` of a key without a value.  The reference's
 // counterpart is its query-tiled flash prefill over the page table
 // (model/AttnKernel.cajeta:2903).
 //
@@ -65,7 +66,7 @@ __global__ void __launch_bounds__(BM / (16 * MT) * 32) prefill_attention_kernel(
     const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ kplane,
     const __nv_bfloat16* __restrict__ vplane, const int* __restrict__ req_start, const int* __restrict__ req_prior,
     int n_requests, const int* __restrict__ table, int table_stride, int page_tokens, int n_heads, int n_kv, int window,
-    float scale, float softcap, const float* __restrict__ head_gate, int gate_ld) {
+    float scale, float softcap, const float* __restrict__ head_gate, int gate_ld, float sink_log2) {
     cj::after_predecessor();
     cj::release_successor();
     extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -256,6 +257,9 @@ __global__ void __launch_bounds__(BM / (16 * MT) * 32) prefill_attention_kernel(
         l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
         l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
         l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+        // the key without a value (sink_log2 = -inf: none); a row without keys keeps zero
+        if (l0 > 0.0f) l0 += exp2f(sink_log2 - mrun[mt][0]);
+        if (l1 > 0.0f) l1 += exp2f(sink_log2 - mrun[mt][1]);
         float i0 = l0 > 0.0f ? 1.0f / l0 : 0.0f, i1 = l1 > 0.0f ? 1.0f / l1 : 0.0f;
         const int r0 = wrow + mt * 16 + g, r1 = r0 + 8;
         if (head_gate) {
@@ -277,10 +281,11 @@ __global__ void __launch_bounds__(BM / (16 * MT) * 32) prefill_attention_kernel(
 // [n_requests + 1], req_prior [n_requests] as the step function lays them out.  hd must be
 // 32, 64, 96 or 128.  block_rows: 64 or 128 query rows a block, 0 = chosen from the step's shape.  softcap 0: none.
 // head_gate: null, or float32 with row stride gate_ld whose entry [t, h] gates head h of row t.
+// sink: a constant score of one more key that has no value, exp(sink) in the divisor alone; -infinity: none.
 CJ_EXPORT int cj_prefill_attention(const void* q, void* out, const void* kplane, const void* vplane, const int* req_start,
                                    const int* req_prior, int n_requests, int total_rows, const int* table, int table_stride,
                                    int page_tokens, int n_heads, int n_kv, int hd, int window, float scale,
-                                   int block_rows, float softcap, const float* head_gate, int gate_ld, cudaStream_t stream) {
+                                   int block_rows, float softcap, const float* head_gate, int gate_ld, float sink, cudaStream_t stream) {
     if (total_rows <= 0 || n_requests <= 0) return 0;
     if (!q || !out || !kplane || !vplane || !req_start || !req_prior || !table) return CJ_ERR_ARG;
     if (n_heads <= 0 || n_kv <= 0 || n_heads % n_kv != 0 || page_tokens <= 0 || n_heads > 65535) return CJ_ERR_SIZE;
@@ -300,7 +305,7 @@ CJ_EXPORT int cj_prefill_attention(const void* q, void* out, const void* kplane,
         cj::launch(prefill_attention_kernel<HD, HS, BM, BN, MT>, dim3(grid), dim3(BM / (16 * MT) * 32), smem, stream,                           \
             (const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)kplane, (const __nv_bfloat16*)vplane,   \
             req_start, req_prior, n_requests, table, table_stride, page_tokens, n_heads, n_kv, window, scale, softcap,  \
-            head_gate, gate_ld);                                                                                        \
+            head_gate, gate_ld, sink * 1.4426950408889634f);                                                            \
     }
     if (hd == 128) { if (bm == 128) LAUNCH(128, 128, 128, 32, 2) else LAUNCH(128, 128, 64, 64, 1) }
     else if (hd == 96) { if (bm == 128) LAUNCH(96, 128, 128, 32, 2) else LAUNCH(96, 128, 64, 64, 1) }

@@ -149,10 +149,33 @@ __device__ __forceinline__ float capped_score(float s, float in_cap, float cap_l
     return s == -INFINITY ? -INFINITY : y;
 }
 
+// Capped scores in full float32.  CAP_POLY: every |s| scale / cap is known to be at most CAP_POLY_REACH (queries and keys of
+// known length), where tanh(x) = x P(x^2) with the P below, whose relative error over that reach is 1.1e-7 (a minimax fit of
+// tanh(x) / x in x^2 with five terms); the arguments' scaling and the cap are folded into the terms by the host, so a score
+// costs three packed multiply-adds and no second special function.  CAP_EXP: any score, tanh(x) = 1 - 2 / (e^2x + 1).
+constexpr int CAP_NONE = 0, CAP_APPROX = 1, CAP_POLY = 2, CAP_EXP = 3;
+constexpr float CAP_POLY_REACH = 0.625f;
+constexpr int CAP_TERMS = 5;
+constexpr double CAP_P[CAP_TERMS] = {0.9999998931, -0.3333195425, 0.1330452599, -0.05182186644, 0.01505094485};
+
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+
 __device__ __forceinline__ float ex2(float x) {       // 2^x, 0 for -inf
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
+}
+
+__device__ __forceinline__ float capped_score_exp(float s, float in_cap, float cap_log2, float neg_sub) {
+    const float e = ex2(s * in_cap * 2.8853900817779268f);                   // e^2x
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.0f));
+    const float y = fmaf(r, -2.0f * cap_log2, cap_log2 + neg_sub);
+    return s == -INFINITY ? -INFINITY : y;
 }
 
 // 32 consecutive 32-bit columns of this thread's lane into v[OFF .. OFF + 31]
@@ -180,7 +203,9 @@ struct Args {
     const int* table;
     int n_requests, table_stride, page_tokens, n_heads, n_kv, window;
     float scale_log2;
-    float cap_log2, in_cap;    // capped scores: cap log2(e) and scale / cap (the kernel's CAPPED form)
+    float cap_log2, in_cap;    // capped scores: cap log2(e) and scale / cap (the kernel's CAP forms)
+    float cap_p[CAP_TERMS];    // CAP_POLY: P's terms with both folded in, a score s becomes s P(s^2) in units of log 2
+    float sink_log2;           // score of a key without a value in units of log 2; -infinity: none
     const float* head_gate;    // null, or float32 [rows, gate_ld]: head h of row t is multiplied by sigmoid(head_gate[t, h])
     int gate_ld;
     int plane_rows;            // rows of the [pages * n_kv * page_tokens, 128] view of a cache plane
@@ -194,7 +219,7 @@ struct QueryTile {
     int begin, end;    // key tiles [begin, end] it needs, counted from the block's first key tile (begin > end: none)
 };
 
-template <bool CAPPED>
+template <int CAP>
 __global__ void __launch_bounds__(THREADS, 1)
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, Args p) {
@@ -441,7 +466,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 tmem_ld32<0>(s_addr + half * HC, v);
                 tmem_ld32<32>(s_addr + half * HC + 32, v);
                 tmem_ld_wait();
-                if (lo != 0 || span != BN - 1) {
+                const bool partial = lo != 0 || span != BN - 1;
+                if (partial) {
 #pragma unroll
                     for (int c = 0; c < HC; ++c)
                         if (!((unsigned)(half * HC + c - lo) <= (unsigned)span && span >= 0)) v[c] = 0xff800000u;       // -inf
@@ -464,7 +490,31 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
                     for (int c = 0; c < HC; c += 4) {
                         float2 t0, t1;
-                        if (CAPPED) {
+                        if (CAP == CAP_POLY) {
+                            const f32x2 s0 = pack2(__uint_as_float(v[c]), __uint_as_float(v[c + 1]));
+                            const f32x2 s1 = pack2(__uint_as_float(v[c + 2]), __uint_as_float(v[c + 3]));
+                            const f32x2 x0 = mul2(s0, s0), x1 = mul2(s1, s1);
+                            f32x2 p0 = pack2(p.cap_p[CAP_TERMS - 1], p.cap_p[CAP_TERMS - 1]), p1 = p0;
+#pragma unroll
+                            for (int k = CAP_TERMS - 2; k >= 0; --k) {
+                                const f32x2 ck = pack2(p.cap_p[k], p.cap_p[k]);
+                                p0 = fma2(p0, x0, ck);
+                                p1 = fma2(p1, x1, ck);
+                            }
+                            t0 = unpack2(fma2(p0, s0, sub2));
+                            t1 = unpack2(fma2(p1, s1, sub2));
+                            if (partial) {                     // a masked score (-inf) stays -inf
+                                t0.x = __uint_as_float(v[c]) == -INFINITY ? -INFINITY : t0.x;
+                                t0.y = __uint_as_float(v[c + 1]) == -INFINITY ? -INFINITY : t0.y;
+                                t1.x = __uint_as_float(v[c + 2]) == -INFINITY ? -INFINITY : t1.x;
+                                t1.y = __uint_as_float(v[c + 3]) == -INFINITY ? -INFINITY : t1.y;
+                            }
+                        } else if (CAP == CAP_EXP) {
+                            t0 = make_float2(capped_score_exp(__uint_as_float(v[c]), p.in_cap, p.cap_log2, neg_sub),
+                                             capped_score_exp(__uint_as_float(v[c + 1]), p.in_cap, p.cap_log2, neg_sub));
+                            t1 = make_float2(capped_score_exp(__uint_as_float(v[c + 2]), p.in_cap, p.cap_log2, neg_sub),
+                                             capped_score_exp(__uint_as_float(v[c + 3]), p.in_cap, p.cap_log2, neg_sub));
+                        } else if (CAP == CAP_APPROX) {
                             t0 = make_float2(capped_score(__uint_as_float(v[c]), p.in_cap, p.cap_log2, neg_sub),
                                              capped_score(__uint_as_float(v[c + 1]), p.in_cap, p.cap_log2, neg_sub));
                             t1 = make_float2(capped_score(__uint_as_float(v[c + 2]), p.in_cap, p.cap_log2, neg_sub),
@@ -486,7 +536,9 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     sum = (sa.x + sa.y) + (sb.x + sb.y);
                     if (attempt == 1) break;
                     // scale > 0, and capping keeps the order: the largest raw score is the largest score
-                    const float mx = CAPPED ? capped_score(fmaxf(mx0, mx1), p.in_cap, p.cap_log2, 0.0f) : fmaxf(mx0, mx1) * p.scale_log2;
+                    const float mx_raw = fmaxf(mx0, mx1);
+                    const float mx = CAP == CAP_NONE ? mx_raw * p.scale_log2 : CAP == CAP_APPROX ? capped_score(mx_raw, p.in_cap, p.cap_log2, 0.0f)
+                                     : capped_score_exp(mx_raw, p.in_cap, p.cap_log2, 0.0f);       // only a reference for the sums
                     float m_new = m_ref;
                     if (mx > m_ref + RESCALE_THRESHOLD || m_ref == -INFINITY) m_new = fmaxf(m_ref, mx);
                     if (!__any_sync(0xffffffffu, m_new != m_ref)) break;
@@ -527,6 +579,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         if (ok && n_mine > 0) ok = __all_sync(0xffffffffu, mbar_wait(&o_done[g], 0, 18));
         if (ok && n_mine > 0) {
             tcgen05_fence_after();
+            if (l > 0.0f) l += exp2f(p.sink_log2 - m_ref);           // the key without a value
             float inv = l > 0.0f ? 1.0f / l : 0.0f;
             if (p.head_gate && r < mine.rows) inv *= 1.0f / (1.0f + expf(-p.head_gate[(size_t)(row0 + g * BM + r) * p.gate_ld + h]));
             __nv_bfloat16* dst = p.out + ((size_t)(row0 + g * BM + r) * p.n_heads + h) * HD;
@@ -568,12 +621,16 @@ bool make_map(CUtensorMap* map, const void* base, long long rows, long long cols
 // q, out: [T, n_heads, 128] bf16; planes [pages, n_kv, 16, 128] bf16; req_start [n_requests + 1],
 // req_prior [n_requests].  Head size 128 and 16-token pages only; refuses anything else.  force_block_rows: 128 or 256
 // query rows a block, or 0 to let the launch's size decide.  softcap > 0: a score becomes cap tanh(s / cap)
-// after the scale.  head_gate: null, or float32 with row stride gate_ld whose entry [t, h] gates head h of row t.
+// after the scale; exact_cap 0: by the special-function unit's tangent, 1: in full float32 (score_bound > 0: no |q . k| scale
+// is larger, which allows the cheaper of the two exact forms).  head_gate: null, or float32 with row stride gate_ld whose
+// entry [t, h] gates head h of row t.  sink: a constant score of one more key that has no value, exp(sink) in the
+// divisor alone; -infinity: none.
 CJ_EXPORT int cj_prefill_attention_tc(const void* q, void* out, const void* kplane, const void* vplane, int n_pages,
                                       const int* req_start, const int* req_prior, int n_requests, int total_rows,
                                       const int* table, int table_stride, int page_tokens, int n_heads, int n_kv,
                                       int hd, int window, float scale, int force_block_rows, float softcap,
-                                      const float* head_gate, int gate_ld, cudaStream_t stream) {
+                                      int exact_cap, float score_bound, const float* head_gate, int gate_ld, float sink,
+                                      cudaStream_t stream) {
     if (total_rows <= 0 || n_requests <= 0) return 0;
     if (!q || !out || !kplane || !vplane || !req_start || !req_prior || !table) return CJ_ERR_ARG;
     if (hd != HD || page_tokens != 16) return CJ_ERR_SIZE;
@@ -587,9 +644,13 @@ CJ_EXPORT int cj_prefill_attention_tc(const void* q, void* out, const void* kpla
     if (!make_map(&mv, vplane, plane_rows, HD, HD, 16)) return CJ_ERR_ARG;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
+        cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<CAP_NONE>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
         if (e == cudaSuccess)
-            e = cudaFuncSetAttribute(prefill_attention_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
+            e = cudaFuncSetAttribute(prefill_attention_tc_kernel<CAP_APPROX>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
+        if (e == cudaSuccess)
+            e = cudaFuncSetAttribute(prefill_attention_tc_kernel<CAP_POLY>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
+        if (e == cudaSuccess)
+            e = cudaFuncSetAttribute(prefill_attention_tc_kernel<CAP_EXP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
@@ -610,14 +671,23 @@ CJ_EXPORT int cj_prefill_attention_tc(const void* q, void* out, const void* kpla
     }
     Args a{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, req_start, req_prior, table, n_requests, table_stride, page_tokens,
            n_heads, n_kv, window, scale * 1.4426950408889634f, softcap * 1.4426950408889634f,
-           softcap > 0.0f ? scale / softcap : 0.0f, head_gate, gate_ld, (int)plane_rows, block_rows};
+           softcap > 0.0f ? scale / softcap : 0.0f, {}, sink * 1.4426950408889634f, head_gate, gate_ld, (int)plane_rows, block_rows};
+    int cap = softcap > 0.0f ? CAP_APPROX : CAP_NONE;
+    if (softcap > 0.0f && exact_cap) {
+        cap = score_bound > 0.0f && score_bound <= CAP_POLY_REACH * softcap ? CAP_POLY : CAP_EXP;
+        // cap log2(e) tanh(x), x = s scale / cap: the k-th term carries x^(2k + 1)
+        const double x = (double)scale / (double)softcap;
+        double f = (double)softcap * 1.4426950408889634 * x;
+        for (int k = 0; k < CAP_TERMS; ++k, f *= x * x) a.cap_p[k] = (float)(CAP_P[k] * f);
+    }
     // heads run fastest, so that blocks start in the order of their length (the last rows of a
     // request see the most keys) and the heads of one group read the same keys one after another
     const long long row_blocks = (total_rows + block_rows - 1) / block_rows + n_requests;
     if (row_blocks > 65535) return CJ_ERR_SIZE;
     dim3 grid(n_heads, (unsigned)row_blocks);
-    if (softcap > 0.0f) cj::launch(prefill_attention_tc_kernel<true>, dim3(grid), dim3(THREADS), SMEM_TOTAL, stream, mq, mk, mv, a);
-    else cj::launch(prefill_attention_tc_kernel<false>, dim3(grid), dim3(THREADS), SMEM_TOTAL, stream, mq, mk, mv, a);
+    auto kern = cap == CAP_NONE ? prefill_attention_tc_kernel<CAP_NONE> : cap == CAP_APPROX ? prefill_attention_tc_kernel<CAP_APPROX>
+                : cap == CAP_POLY ? prefill_attention_tc_kernel<CAP_POLY> : prefill_attention_tc_kernel<CAP_EXP>;
+    cj::launch(kern, dim3(grid), dim3(THREADS), SMEM_TOTAL, stream, mq, mk, mv, a);
     return cj::launch_status();
 }
 

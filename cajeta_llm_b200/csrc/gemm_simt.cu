@@ -1,4 +1,4 @@
-// Matrix products on the float32 FMA pipe:  C[M,N] (+)= A[M,K] . W[N,K]^T (+ bias).
+// Matrix products on the float32 FMA pipe:  C[M,N] (+)= scale (A[M,K] . W[N,K]^T (+ bias)).
 //
 // This is the true 32-bit path of every projection (no reduced-precision matrix mode)
 // and the general fallback of the bfloat16 path for sizes the tensor-core kernels
@@ -34,6 +34,7 @@ struct GemmArgs {
     long long w_group_stride;
     int num_groups;
     float act_limit, act_alpha;   // the gated form's activation (see gated_act)
+    float out_scale;              // multiplies the sum (bias included) before it is stored or added; 1 = as it is
 };
 
 template <typename TA, typename TW, typename TC, bool SWIGLU>
@@ -144,6 +145,7 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(GemmArgs p) {
             float v = acc[i][j];
             if (SWIGLU) v = gated_act(v, acc2[i][j], p.act_limit, p.act_alpha);
             if (p.bias) v += p.bias[c];
+            v *= p.out_scale;
             size_t o = (size_t)r * p.ldc + c;
             if (p.accumulate) v += to_f32(C[o]);
             C[o] = from_f32<TC>(v);
@@ -168,11 +170,11 @@ int launch(const GemmArgs& p, bool swiglu, cudaStream_t stream) {
 CJ_EXPORT int cj_gemm_simt(const void* A, long long lda, int a_dtype, const void* W, const void* W2, long long ldw,
                            int w_dtype, const float* bias, void* C, long long ldc, int c_dtype, int M, int N, int K,
                            int accumulate, const int* group_offsets, int num_groups, long long w_group_stride,
-                           const int* a_row_index, float act_limit, float act_alpha, cudaStream_t stream) {
+                           const int* a_row_index, float act_limit, float act_alpha, float out_scale, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (!A || !W || !C || K <= 0) return CJ_ERR_ARG;
     if (group_offsets && num_groups <= 0) return CJ_ERR_ARG;
-    GemmArgs p{A, lda, W, W2, ldw, bias, C, ldc, M, N, K, accumulate, group_offsets, a_row_index, w_group_stride, num_groups, act_limit, act_alpha};
+    GemmArgs p{A, lda, W, W2, ldw, bias, C, ldc, M, N, K, accumulate, group_offsets, a_row_index, w_group_stride, num_groups, act_limit, act_alpha, out_scale};
     bool sw = W2 != nullptr;
     if (a_dtype == CJ_F32 && w_dtype == CJ_F32 && c_dtype == CJ_F32) return launch<float, float, float>(p, sw, stream);
     if (a_dtype == CJ_BF16 && w_dtype == CJ_BF16 && c_dtype == CJ_F32) return launch<__nv_bfloat16, __nv_bfloat16, float>(p, sw, stream);

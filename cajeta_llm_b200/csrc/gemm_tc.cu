@@ -57,6 +57,7 @@ struct Args {
     long long split_stride;
     int offsets_settled;        // the groups' offsets were complete before the kernel before this one began
     float act_limit, act_alpha; // the gated form's activation (see gated_act)
+    float out_scale;            // float32 store / accumulate: multiplies the sum (bias included); 1 = as it is
     int choose_height;          // grouped, weights on the rows: the tile's height is chosen in the kernel (see LowTiles)
 };
 
@@ -386,6 +387,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
                         for (int j = 0; j < 16; ++j) { const float t = fmaxf(v[j], 0.0f); v[j] = t * t; }
                     }
                     if (EPI == EPI_STORE_F32 || EPI == EPI_ACC_F32) {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) v[j] *= p.out_scale;
                         float* dst = (float*)p.out + o + (EPI == EPI_STORE_F32 ? split_off : 0);
                         if (whole && (((uintptr_t)dst) & 15) == 0) {
 #pragma unroll
@@ -432,6 +435,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
                         long long o = (long long)token * p.ldo + feat;
                         float val = v[j] + b;
                         if (EPI == EPI_RELU2_BF16) { val = fmaxf(val, 0.0f); val *= val; }
+                        if (EPI == EPI_STORE_F32 || EPI == EPI_ACC_F32) val *= p.out_scale;
                         if (EPI == EPI_STORE_F32) ((float*)p.out)[o + split_off] = val;
                         else if (EPI == EPI_ACC_F32) ((float*)p.out)[o] += val;
                         else ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(val);
@@ -536,7 +540,7 @@ int dispatch_n(int n_mma, const CUtensorMap& mx, const CUtensorMap& mw, const CU
 // x: [tokens, K] bf16 with row stride ldx; w (and w2 for SwiGLU): [groups * features, K] bf16,
 // contiguous.  swap: 0 = tokens on the product's rows (tile 128 tokens x n_mma features),
 // 1 = weights on the rows (tile 128 features x n_mma tokens).  epilogue: 0 float32 store,
-// 1 float32 accumulate, 2 SwiGLU to bf16 (needs w2), 3 bf16 store.  k_splits > 1 only with
+// 1 float32 accumulate, 2 SwiGLU to bf16 (needs w2), 3 bf16 store (0 and 1: out_scale multiplies the sum).  k_splits > 1 only with
 // epilogue 0: split s stores its partial sum at out + s * split_stride (the bias goes to
 // split 0).  offsets_settled: non-zero if group_offsets were complete before the kernel
 // before this launch began (not merely before this launch): the kernel then reads them, and
@@ -545,7 +549,7 @@ int dispatch_n(int n_mma, const CUtensorMap& mx, const CUtensorMap& mw, const CU
 CJ_EXPORT int cj_gemm_tc(const void* x, long long ldx, const void* w, const void* w2, const float* bias, void* out,
                          long long ldo, int tokens, int features, int K, int epilogue, int swap, int n_mma,
                          const int* group_offsets, int groups, int k_splits, long long split_stride,
-                         int offsets_settled, float act_limit, float act_alpha, cudaStream_t stream) {
+                         int offsets_settled, float act_limit, float act_alpha, float out_scale, cudaStream_t stream) {
     if (tokens <= 0 || features <= 0) return 0;
     if (!x || !w || !out || K <= 0) return CJ_ERR_ARG;
     if (K % 8 != 0 || ldx % 8 != 0) return CJ_ERR_ALIGN;               // TMA: 16-byte strides
@@ -571,7 +575,7 @@ CJ_EXPORT int cj_gemm_tc(const void* x, long long ldx, const void* w, const void
             if (w2 && !make_map_bf16(&low.w2[i], w2, total_w_rows, K, K, low_height(i))) return CJ_ERR_ARG;
         }
     }
-    Args a{tokens, features, K, out, ldo, bias, group_offsets, groups, k_splits, split_stride, offsets_settled, act_limit, act_alpha, choose_height};
+    Args a{tokens, features, K, out, ldo, bias, group_offsets, groups, k_splits, split_stride, offsets_settled, act_limit, act_alpha, out_scale, choose_height};
 #define CASE(EPI, DUAL)                                                                              \
     if (swap) return dispatch_n<true, DUAL, EPI>(n_mma, mx, mw, mw2, low, a, stream);                 \
     else return dispatch_n<false, DUAL, EPI>(n_mma, mx, mw, mw2, low, a, stream);

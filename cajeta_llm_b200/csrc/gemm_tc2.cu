@@ -57,6 +57,7 @@ struct Args {
     const int* group_offsets;
     int groups;
     float act_limit, act_alpha;  // the gated form's activation (see gated_act)
+    float out_scale;             // float32 store / accumulate: multiplies the sum (bias included); 1 = as it is
 };
 
 template <int N_TOK, int STAGES>
@@ -262,14 +263,14 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant
                         for (int j = 0; j < 32; ++j) old[j] = c0 + j < n_cols ? ((const float*)p.out)[o0 + j * p.ldo] : 0.0f;
 #pragma unroll
                         for (int j = 0; j < 32; ++j)
-                            if (c0 + j < n_cols) ((float*)p.out)[o0 + j * p.ldo] = old[j] + __uint_as_float(v[j]) + b;
+                            if (c0 + j < n_cols) ((float*)p.out)[o0 + j * p.ldo] = old[j] + (__uint_as_float(v[j]) + b) * p.out_scale;
                     } else {
 #pragma unroll
                         for (int j = 0; j < 32; ++j) {
                             if (c0 + j >= n_cols) break;
                             float val = __uint_as_float(v[j]) + b;
                             if (EPI == EPI_RELU2_BF16) { val = fmaxf(val, 0.0f); val *= val; }       // an expert without a gate
-                            if (EPI == EPI_STORE_F32) ((float*)p.out)[o0 + j * p.ldo] = val;
+                            if (EPI == EPI_STORE_F32) ((float*)p.out)[o0 + j * p.ldo] = val * p.out_scale;
                             else ((__nv_bfloat16*)p.out)[o0 + j * p.ldo] = __float2bfloat16_rn(val);
                         }
                     }
@@ -562,7 +563,7 @@ int launch_swiglu(const CUtensorMap& mx, const CUtensorMap& mwg, const CUtensorM
 // Refuses (negative code) what it cannot run; never a wrong result.
 CJ_EXPORT int cj_gemm_tc2(const void* x, long long ldx, const void* w, const void* w2, const float* bias, void* out,
                           long long ldo, int tokens, int features, int K, int epilogue, int n_tok,
-                          const int* group_offsets, int groups, float act_limit, float act_alpha, cudaStream_t stream) {
+                          const int* group_offsets, int groups, float act_limit, float act_alpha, float out_scale, cudaStream_t stream) {
     if (tokens <= 0 || features <= 0) return 0;
     if (!x || !w || !out || K <= 0) return CJ_ERR_ARG;
     if (K % 8 != 0 || ldx % 8 != 0) return CJ_ERR_ALIGN;
@@ -575,7 +576,7 @@ CJ_EXPORT int cj_gemm_tc2(const void* x, long long ldx, const void* w, const voi
     int total_w_rows = (group_offsets ? groups : 1) * features;
     CUtensorMap mx, mw, mw2;
     if (!make_map_bf16(&mw, w, total_w_rows, K, K, 128)) return CJ_ERR_ARG;
-    Args a{tokens, features, K, out, ldo, bias, group_offsets, groups, act_limit, act_alpha};
+    Args a{tokens, features, K, out, ldo, bias, group_offsets, groups, act_limit, act_alpha, out_scale};
     if (epilogue == EPI_SWIGLU_BF16) {
         // tokens on the rows: a block's box is 128 token rows whatever n_tok says
         if (!make_map_bf16(&mx, x, tokens, K, ldx, 128)) return CJ_ERR_ARG;

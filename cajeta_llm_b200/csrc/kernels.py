@@ -176,6 +176,38 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor
     _check(st, "rmsnorm")
 
 
+def rmsnorm_pair(x: torch.Tensor, weight_a: torch.Tensor, weight_b: torch.Tensor, eps: float, out_a: torch.Tensor, out_b: torch.Tensor,
+                 partials=()) -> None:
+    """Two RMS norms of the rows of x (float32) that share their statistic: out_a = n(x) weight_a, out_b = n(x) weight_b, in
+    the outputs' dtype.  ``partials``: up to two tensors [S, rows, H] float32 whose slices are added to x first, in order;
+    x keeps the sum."""
+    _need(x, "x", torch.float32), _need(weight_a, "weight_a", torch.float32), _need(weight_b, "weight_b", torch.float32)
+    _need(out_a, "out_a"), _need(out_b, "out_b", out_a.dtype)
+    rows, H = x.shape
+    if out_a.shape != x.shape or out_b.shape != x.shape or weight_a.numel() != H or weight_b.numel() != H:
+        raise KernelError("rmsnorm_pair: shapes do not agree")
+    st = library("rowwise").cj_rmsnorm_pair(_ptr(x), _ptr(weight_a), _ptr(weight_b), _f(eps), _i(rows), _i(H), _ptr(out_a), _ptr(out_b),
+                                            _i(_code(out_a)), *_two_partials(x, partials, "rmsnorm_pair"), _stream())
+    _check(st, "rmsnorm_pair")
+
+
+def _two_partials(x: torch.Tensor, partials, what: str):
+    """(pointer, count, stride) twice, for up to two tensors of partial sums [S, rows, H] owed to x [rows, H]."""
+    partials = [t for t in partials if t is not None]
+    if len(partials) > 2:
+        raise KernelError(f"{what}: at most two sets of partial sums, found {len(partials)}")
+    out = []
+    for t in partials + [None] * (2 - len(partials)):
+        if t is None:
+            out += [_ptr(None), _i(0), _ll(0)]
+            continue
+        _need(t, "partials", torch.float32)
+        if t.dim() != 3 or tuple(t.shape[1:]) != tuple(x.shape):
+            raise KernelError(f"{what}: partial sums {tuple(t.shape)} do not fit {tuple(x.shape)}")
+        out += [_ptr(t), _i(t.shape[0]), _ll(t.stride(0))]
+    return out
+
+
 def dyt(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, alpha: float, out: torch.Tensor,
         out_f32: Optional[torch.Tensor] = None, row_index: Optional[torch.Tensor] = None,
         partials: Optional[torch.Tensor] = None, out_split: Optional[torch.Tensor] = None) -> None:
@@ -217,8 +249,8 @@ def dyt_add(hs: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, bias: torch
 def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
          accumulate: bool = False, w_up: Optional[torch.Tensor] = None, group_offsets: Optional[torch.Tensor] = None,
          a_row_index: Optional[torch.Tensor] = None, rows: Optional[int] = None, act_limit: float = 0.0,
-         act_alpha: float = 1.0) -> None:
-    """out[M, N] (+)= a[M, K] . w[N, K]^T (+ bias) on the float32 FMA pipe.
+         act_alpha: float = 1.0, out_scale: float = 1.0) -> None:
+    """out[M, N] (+)= out_scale (a[M, K] . w[N, K]^T (+ bias)) on the float32 FMA pipe.
 
     ``w_up`` selects the gated form: silu(a.w^T) * (a.w_up^T), or with ``act_limit`` > 0 the capped one,
     g = min(a.w^T, limit), u = clamp(a.w_up^T, +-limit), g * sigmoid(act_alpha g) * (u + 1).  With ``group_offsets``
@@ -250,7 +282,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[tor
     st = library("gemm_simt").cj_gemm_simt(
         _ptr(a), _ll(a.stride(0)), _i(_code(a)), _ptr(w), _ptr(w_up), _ll(K), _i(_code(w)), _ptr(bias),
         _ptr(out), _ll(out.stride(0)), _i(_code(out)), _i(M), _i(N), _i(K), _i(1 if accumulate else 0),
-        _ptr(group_offsets), _i(G), _ll(N * K), _ptr(a_row_index), _f(act_limit), _f(act_alpha), _stream())
+        _ptr(group_offsets), _i(G), _ll(N * K), _ptr(a_row_index), _f(act_limit), _f(act_alpha), _f(out_scale), _stream())
     _check(st, "gemm")
 
 
@@ -279,14 +311,17 @@ def head_prepare(x: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: tor
                  table: Optional[torch.Tensor], page_tokens: int, n_heads: int, n_kv: int, head_dim: int, value_dim: int,
                  rotary_dim: int, inv_freq: Optional[torch.Tensor], magnitude: float, q_norm: Optional[torch.Tensor],
                  k_norm: Optional[torch.Tensor], eps: float, write_kv: bool, norm_whole: bool = False,
-                 q_temp_coef: float = 0.0, q_temp_every: int = 1) -> None:
+                 q_temp_coef: float = 0.0, q_temp_every: int = 1, unit_qk: bool = False, unit_v: bool = False,
+                 pairs: bool = False) -> None:
     """Queries, keys and values of a step's rows (x float32 [T, ld], columns from q_off, k_off, v_off) made ready
     for attention: an RMS norm over each head of q and k (when ``q_norm`` / ``k_norm``, float32 [head_dim], are
     given), the rotation of their first ``rotary_dim`` entries (entry i with i + rotary_dim / 2; cos and sin times
     ``magnitude``), q to ``q_out``, k and v into the cache pages of the row's request.  ``v_off`` < 0: the
     values are the keys as projected, before norm and rotation.  ``norm_whole``: one statistic over all heads of q
     (of k) at once, and weights of ``n_heads * head_dim`` (``n_kv * head_dim``) entries.  ``q_temp_coef`` != 0: the
-    queries are multiplied by ``1 + q_temp_coef * ln(floor((p + 1) / q_temp_every) + 1)`` at position p."""
+    queries are multiplied by ``1 + q_temp_coef * ln(floor((p + 1) / q_temp_every) + 1)`` at position p.  ``unit_qk``: every
+    head of q and k is divided by its root mean square (no weight; before or after the rotation is the same); ``unit_v``: every
+    head's value by its own, before it is written; ``pairs``: entries 2i and 2i + 1 rotate together, angle i."""
     _need(x, "x", torch.float32), _need(q_out, "q_out"), _need(positions, "positions", torch.int32)
     cache_dtype = _code(q_out)
     if write_kv:
@@ -303,7 +338,8 @@ def head_prepare(x: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: tor
         _ptr(x), _i(x.stride(0)), _i(q_off), _i(k_off), _i(v_off), _ptr(q_out), _i(_code(q_out)), _ptr(k_plane), _ptr(v_plane),
         _i(cache_dtype), _ptr(positions), _ptr(row_req), _ptr(table), _i(table.stride(0) if table is not None else 0),
         _i(page_tokens), _i(x.shape[0]), _i(n_heads), _i(n_kv), _i(head_dim), _i(value_dim), _i(rotary_dim), _ptr(inv_freq),
-        _f(magnitude), _ptr(q_norm), _ptr(k_norm), _f(eps), _i(1 if write_kv else 0), _i(1 if norm_whole else 0),
+        _f(magnitude), _ptr(q_norm), _ptr(k_norm), _f(eps), _i(1 if write_kv else 0),
+        _i((1 if norm_whole else 0) | (2 if unit_qk else 0) | (4 if unit_v else 0) | (8 if pairs else 0)),
         _f(q_temp_coef), _i(q_temp_every), _stream())
     _check(st, "head_prepare")
 
@@ -316,13 +352,18 @@ def _gate(head_gate: Optional[torch.Tensor], gate_offset: int):
     return ctypes.c_void_p(head_gate.data_ptr() + 4 * gate_offset), head_gate.stride(0)
 
 
+NO_SINK = float("-inf")      # no key without a value joins the softmax
+
+
 def paged_attention(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tensor,
                     positions: torch.Tensor, row_req: torch.Tensor, table: torch.Tensor, page_tokens: int,
                     n_heads: int, n_kv: int, head_dim: int, window: int, scale: float, value_dim: int = 0,
-                    softcap: float = 0.0, head_gate: Optional[torch.Tensor] = None, gate_offset: int = 0) -> None:
+                    softcap: float = 0.0, head_gate: Optional[torch.Tensor] = None, gate_offset: int = 0,
+                    sink: float = NO_SINK) -> None:
     """Attention of every row over its request's cached keys [from, position].  ``value_dim``: the values'
     size when it is not the keys'; ``softcap`` > 0: s <- cap tanh(s / cap); ``head_gate`` (float32 [T, ld]):
-    head h of row t is multiplied by sigmoid(head_gate[t, gate_offset + h])."""
+    head h of row t is multiplied by sigmoid(head_gate[t, gate_offset + h]).  ``sink``: a constant score of one more key that
+    has no value (exp(sink) in the softmax's divisor alone, neither scaled nor capped; 0 adds one); NO_SINK: none."""
     _need(q, "q"), _need(out, "out"), _need(k_plane, "k_plane"), _need(v_plane, "v_plane")
     _need(positions, "positions", torch.int32), _need(row_req, "row_req", torch.int32), _need(table, "table", torch.int32)
     T = q.shape[0]
@@ -332,7 +373,7 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor, v
     st = library("attention_paged").cj_paged_attention(
         _ptr(q), _ptr(out), _i(_code(q)), _ptr(k_plane), _ptr(v_plane), _i(_code(k_plane)), _ptr(positions),
         _ptr(row_req), _ptr(table), _i(table.stride(0)), _i(page_tokens), _i(T), _i(n_heads), _i(n_kv), _i(head_dim),
-        _i(value_dim or head_dim), _i(window), _f(scale), _f(softcap), gate_ptr, _i(gate_ld), _stream())
+        _i(value_dim or head_dim), _i(window), _f(scale), _f(softcap), gate_ptr, _i(gate_ld), _f(sink), _stream())
     _check(st, "paged_attention")
 
 
@@ -639,13 +680,11 @@ def add_rows(hs: torch.Tensor, other: Optional[torch.Tensor], vec: Optional[torc
     _check(library("stream_ops").cj_add_rows(_ptr(hs), _ptr(other), _ptr(vec), _i(T), _i(H), _stream()), "add_rows")
 
 
-def add_partials(hs: torch.Tensor, parts: torch.Tensor) -> None:
-    """hs += parts[0] + parts[1] + ... in that order; hs float32 [T, H], parts float32 [S, T, H] (the partial sums a
-    product cut along K leaves behind, when no norm follows that could add them while it reads the row)."""
-    _need(hs, "hs", torch.float32), _need(parts, "parts", torch.float32)
-    if parts.dim() != 3 or tuple(parts.shape[1:]) != tuple(hs.shape):
-        raise KernelError(f"add_partials: parts {tuple(parts.shape)} do not fit hs {tuple(hs.shape)}")
-    st = library("stream_ops").cj_add_partials(_ptr(hs), _ptr(parts), _i(parts.shape[0]), _ll(parts.stride(0)), _ll(hs.numel()), _stream())
+def add_partials(hs: torch.Tensor, parts: torch.Tensor, more: Optional[torch.Tensor] = None) -> None:
+    """hs += parts[0] + parts[1] + ... (+ more[0] + ...) in that order; hs float32 [T, H], parts and more float32 [S, T, H]
+    (the partial sums products cut along K leave behind, when no norm follows that could add them while it reads the row)."""
+    _need(hs, "hs", torch.float32)
+    st = library("stream_ops").cj_add_partials(_ptr(hs), *_two_partials(hs, (parts, more), "add_partials"), _ll(hs.numel()), _stream())
     _check(st, "add_partials")
 
 
@@ -798,6 +837,22 @@ def state_scan(mode: int, x: torch.Tensor, off_a: int, off_b: int, off_v: int, r
         _ptr(A_log), _ptr(dt_bias), _ptr(skip), ctypes.c_void_p(state.data_ptr() + 4 * state_offset), _ll(state.stride(0)),
         _ll(state[0].numel() - state_offset), _ptr(req_start), _ptr(req_slot), _ptr(out), _i(requests), _i(heads), _i(groups), _i(rows), _i(cols), _f(q_scale), _f(c0), _f(c1), _stream())
     _check(st, "state_scan")
+
+
+def gated_scan(x: torch.Tensor, off_z: int, off_x: int, off_g: int, width: int, state: torch.Tensor, state_offset: int,
+               req_start: torch.Tensor, req_slot: torch.Tensor, requests: int, out: torch.Tensor, single: bool = False) -> None:
+    """A gated recurrence channel by channel (minGRU) over every request's rows of the step: with zp, u, g the columns
+    off_z + k, off_x + k, off_g + k of x (float32 [T, ld], biases included), z = sigmoid(zp), c = u + 1/2 where u >= 0 and
+    sigmoid(u) where u < 0: ``S_t = (1 - z) S_(t-1) + z c`` (float32, ``width`` entries of ``state[slot]`` from
+    ``state_offset`` on), ``out[t] = S_t silu(g)``.  ``single``: every request of the step brings one token."""
+    _need(x, "x", torch.float32), _need(state, "state", torch.float32), _need(out, "out")
+    _need(req_start, "req_start", torch.int32), _need(req_slot, "req_slot", torch.int32)
+    if tuple(out.shape) != (x.shape[0], width) or max(off_z, off_x, off_g) + width > x.shape[1] or state[0].numel() < state_offset + width:
+        raise KernelError("gated_scan: sizes do not agree")
+    st = library("recurrent").cj_gated_scan(_ptr(x), _i(x.stride(0)), _i(off_z), _i(off_x), _i(off_g), _i(width),
+                                            ctypes.c_void_p(state.data_ptr() + 4 * state_offset), _ll(state.stride(0)), _ptr(req_start),
+                                            _ptr(req_slot), _i(requests), _i(1 if single else 0), _ptr(out), _i(_code(out)), _stream())
+    _check(st, "gated_scan")
 
 
 def gated_group_norm(y: torch.Tensor, part_len: int, z: torch.Tensor, z_offset: int, weight: torch.Tensor, eps: float,
@@ -1047,8 +1102,8 @@ EPI_STORE_F32, EPI_ACC_F32, EPI_SWIGLU_BF16, EPI_STORE_BF16, EPI_RELU2_BF16 = 0,
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, swap: bool, n_mma: int,
             bias: Optional[torch.Tensor] = None, w_up: Optional[torch.Tensor] = None,
             group_offsets: Optional[torch.Tensor] = None, tokens: Optional[int] = None, k_splits: int = 1,
-            offsets_settled: bool = False, act_limit: float = 0.0, act_alpha: float = 1.0) -> None:
-    """Tensor-core product out[token, feature] (+)= x[token, :] . w[feature, :] (+ bias) in
+            offsets_settled: bool = False, act_limit: float = 0.0, act_alpha: float = 1.0, out_scale: float = 1.0) -> None:
+    """Tensor-core product out[token, feature] (+)= out_scale (x[token, :] . w[feature, :] (+ bias)) in
     bfloat16 with float32 accumulation (tcgen05, TMA).
 
     ``swap`` False: tiles of 128 tokens x ``n_mma`` (128 or 256) features; True: tiles of 128
@@ -1058,7 +1113,10 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, 
     only): ``out`` is [k_splits, tokens, features] of partial sums.  ``offsets_settled``: the
     kernel that wrote ``group_offsets`` is not the one launched just before this product but an
     earlier one; the product then reads them before it waits for the kernel before it.
+    ``out_scale``: the float32 epilogues only.
     """
+    if out_scale != 1.0 and epilogue not in (EPI_STORE_F32, EPI_ACC_F32):
+        raise KernelError("gemm_tc: out_scale is part of the float32 epilogues")
     _need(x, "x", torch.bfloat16), _need(w, "w", torch.bfloat16), _need(out, "out")
     features, K = w.shape[-2], w.shape[-1]
     T = tokens if tokens is not None else x.shape[0]
@@ -1080,17 +1138,19 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, 
     st = library("gemm_tc").cj_gemm_tc(
         _ptr(x), _ll(x.stride(0)), _ptr(w), _ptr(w_up), _ptr(bias), _ptr(out), _ll(ldo), _i(T), _i(features), _i(K),
         _i(epilogue), _i(1 if swap else 0), _i(n_mma), _ptr(group_offsets), _i(G), _i(k_splits), _ll(split_stride),
-        _i(1 if offsets_settled and group_offsets is not None else 0), _f(act_limit), _f(act_alpha), _stream())
+        _i(1 if offsets_settled and group_offsets is not None else 0), _f(act_limit), _f(act_alpha), _f(out_scale), _stream())
     _check(st, "gemm_tc")
 
 
 def gemm_tc2(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, n_tok: int,
              bias: Optional[torch.Tensor] = None, w_up: Optional[torch.Tensor] = None,
              group_offsets: Optional[torch.Tensor] = None, tokens: Optional[int] = None, act_limit: float = 0.0,
-             act_alpha: float = 1.0) -> None:
+             act_alpha: float = 1.0, out_scale: float = 1.0) -> None:
     """The same product as ``gemm_tc`` on pairs of SMs (tcgen05 cta_group::2): tiles of 256
     features x ``n_tok`` (128 or 256) tokens, each SM of a pair loading its own 128 weight rows
     and half of the token rows.  For steps with many rows."""
+    if out_scale != 1.0 and epilogue not in (EPI_STORE_F32, EPI_ACC_F32):
+        raise KernelError("gemm_tc2: out_scale is part of the float32 epilogues")
     _need(x, "x", torch.bfloat16), _need(w, "w", torch.bfloat16), _need(out, "out")
     features, K = w.shape[-2], w.shape[-1]
     T = tokens if tokens is not None else x.shape[0]
@@ -1109,7 +1169,7 @@ def gemm_tc2(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int,
         G = w.shape[0]
     st = library("gemm_tc2").cj_gemm_tc2(
         _ptr(x), _ll(x.stride(0)), _ptr(w), _ptr(w_up), _ptr(bias), _ptr(out), _ll(out.stride(-2)), _i(T), _i(features), _i(K),
-        _i(epilogue), _i(n_tok), _ptr(group_offsets), _i(G), _f(act_limit), _f(act_alpha), _stream())
+        _i(epilogue), _i(n_tok), _ptr(group_offsets), _i(G), _f(act_limit), _f(act_alpha), _f(out_scale), _stream())
     _check(st, "gemm_tc2")
 
 
@@ -1147,12 +1207,12 @@ def decode_attention(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor, 
                      n_heads: int, n_kv: int, head_dim: int, window: int, scale: float, max_context: int,
                      scratch: "DecodeScratch", chunk: int = 0, tensor_cores: Optional[bool] = None,
                      merge_later: Optional[bool] = None, softcap: float = 0.0, head_gate: Optional[torch.Tensor] = None,
-                     gate_offset: int = 0) -> None:
+                     gate_offset: int = 0, sink: float = NO_SINK) -> None:
     """Split-KV attention of few bfloat16 query rows over their cached keys (head_dim 64 or 128).
     ``tensor_cores``: scores and weighted values of a chunk by mma.sync (the default) or on the
     FMA pipe (``chunk`` 64 or 128 applies to that form only).  ``merge_later``: the chunks of a
     row are merged by a kernel of its own instead of the row's last block (the default for steps
-    with many rows; same results to the bit).  ``softcap`` and ``head_gate`` as in ``paged_attention``
+    with many rows; same results to the bit).  ``softcap``, ``head_gate`` and ``sink`` as in ``paged_attention``
     (tensor-core form only)."""
     for n, t in (("q", q), ("out", out), ("k_plane", k_plane), ("v_plane", v_plane)):
         _need(t, n, torch.bfloat16)
@@ -1161,7 +1221,7 @@ def decode_attention(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor, 
     span = min(window, max_context) if window > 0 else max_context
     gate_ptr, gate_ld = _gate(head_gate, gate_offset)
     if tensor_cores is None:
-        tensor_cores = (DECODE_TENSOR_CORES and chunk == 0) or softcap > 0.0 or head_gate is not None
+        tensor_cores = (DECODE_TENSOR_CORES and chunk == 0) or softcap > 0.0 or head_gate is not None or sink != NO_SINK
     if tensor_cores:
         splits = max(1, -(-span // 128))
         scratch.ensure(T, n_heads, n_kv, head_dim, splits, q.device)
@@ -1171,14 +1231,14 @@ def decode_attention(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor, 
             _ptr(q), _ptr(out), _ptr(k_plane), _ptr(v_plane), _ptr(positions), _ptr(row_req), _ptr(table),
             _i(table.stride(0)), _i(page_tokens), _i(T), _i(n_heads), _i(n_kv), _i(head_dim), _i(window), _f(scale),
             _i(max_context), _ptr(scratch.acc), _ptr(scratch.ml), _ptr(scratch.counters), _i(scratch.splits),
-            _i(1 if merge_later else 0), _f(softcap), gate_ptr, _i(gate_ld), _stream())
+            _i(1 if merge_later else 0), _f(softcap), gate_ptr, _i(gate_ld), _f(sink), _stream())
         _check(st, "decode_attention")
         if merge_later and splits > 1:
             global launches
             launches += 1                  # the merge kernel
         return
-    if softcap > 0.0 or head_gate is not None:
-        raise KernelError("decode_attention: capped scores and gated heads are built into the tensor-core form only")
+    if softcap > 0.0 or head_gate is not None or sink != NO_SINK:
+        raise KernelError("decode_attention: capped scores, gated heads and a sink are built into the tensor-core form only")
     chunk = chunk or decode_chunk(span)
     splits = max(1, -(-span // chunk))
     scratch.ensure(T, n_heads, n_kv, head_dim, splits, q.device)
@@ -1210,10 +1270,11 @@ class DecodeScratch:
 def prefill_attention(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tensor,
                       req_start: torch.Tensor, req_prior: torch.Tensor, table: torch.Tensor, page_tokens: int,
                       n_heads: int, n_kv: int, head_dim: int, window: int, scale: float, block_rows: int = 0,
-                      softcap: float = 0.0, head_gate: Optional[torch.Tensor] = None, gate_offset: int = 0) -> None:
+                      softcap: float = 0.0, head_gate: Optional[torch.Tensor] = None, gate_offset: int = 0,
+                      sink: float = NO_SINK) -> None:
     """Tensor-core attention of a step's rows (request r owns rows req_start[r]..req_start[r+1]
     at positions req_prior[r] + i) over the paged cache; bfloat16, head_dim 32, 64, 96 or 128.
-    ``softcap`` and ``head_gate`` as in ``paged_attention``."""
+    ``softcap``, ``head_gate`` and ``sink`` as in ``paged_attention``."""
     for n, t in (("q", q), ("out", out), ("k_plane", k_plane), ("v_plane", v_plane)):
         _need(t, n, torch.bfloat16)
     _need(req_start, "req_start", torch.int32), _need(req_prior, "req_prior", torch.int32), _need(table, "table", torch.int32)
@@ -1221,18 +1282,21 @@ def prefill_attention(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor,
     st = library("attention_prefill").cj_prefill_attention(
         _ptr(q), _ptr(out), _ptr(k_plane), _ptr(v_plane), _ptr(req_start), _ptr(req_prior), _i(req_prior.numel()),
         _i(q.shape[0]), _ptr(table), _i(table.stride(0)), _i(page_tokens), _i(n_heads), _i(n_kv), _i(head_dim), _i(window),
-        _f(scale), _i(block_rows), _f(softcap), gate_ptr, _i(gate_ld), _stream())
+        _f(scale), _i(block_rows), _f(softcap), gate_ptr, _i(gate_ld), _f(sink), _stream())
     _check(st, "prefill_attention")
 
 
 def prefill_attention_tc(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tensor,
                          req_start: torch.Tensor, req_prior: torch.Tensor, table: torch.Tensor, page_tokens: int,
                          n_heads: int, n_kv: int, head_dim: int, window: int, scale: float, block_rows: int = 0,
-                         softcap: float = 0.0, head_gate: Optional[torch.Tensor] = None, gate_offset: int = 0) -> None:
+                         softcap: float = 0.0, head_gate: Optional[torch.Tensor] = None, gate_offset: int = 0,
+                         sink: float = NO_SINK, exact_cap: bool = False, score_bound: float = 0.0) -> None:
     """The same arguments and meaning as ``prefill_attention``, on the tcgen05 tensor cores: both products
     from shared memory into tensor memory.  ``block_rows``: 256 query rows a block (two tiles
     taking turns), 128, or 0 = by the size of the launch.  Head size 128 and pages of 16 tokens
-    only; anything else is refused."""
+    only; anything else is refused.  ``exact_cap``: a capped score's tangent in full float32 instead of the special-function
+    unit's (relative error 2^-11); ``score_bound`` > 0 promises that no |q . k| * scale is larger, which, when it is well
+    below the cap, allows the cheaper exact form."""
     for n, t in (("q", q), ("out", out), ("k_plane", k_plane), ("v_plane", v_plane)):
         _need(t, n, torch.bfloat16)
     _need(req_start, "req_start", torch.int32), _need(req_prior, "req_prior", torch.int32), _need(table, "table", torch.int32)
@@ -1242,7 +1306,8 @@ def prefill_attention_tc(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tens
     st = library("attention_prefill_tc").cj_prefill_attention_tc(
         _ptr(q), _ptr(out), _ptr(k_plane), _ptr(v_plane), _i(k_plane.shape[0]), _ptr(req_start), _ptr(req_prior),
         _i(req_prior.numel()), _i(q.shape[0]), _ptr(table), _i(table.stride(0)), _i(page_tokens), _i(n_heads), _i(n_kv),
-        _i(head_dim), _i(window), _f(scale), _i(block_rows), _f(softcap), gate_ptr, _i(gate_ld), _stream())
+        _i(head_dim), _i(window), _f(scale), _i(block_rows), _f(softcap), _i(1 if exact_cap else 0), _f(score_bound), gate_ptr,
+        _i(gate_ld), _f(sink), _stream())
     _check(st, "prefill_attention_tc")
 
 

@@ -18,6 +18,7 @@
 //   gla_scan           S_t = diag(alpha_t) S_(t-1) + k_t v_t^T ;  o_t = S_t^T q_t   (a decay per state row)
 //   mlstm_scan         m_t = max(f + m, i) ; S_t = e^(f + m - m_t) S + e^(i - m_t) k v^T ; n likewise with k alone ;
 //                      o = S^T q / (max(|n . q|, e^(-m_t)) + floor)
+//   gated_scan         S_t = (1 - z_t) S_(t-1) + z_t c_t per channel, out = S_t silu(g_t) (minGRU: gates of the current token only)
 //   rmsnorm_mix2       out (+)= c (a / rms(a) * wa + b / rms(b) * wb)
 //   relu2_rows         max(x, 0)^2 into the activation dtype
 //   softcap_rows       x <- cap tanh(x / cap), float32 in place (a head whose logits are capped)
@@ -531,6 +532,141 @@ __global__ void softcap_rows_kernel(float* __restrict__ x, float cap, long long 
         x[i] = cap * tanhf(x[i] / cap);
 }
 
+// ---------------------------------------------------------------------------------
+// A gated recurrence channel by channel whose gates read the current token alone (minGRU):
+//     z = sigmoid(zp) ; c = u + 1/2 for u >= 0, sigmoid(u) below ; S_t = (1 - z) S_(t-1) + z c ; out = S_t silu(g)
+// zp, u and g are columns off_z + k, off_x + k, off_g + k of the step's projected rows (biases included).  Because the
+// gates do not read the state, a stretch of tokens is one affine map S -> A S + B, and stretches compose: a block takes
+// CT neighbouring channels of one request, a thread PER consecutive tokens of a channel (their a = 1 - z and b = z c in
+// registers), the threads of a channel compose their stretches' maps by a warp's prefix scan, and every thread
+// then walks its tokens from the state its stretch begins with.  A request is cut into tiles from its own first row of the
+// step; requests of a few tokens (single decoded ones) are walked by a thread a channel instead, in the leading blocks.
+// Everything is float32 but the result.
+// ---------------------------------------------------------------------------------
+struct GatedScanArgs {
+    const float* x;
+    int ld, off_z, off_x, off_g, width;
+    float* state;
+    long long slot_stride;
+    const int* req_start;
+    const int* req_slot;
+};
+
+// a = 1 - z and b = z c; both sides of the sigmoid come from one exponential, so neither loses digits near 0 or 1
+__device__ __forceinline__ void gated_step(float zp, float u, float& a, float& b) {
+    const float e = expf(-fabsf(zp)), big = 1.0f / (1.0f + e), small = e * big;
+    const float z = zp >= 0.0f ? big : small;
+    a = zp >= 0.0f ? small : big;
+    b = z * (u >= 0.0f ? u + 0.5f : sigmoid_f(u));
+}
+
+constexpr int GS_PER = 16;           // tokens a thread takes in a tile; a request of at most this many is walked by a thread a channel
+constexpr int GS_THREADS = 512;
+
+template <typename TO, int CT>
+__global__ void __launch_bounds__(GS_THREADS) gated_scan_kernel(GatedScanArgs p, TO* __restrict__ out) {
+    cj::after_predecessor();
+    cj::release_successor();
+    constexpr int NSEG = GS_THREADS / CT;          // stretches of a tile, one a thread
+    constexpr int PL = NSEG / 32;                  // stretches a lane of the composing warp holds
+    static_assert(NSEG % 32 == 0 && CT <= GS_THREADS / 32, "a warp composes a channel's stretches");
+    const int req = blockIdx.y;
+    const int slot = p.req_slot[req];
+    const int first = p.req_start[req], n = p.req_start[req + 1] - first;
+    if (slot < 0 || n <= 0) return;
+    float* st = p.state + (size_t)slot * p.slot_stride;
+    if (n <= GS_PER || blockDim.x != GS_THREADS) {
+        // a thread a channel: the launch has at least enough blocks of its size for all channels
+        const int c = blockIdx.x * blockDim.x + threadIdx.x;
+        if (c >= p.width) return;
+        float S = st[c];
+        for (int t = 0; t < n; ++t) {
+            const float* row = p.x + (size_t)(first + t) * p.ld;
+            const float g = row[p.off_g + c];
+            float a, b;
+            gated_step(row[p.off_z + c], row[p.off_x + c], a, b);
+            S = fmaf(a, S, b);
+            out[(size_t)(first + t) * p.width + c] = from_f32<TO>(S * silu(g));
+        }
+        st[c] = S;
+        return;
+    }
+    __shared__ float As[NSEG][CT + 1], Bs[NSEG][CT + 1];        // a stretch's map, then (in Bs) the state it begins with
+    __shared__ float carry[CT];
+    const int ch = threadIdx.x % CT, seg = threadIdx.x / CT;
+    const int c = blockIdx.x * CT + ch;
+    const bool live = c < p.width;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    if (threadIdx.x < CT) carry[threadIdx.x] = live ? st[c] : 0.0f;
+    for (int tile0 = 0; tile0 < n; tile0 += NSEG * GS_PER) {
+        const int t0 = tile0 + seg * GS_PER;
+        const int mine = live ? max(0, min(GS_PER, n - t0)) : 0;
+        const float* row = p.x + (size_t)(first + t0) * p.ld + c;
+        float a[GS_PER], b[GS_PER];
+#pragma unroll
+        for (int i = 0; i < GS_PER; ++i) {
+            a[i] = i < mine ? row[(size_t)i * p.ld + p.off_z] : 0.0f;
+            b[i] = i < mine ? row[(size_t)i * p.ld + p.off_x] : 0.0f;
+        }
+        float A = 1.0f, B = 0.0f;
+#pragma unroll
+        for (int i = 0; i < GS_PER; ++i) {
+            float ai, bi;
+            gated_step(a[i], b[i], ai, bi);
+            a[i] = i < mine ? ai : 1.0f;                        // past the end: the map that changes nothing
+            b[i] = i < mine ? bi : 0.0f;
+            A *= a[i];
+            B = fmaf(a[i], B, b[i]);
+        }
+        As[seg][ch] = A;
+        Bs[seg][ch] = B;
+        __syncthreads();
+        if (warp < CT) {
+            // this warp composes channel `warp`: a lane its PL stretches in order, then a prefix scan over the lanes
+            float la[PL], lb[PL], ta = 1.0f, tb = 0.0f;
+#pragma unroll
+            for (int k = 0; k < PL; ++k) {
+                la[k] = As[lane * PL + k][warp];
+                lb[k] = Bs[lane * PL + k][warp];
+                tb = fmaf(la[k], tb, lb[k]);
+                ta *= la[k];
+            }
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const float pa = __shfl_up_sync(0xffffffffu, ta, o), pb = __shfl_up_sync(0xffffffffu, tb, o);
+                if (lane >= o) {
+                    tb = fmaf(ta, pb, tb);
+                    ta *= pa;
+                }
+            }
+            const float S0 = carry[warp];
+            float pa = __shfl_up_sync(0xffffffffu, ta, 1), pb = __shfl_up_sync(0xffffffffu, tb, 1);
+            float S = lane == 0 ? S0 : fmaf(pa, S0, pb);        // the state this lane's first stretch begins with
+#pragma unroll
+            for (int k = 0; k < PL; ++k) {
+                Bs[lane * PL + k][warp] = S;
+                S = fmaf(la[k], S, lb[k]);
+            }
+            __syncwarp();
+            if (lane == 31) carry[warp] = S;
+        }
+        __syncthreads();
+        float S = Bs[seg][ch];
+        const float* grow = row + p.off_g;
+        float g[GS_PER];
+#pragma unroll
+        for (int i = 0; i < GS_PER; ++i) g[i] = i < mine ? grow[(size_t)i * p.ld] : 0.0f;
+        TO* dst = out + (size_t)(first + t0) * p.width + c;
+#pragma unroll
+        for (int i = 0; i < GS_PER; ++i) {
+            S = fmaf(a[i], S, b[i]);
+            if (i < mine) dst[(size_t)i * p.width] = from_f32<TO>(S * silu(g[i]));
+        }
+        __syncthreads();                                        // Bs is read before the next tile writes it
+    }
+    if (threadIdx.x < CT && live) st[c] = carry[threadIdx.x];
+}
+
 }  // namespace
 
 // Lanes a column's rows are dealt to (4, 8, 16 or 32).  Every (column, token) costs a warp its staging,
@@ -700,6 +836,37 @@ CJ_EXPORT int cj_gated_group_norm(const float* y, int n, int part_len, const flo
     if (out_dtype == CJ_F32) cj::launch(gated_group_norm_kernel<float>, grid, dim3(warps * 32), 0, stream, y, n, part_len, z, ld_z, w, w_len, eps, gate_first, (float*)out);
     else if (out_dtype == CJ_BF16) cj::launch(gated_group_norm_kernel<__nv_bfloat16>, grid, dim3(warps * 32), 0, stream, y, n, part_len, z, ld_z, w, w_len, eps, gate_first, (__nv_bfloat16*)out);
     else return CJ_ERR_DTYPE;
+    return launch_status();
+}
+
+// x: float32 rows with stride ld holding the gate's, the candidate's and the output gate's pre-activations (biases included) at
+// columns off_z, off_x, off_g; state: per slot `width` float32 from the given pointer on, slot_stride apart.  single: every
+// request of the step brings one token.  out: [T, width] in out_dtype.
+CJ_EXPORT int cj_gated_scan(const float* x, int ld, int off_z, int off_x, int off_g, int width, float* state, long long slot_stride,
+                            const int* req_start, const int* req_slot, int requests, int single, void* out, int out_dtype,
+                            cudaStream_t stream) {
+    if (requests <= 0) return 0;
+    if (!x || !state || !req_start || !req_slot || !out) return CJ_ERR_ARG;
+    if (width <= 0 || ld < width || slot_stride < width || requests > 65535) return CJ_ERR_SIZE;
+    GatedScanArgs p{x, ld, off_z, off_x, off_g, width, state, slot_stride, req_start, req_slot};
+    // single tokens: small blocks, a thread a channel.  Otherwise tiles of 16 channels (64-byte pieces of a row), or of 8
+    // when tiles of 16 would leave SMs idle.
+    if (single) {
+        const dim3 grid((width + 127) / 128, requests);
+        if (out_dtype == CJ_F32) cj::launch(gated_scan_kernel<float, 16>, grid, dim3(128), 0, stream, p, (float*)out);
+        else if (out_dtype == CJ_BF16) cj::launch(gated_scan_kernel<__nv_bfloat16, 16>, grid, dim3(128), 0, stream, p, (__nv_bfloat16*)out);
+        else return CJ_ERR_DTYPE;
+        return launch_status();
+    }
+    const int ct = (long long)((width + 15) / 16) * requests >= 132 ? 16 : 8;
+    const dim3 grid((width + ct - 1) / ct, requests);
+#define LAUNCH(TO)                                                                                            \
+    if (ct == 16) cj::launch(gated_scan_kernel<TO, 16>, grid, dim3(GS_THREADS), 0, stream, p, (TO*)out);      \
+    else cj::launch(gated_scan_kernel<TO, 8>, grid, dim3(GS_THREADS), 0, stream, p, (TO*)out)
+    if (out_dtype == CJ_F32) { LAUNCH(float); }
+    else if (out_dtype == CJ_BF16) { LAUNCH(__nv_bfloat16); }
+    else return CJ_ERR_DTYPE;
+#undef LAUNCH
     return launch_status();
 }
 

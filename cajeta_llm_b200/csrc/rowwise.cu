@@ -373,6 +373,127 @@ CJ_EXPORT int cj_rmsnorm(float* x, const float* w, float eps, int rows, int H, v
 }
 
 // ---------------------------------------------------------------------------------
+// Two RMS norms of the same row: one statistic, two weights, two results in the activation dtype (a block whose mixer and
+// feed-forward each read a norm of their own of one stream).  Partial sums owed to the row by the layer before - of up to
+// two products cut along K - are added first, in order, and x keeps the sum.  A row of at most 8,192 entries in multiples of
+// four stays in registers between the sum and the scaling (VEC); any other row is read twice.
+// ---------------------------------------------------------------------------------
+template <typename TO, int V>
+__global__ void rmsnorm_pair_kernel(float* __restrict__ x, const float* __restrict__ wa, const float* __restrict__ wb, float eps, int H,
+                                    TO* __restrict__ out_a, TO* __restrict__ out_b, const float* __restrict__ parts, int n_parts,
+                                    long long part_stride, const float* __restrict__ more, int n_more, long long more_stride) {
+    cj::after_predecessor();
+    cj::release_successor();
+    __shared__ float partial[32];
+    const int r = blockIdx.x;
+    const size_t base = (size_t)r * H;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+    float ss = 0.0f;
+    float4 xv[V > 0 ? V : 1];
+    if (V > 0) {
+        const int n4 = H >> 2;
+#pragma unroll
+        for (int q = 0; q < V; ++q) {
+            const int u = threadIdx.x + q * blockDim.x;
+            xv[q] = u < n4 ? ((const float4*)(x + base))[u] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        }
+        if (n_parts + n_more > 0) {
+#pragma unroll
+            for (int q = 0; q < V; ++q) {
+                const int u = threadIdx.x + q * blockDim.x;
+                if (u < n4) {
+                    for (int s = 0; s < n_parts; ++s) {
+                        const float4 p4 = ((const float4*)(parts + s * part_stride + base))[u];
+                        xv[q].x += p4.x; xv[q].y += p4.y; xv[q].z += p4.z; xv[q].w += p4.w;
+                    }
+                    for (int s = 0; s < n_more; ++s) {
+                        const float4 p4 = ((const float4*)(more + s * more_stride + base))[u];
+                        xv[q].x += p4.x; xv[q].y += p4.y; xv[q].z += p4.z; xv[q].w += p4.w;
+                    }
+                    ((float4*)(x + base))[u] = xv[q];
+                }
+            }
+        }
+#pragma unroll
+        for (int q = 0; q < V; ++q) {
+            ss = fmaf(xv[q].x, xv[q].x, ss);
+            ss = fmaf(xv[q].y, xv[q].y, ss);
+            ss = fmaf(xv[q].z, xv[q].z, ss);
+            ss = fmaf(xv[q].w, xv[q].w, ss);
+        }
+    } else {
+        for (int i = threadIdx.x; i < H; i += blockDim.x) {
+            float v = x[base + i];
+            if (n_parts + n_more > 0) {
+                for (int s = 0; s < n_parts; ++s) v += parts[s * part_stride + base + i];
+                for (int s = 0; s < n_more; ++s) v += more[s * more_stride + base + i];
+                x[base + i] = v;
+            }
+            ss = fmaf(v, v, ss);
+        }
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) partial[warp] = ss;
+    __syncthreads();
+    float total = 0.0f;
+    for (int i = 0; i < nwarps; ++i) total += partial[i];           // every thread in the same order: no second barrier
+    const float scale = 1.0f / sqrtf(total / (float)H + eps);
+    if (V > 0) {
+        const int n4 = H >> 2;
+#pragma unroll
+        for (int q = 0; q < V; ++q) {
+            const int u = threadIdx.x + q * blockDim.x;
+            if (u < n4) {
+                const float4 a = ((const float4*)wa)[u], b = ((const float4*)wb)[u];
+                const float4 y = make_float4(xv[q].x * scale, xv[q].y * scale, xv[q].z * scale, xv[q].w * scale);
+                store4<TO>(out_a + base + 4 * u, make_float4(y.x * a.x, y.y * a.y, y.z * a.z, y.w * a.w));
+                store4<TO>(out_b + base + 4 * u, make_float4(y.x * b.x, y.y * b.y, y.z * b.z, y.w * b.w));
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < H; i += blockDim.x) {
+            const float y = x[base + i] * scale;
+            out_a[base + i] = from_f32<TO>(y * wa[i]);
+            out_b[base + i] = from_f32<TO>(y * wb[i]);
+        }
+    }
+}
+
+CJ_EXPORT int cj_rmsnorm_pair(float* x, const float* wa, const float* wb, float eps, int rows, int H, void* out_a, void* out_b,
+                              int out_dtype, const float* parts, int n_parts, long long part_stride, const float* more, int n_more,
+                              long long more_stride, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (!x || !wa || !wb || !out_a || !out_b || H <= 0) return CJ_ERR_ARG;
+    if (n_parts < 0 || n_more < 0 || (n_parts > 0 && !parts) || (n_more > 0 && !more)) return CJ_ERR_ARG;
+    const bool aligned = ((((uintptr_t)x) | ((uintptr_t)wa) | ((uintptr_t)wb) | ((uintptr_t)out_a) | ((uintptr_t)out_b) |
+                           ((uintptr_t)parts) | ((uintptr_t)more)) & 15) == 0;
+    const bool vec = H % 4 == 0 && H <= 8192 && aligned && part_stride % 4 == 0 && more_stride % 4 == 0;
+    // few rows: a 16-byte piece a thread, one round trip; many rows: four pieces a thread, so that more rows share an SM
+    const int n4 = H / 4;
+    int threads, v;
+    if (vec) {
+        const int want = rows >= NORM_QUARTER_MIN_ROWS ? (n4 + 3) / 4 : n4;
+        threads = want >= 512 ? 512 : (want <= 32 ? 32 : ((want + 31) / 32) * 32);
+        v = (n4 + threads - 1) / threads;
+    } else {
+        threads = H >= 512 ? 256 : 128;
+        v = 0;
+    }
+#define LAUNCH(TO, V) cj::launch(rmsnorm_pair_kernel<TO, V>, dim3(rows), dim3(threads), 0, stream, x, wa, wb, eps, H, (TO*)out_a, (TO*)out_b, parts, n_parts, part_stride, more, n_more, more_stride)
+#define PICK(TO)                    \
+    if (v == 0) LAUNCH(TO, 0);      \
+    else if (v == 1) LAUNCH(TO, 1); \
+    else if (v == 2) LAUNCH(TO, 2); \
+    else LAUNCH(TO, 4)
+    if (out_dtype == CJ_F32) { PICK(float); }
+    else if (out_dtype == CJ_BF16) { PICK(__nv_bfloat16); }
+    else return CJ_ERR_DTYPE;
+#undef PICK
+#undef LAUNCH
+    return launch_status();
+}
+
+// ---------------------------------------------------------------------------------
 // Dynamic Tanh, a norm that takes no statistic of the row: y = tanh(alpha x) w + b, with a scalar alpha,
 // a weight and a bias of the row's width, all float32.  Same outputs as the RMS norm above (the result in
 // the activation dtype, optionally its float32 copy or its three-term bfloat16 form; rows picked through

@@ -65,9 +65,11 @@ __global__ void add_rows_kernel(float* __restrict__ hs, const float* __restrict_
     }
 }
 
-// hs[i] += parts[0][i] + parts[1][i] + ... in that order (partial sums of a product cut along K)
+// hs[i] += parts[0][i] + parts[1][i] + ..., then more[0][i] + more[1][i] + ..., in that order (partial sums of one or two
+// products cut along K)
 template <bool VEC>
-__global__ void add_partials_kernel(float* __restrict__ hs, const float* __restrict__ parts, int n_parts, long long stride, long long n) {
+__global__ void add_partials_kernel(float* __restrict__ hs, const float* __restrict__ parts, int n_parts, long long stride,
+                                    const float* __restrict__ more, int n_more, long long more_stride, long long n) {
     cj::after_predecessor();
     cj::release_successor();
     constexpr int W = VEC ? 4 : 1;
@@ -78,10 +80,15 @@ __global__ void add_partials_kernel(float* __restrict__ hs, const float* __restr
                 const float4 p = *(const float4*)(parts + s * stride + i);
                 v.x += p.x; v.y += p.y; v.z += p.z; v.w += p.w;
             }
+            for (int s = 0; s < n_more; ++s) {
+                const float4 p = *(const float4*)(more + s * more_stride + i);
+                v.x += p.x; v.y += p.y; v.z += p.z; v.w += p.w;
+            }
             *(float4*)(hs + i) = v;
         } else {
             float v = hs[i];
             for (int s = 0; s < n_parts; ++s) v += parts[s * stride + i];
+            for (int s = 0; s < n_more; ++s) v += more[s * more_stride + i];
             hs[i] = v;
         }
     }
@@ -186,14 +193,15 @@ CJ_EXPORT int cj_add_rows(float* hs, const float* other, const float* vec, int T
     return launch_status();
 }
 
-CJ_EXPORT int cj_add_partials(float* hs, const float* parts, int n_parts, long long stride, long long n, cudaStream_t stream) {
+CJ_EXPORT int cj_add_partials(float* hs, const float* parts, int n_parts, long long stride, const float* more, int n_more,
+                              long long more_stride, long long n, cudaStream_t stream) {
     if (n <= 0 || n_parts <= 0) return 0;
-    if (!hs || !parts) return CJ_ERR_ARG;
-    const bool vec = (n | stride) % 4 == 0 && ((((uintptr_t)hs) | ((uintptr_t)parts)) & 15) == 0;
+    if (!hs || !parts || n_more < 0 || (n_more > 0 && !more)) return CJ_ERR_ARG;
+    const bool vec = (n | stride | more_stride) % 4 == 0 && ((((uintptr_t)hs) | ((uintptr_t)parts) | ((uintptr_t)more)) & 15) == 0;
     long long blocks = (n / (vec ? 4 : 1) + 255) / 256;
     if (blocks > 148 * 8) blocks = 148 * 8;
-    if (vec) cj::launch(add_partials_kernel<true>, dim3((unsigned)blocks), dim3(256), 0, stream, hs, parts, n_parts, stride, n);
-    else cj::launch(add_partials_kernel<false>, dim3((unsigned)blocks), dim3(256), 0, stream, hs, parts, n_parts, stride, n);
+    if (vec) cj::launch(add_partials_kernel<true>, dim3((unsigned)blocks), dim3(256), 0, stream, hs, parts, n_parts, stride, more, n_more, more_stride, n);
+    else cj::launch(add_partials_kernel<false>, dim3((unsigned)blocks), dim3(256), 0, stream, hs, parts, n_parts, stride, more, n_more, more_stride, n);
     return launch_status();
 }
 

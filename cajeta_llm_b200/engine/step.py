@@ -25,6 +25,7 @@ import numpy as np
 import torch
 
 from ..cache.manager import CacheManager
+from ..parts.block import settle
 from .model import Model
 
 
@@ -83,6 +84,7 @@ class StepContext:
     routing_pin: Optional[Dict[str, torch.Tensor]] = None     # a routed feed-forward's prefix -> int32 [rows, k]: experts given, not chosen
     routing_dump: Optional[Dict[str, tuple]] = None           # filled by routed feed-forwards: prefix -> (experts [rows, k], margins [rows])
     routing_seen: Dict[str, int] = field(default_factory=dict)  # how often each routed feed-forward has run in this step
+    owed: tuple = ()               # partial sums [S, rows, H] a block left to be added to the stream before anything else reads it
     embedding_output: Optional[torch.Tensor] = None           # the embedding's rows of the step, kept when a stream part of the plan reads them
 
 
@@ -281,6 +283,8 @@ class ModelRunner:
         if self.model.keeps_embedding_output:
             ctx.embedding_output = hs.clone()
         for i, e in enumerate(self.model.plan.schedule):
+            if self.model.before[i] is not None or not getattr(self.model.blocks[e.layer], "takes_owed", False):
+                settle(hs, ctx)
             if self.model.before[i] is not None:
                 self.model.before[i].forward(hs, ctx)
             k_plane, v_plane, group = self.cache.plane(i)
@@ -289,7 +293,9 @@ class ModelRunner:
                                 page_tokens=self.page_tokens, state=self.cache.state.get(i))
             self.model.blocks[e.layer].forward(hs, ctx, ectx)
         if ctx.want_rows.numel() == 0:
+            ctx.owed = ()
             return torch.empty((0, self.model.vocab), dtype=torch.float32, device=self.runtime.device)
+        settle(hs, ctx)
         return self.model.logits(hs, ctx.want_rows)
 
     def step_chained(self, slots: Sequence[int], device_tokens: torch.Tensor) -> Optional[torch.Tensor]:

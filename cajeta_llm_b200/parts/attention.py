@@ -23,7 +23,15 @@ weight of ``head_dim`` shared by the heads, before the rotation;
 is also the value;
 ``head_gate``: a tensor name; ``W_g`` of ``[num_heads, hidden]`` reads the mixer's input and head
 ``h``'s output is multiplied by ``sigmoid(W_g x)_h`` before the output projection;
+``qk_norm`` with an ``eps`` alone (no names): the heads of q and k are divided by their root mean square, without a weight;
+since a rotation keeps a head's length, that is the same before and after it;
+``value_norm``: ``{"eps": e}``, every head's value is divided by its root mean square before it is cached;
+``sink_score``: a number, the score of one more key that has no value: the softmax's divisor also holds ``exp`` of it
+(neither scaled nor capped; 0 adds one);
+``exact_cap``: capped scores in full float32 in every kernel (the tcgen05 prompt kernel otherwise takes the special-function
+unit's hyperbolic tangent);
 ``names``: the tensor names of ``q``, ``k``, ``v``, ``o`` under the part's prefix.
+A position part's ``pairs`` rotates neighbouring entries.
 A position part's ``magnitude`` (a stretched rotation's) multiplies cos and sin.
 
 Further optional parameters; a mixer that sets any of them runs ``head_prepare`` and the attention kernel that
@@ -40,6 +48,9 @@ softmax, ``s_h <- sum_g talk[h, g] s_g``;
 ``sink``: a tensor name, ``[heads]``: the softmax's divisor also holds ``exp(sink[h])``, a key without value
 that is neither scaled nor mixed.
 
+A block may set ``out_scale``: it multiplies the output projection as that is added to the stream (or handed back as
+partial sums).
+
 An entry that reads another entry's cache (``entry.writes_cache`` false) projects and
 rotates only q.
 """
@@ -52,7 +63,7 @@ import torch
 
 from ..csrc import kernels as K
 from .base import KvNeed, Part, make_part, register_part
-from .linear import project, project_split
+from .linear import project, project_split, splits_few_rows
 from .plan import ParamSpec
 
 
@@ -78,6 +89,12 @@ class PagedAttention(Part):
         self.head_temp = spec.get("head_temp") or None
         self.talk = spec.get("talk") or None
         self.sink = spec.get("sink") or None
+        self.unit_qk = bool(self.qk_norm and not self.qk_norm.get("q"))
+        self.value_norm = dict(spec.get("value_norm") or {}) or None
+        sink_score = spec.get("sink_score")
+        self.sink_score = float(sink_score) if sink_score is not None else K.NO_SINK
+        self.exact_cap = bool(spec.get("exact_cap", False))
+        self.out_scale = 1.0               # a block with a residual multiplier sets this
         names = dict(spec.get("names") or {})
         self.n_proj = {n: self.name(names.get(n, f"{n}_proj.weight")) for n in ("q", "k", "v", "o")}
         self.allow_pending = True          # a block that has no norm after the mixer sets this False
@@ -95,7 +112,8 @@ class PagedAttention(Part):
         self.v_dim = 0 if self.values_from_keys else self.kv_heads * self.value_dim
         self.o_dim = self.heads * self.value_dim
         self.general = bool(self.softcap > 0.0 or self.qk_norm or self.values_from_keys or self.head_gate
-                            or self.value_dim != self.head_dim or getattr(self.position, "magnitude", 1.0) != 1.0)
+                            or self.value_dim != self.head_dim or getattr(self.position, "magnitude", 1.0) != 1.0
+                            or getattr(self.position, "pairs", False) or self.value_norm or self.sink_score != K.NO_SINK)
         self.norm_whole = bool(self.qk_norm and self.qk_norm.get("whole"))
         self.mixed = bool(self.proj_conv or self.head_temp or self.talk or self.sink or self.norm_whole)
         self.general = self.general or self.mixed
@@ -103,6 +121,18 @@ class PagedAttention(Part):
             raise ValueError("the general attention path is built without biases")
         if self.mixed and (self.softcap > 0.0 or self.head_gate or self.values_from_keys):
             raise ValueError("mixed heads, a sink or a convolved projection are built without softcap, head_gate and values_from_keys")
+        if self.unit_qk and getattr(self.position, "magnitude", 1.0) != 1.0:
+            raise ValueError("heads normed without a weight go with a rotation that keeps their length")
+        if self.mixed and (self.unit_qk or self.value_norm or self.sink_score != K.NO_SINK):
+            raise ValueError("heads normed without a weight, normed values and a constant sink are not built into the mixed-heads path")
+        if self.values_from_keys and self.value_norm:
+            raise ValueError("values_from_keys takes the keys as projected: no value_norm")
+        eps = {float(n["eps"]) for n in (self.qk_norm, self.value_norm) if n}
+        if len(eps) > 1:
+            raise ValueError("qk_norm and value_norm share one eps")
+        self.head_eps = eps.pop() if eps else 0.0
+        # heads of length at most sqrt(head_dim) (a bfloat16 rounding more): no score is larger than this
+        self.score_bound = abs(self.scale) * self.head_dim * 1.02 if self.unit_qk else 0.0
         self.taps = int(self.proj_conv["taps"]) if self.proj_conv else 1
         if self.taps < 1:
             raise ValueError(f"proj_conv.taps must be >= 1, found {self.taps}")
@@ -133,7 +163,7 @@ class PagedAttention(Part):
         }
         if not self.values_from_keys:
             p[self.n_proj["v"]] = ParamSpec((self.v_dim, self.hidden))
-        if self.qk_norm:
+        if self.qk_norm and not self.unit_qk:
             p[self.name(self.qk_norm["q"])] = ParamSpec((self.q_dim if self.norm_whole else self.head_dim,), role="vector", init="ones")
             p[self.name(self.qk_norm["k"])] = ParamSpec((self.kv_dim if self.norm_whole else self.head_dim,), role="vector", init="ones")
         if self.proj_conv:
@@ -182,7 +212,7 @@ class PagedAttention(Part):
         if self.head_gate:
             rows.append(self.fetch(source, self.name(self.head_gate)))      # the gate's rows ride along: one product
         self.w_qkv = torch.cat(rows, dim=0).contiguous()
-        if self.qk_norm:
+        if self.qk_norm and not self.unit_qk:
             self.q_norm_w = self.fetch(source, self.name(self.qk_norm["q"]))
             self.k_norm_w = self.fetch(source, self.name(self.qk_norm["k"]))
         if self.proj_conv:
@@ -195,6 +225,9 @@ class PagedAttention(Part):
         self.w_o = self.fetch(source, self.n_proj["o"])
         if self.out_bias:
             self.b_o = self.fetch(source, self.name("o_proj.bias"))
+
+    def defers(self, rows: int) -> bool:
+        return self.allow_pending and not self.mixed and splits_few_rows(self.runtime, rows, self.w_o)
 
     # -- one step --------------------------------------------------------------------
     def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, entry) -> Optional[torch.Tensor]:
@@ -235,9 +268,9 @@ class PagedAttention(Part):
             K.paged_attention(q, out, entry.k_plane, entry.v_plane, ctx.positions, ctx.row_req, entry.block_table,
                               entry.page_tokens, self.heads, self.kv_heads, self.head_dim, self.window, self.scale)
         K.tag = "o"
-        parts = project_split(rt, out.view(T, self.q_dim), self.w_o, bias=self.b_o) if self.allow_pending else None
+        parts = project_split(rt, out.view(T, self.q_dim), self.w_o, bias=self.b_o, out_scale=self.out_scale) if self.allow_pending else None
         if parts is None:
-            project(rt, out.view(T, self.q_dim), self.w_o, residual, bias=self.b_o, accumulate=True)
+            project(rt, out.view(T, self.q_dim), self.w_o, residual, bias=self.b_o, accumulate=True, out_scale=self.out_scale)
         K.tag = None
         return parts                         # partial sums owed to the residual stream (the next norm adds them), or None
 
@@ -263,7 +296,8 @@ class PagedAttention(Part):
         K.head_prepare(qkv, 0, k_off, -1 if self.values_from_keys else v_off, q, entry.k_plane, entry.v_plane, ctx.positions,
                        ctx.row_req, entry.block_table, entry.page_tokens, self.heads, self.kv_heads, self.head_dim, self.value_dim,
                        pos.rotary_dim, pos.inv_freq, getattr(pos, "magnitude", 1.0), self.q_norm_w, self.k_norm_w,
-                       float(self.qk_norm["eps"]) if self.qk_norm else 0.0, write)
+                       self.head_eps, write, unit_qk=self.unit_qk, unit_v=self.value_norm is not None,
+                       pairs=getattr(pos, "pairs", False))
         out = torch.empty((T, self.heads, self.value_dim), dtype=rt.act_dtype, device=x.device)
         K.tag = "attention"
         gate = qkv if gate_cols else None
@@ -273,25 +307,26 @@ class PagedAttention(Part):
             K.decode_attention(q, out, entry.k_plane, entry.v_plane, ctx.positions, ctx.row_req, entry.block_table,
                                entry.page_tokens, self.heads, self.kv_heads, self.head_dim, self.window, self.scale,
                                ctx.max_context, getattr(ctx, "decode_scratch", None) or rt.decode_scratch,
-                               softcap=self.softcap, head_gate=gate, gate_offset=g_off)
+                               softcap=self.softcap, head_gate=gate, gate_offset=g_off, sink=self.sink_score)
         elif fast and self.head_dim == 128 and entry.page_tokens == 16 and hasattr(ctx, "req_start"):
             # portions of prompts (and whatever single tokens ride along): both products on tcgen05
             K.prefill_attention_tc(q, out, entry.k_plane, entry.v_plane, ctx.req_start, ctx.req_prior, entry.block_table,
                                    entry.page_tokens, self.heads, self.kv_heads, self.head_dim, self.window, self.scale,
-                                   softcap=self.softcap, head_gate=gate, gate_offset=g_off)
+                                   softcap=self.softcap, head_gate=gate, gate_offset=g_off, sink=self.sink_score,
+                                   exact_cap=self.exact_cap, score_bound=self.score_bound)
         elif fast and self.head_dim in (32, 64, 96, 128) and hasattr(ctx, "req_start"):
             # portions of prompts (and whatever single tokens ride along): query tiles on the tensor cores
             K.prefill_attention(q, out, entry.k_plane, entry.v_plane, ctx.req_start, ctx.req_prior, entry.block_table,
                                 entry.page_tokens, self.heads, self.kv_heads, self.head_dim, self.window, self.scale,
-                                softcap=self.softcap, head_gate=gate, gate_offset=g_off)
+                                softcap=self.softcap, head_gate=gate, gate_offset=g_off, sink=self.sink_score)
         else:
             K.paged_attention(q, out, entry.k_plane, entry.v_plane, ctx.positions, ctx.row_req, entry.block_table, entry.page_tokens,
                               self.heads, self.kv_heads, self.head_dim, self.window, self.scale, value_dim=self.value_dim,
-                              softcap=self.softcap, head_gate=gate, gate_offset=g_off)
+                              softcap=self.softcap, head_gate=gate, gate_offset=g_off, sink=self.sink_score)
         K.tag = "o"
-        parts = project_split(rt, out.view(T, self.o_dim), self.w_o) if self.allow_pending else None
+        parts = project_split(rt, out.view(T, self.o_dim), self.w_o, out_scale=self.out_scale) if self.allow_pending else None
         if parts is None:
-            project(rt, out.view(T, self.o_dim), self.w_o, residual, accumulate=True)
+            project(rt, out.view(T, self.o_dim), self.w_o, residual, accumulate=True, out_scale=self.out_scale)
         K.tag = None
         return parts
 
@@ -337,6 +372,6 @@ class PagedAttention(Part):
                                 self.scale, temp=self.temp_w, talk=self.talk_w, sink=self.sink_w,
                                 req_start=ctx.req_start if self._tiled() else None, n_requests=ctx.n_requests)
         K.tag = "o"
-        project(rt, out.view(T, self.o_dim), self.w_o, residual, accumulate=True)
+        project(rt, out.view(T, self.o_dim), self.w_o, residual, accumulate=True, out_scale=self.out_scale)
         K.tag = None
         return None

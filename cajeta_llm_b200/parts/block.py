@@ -16,7 +16,14 @@ kernel norms and adds.  Same parameters as ``prenorm``.
 ``parallel``: one norm, both sublayers read its output: ``h = norm(hs); hs += mixer(h) + feed_forward(h)``
 (each adds its result into the float32 stream).  A layer may have no feed-forward.  After the
 sublayers the layer's ``stream_after`` part, when it has one, runs on the stream.  Parameters:
-``mixer_norm_name``, ``mixer_name``, ``feed_forward_name``, ``stream_after_name``.
+``mixer_norm_name``, ``mixer_name``, ``feed_forward_name``, ``stream_after_name``; optional:
+``feed_forward_norm_name``: the feed-forward reads a norm of its own (``LayerSpec.feed_forward_norm``) of the same stream,
+``hs += mixer(norm_1(hs)) + feed_forward(norm_2(hs))``, both norms taken before either sublayer adds anything (two RMS norms of one
+eps are one kernel); ``residual_mult`` m: ``hs += m (mixer(.) + feed_forward(.))``, the factor applied to the float32 sums in the
+output products' epilogues (both sublayers must offer ``out_scale``); ``overlap`` (default true): in a step of few rows, where at
+least one of the two hands back partial sums instead of adding to the stream, the feed-forward runs on a side stream beside the
+mixer.  Partial sums of such a block are left owed to the stream (``ctx.owed``): the next block of this form adds them while its
+norms read the row, anything else that reads the stream has the step add them first.
 
 ``sandwich``: a norm before AND after each sublayer: ``hs += norm_1b(mixer(c(norm_1(hs))))``,
 ``hs += norm_2b(feed_forward(norm_2(hs)))``; a layer may have no feed-forward.  ``c`` is an optional causal
@@ -39,7 +46,26 @@ import torch
 
 from ..csrc import kernels as K
 from .base import Part, StateNeed, make_part, register_part
+from .norm import RMSNorm
 from .plan import LayerSpec, ParamSpec
+
+_side_streams: Dict[torch.device, "torch.cuda.Stream"] = {}
+
+
+def side_stream(device) -> "torch.cuda.Stream":
+    """One stream a device for sublayers that run beside the step's own stream, shared by all blocks."""
+    if device not in _side_streams:
+        _side_streams[device] = torch.cuda.Stream(device=device)
+    return _side_streams[device]
+
+
+def settle(hs: torch.Tensor, ctx) -> None:
+    """Adds the partial sums that a block left owed to the stream (``ctx.owed``), if any."""
+    if ctx.owed:
+        K.tag = "partial sums"
+        K.add_partials(hs, *ctx.owed)
+        K.tag = None
+        ctx.owed = ()
 
 
 @register_part("block", "prenorm")
@@ -158,14 +184,37 @@ class ParallelBlock(Part):
         self.after = None
         if layer.stream_after is not None:
             self.after = make_part("stream", layer.stream_after, self.name(spec.get("stream_after_name", "")), runtime)
+        self.feed_forward_norm = None
+        self.idle_norm = None              # the name of the second norm's weight in a layer without a feed-forward: nothing reads it
+        self.two_norms = bool(spec.get("feed_forward_norm_name"))
+        if self.two_norms and self.feed_forward is not None:
+            self.feed_forward_norm = make_part("norm", layer.feed_forward_norm, self.name(spec["feed_forward_norm_name"]), runtime)
+        elif self.two_norms:
+            self.idle_norm = self.name(spec["feed_forward_norm_name"])
+        self.takes_owed = self.two_norms
+        mult = float(spec.get("residual_mult", 1.0))
+        for p in (self.mixer, self.feed_forward):
+            if p is None:
+                continue
+            if mult != 1.0:
+                if not hasattr(p, "out_scale"):
+                    raise ValueError("residual_mult needs a mixer and a feed-forward that scale their results (out_scale)")
+                p.out_scale = mult
+            if self.two_norms and hasattr(p, "allow_pending"):
+                p.allow_pending = True
+        self.overlap = bool(spec.get("overlap", True))
+        self._side = None
 
     def parts(self):
-        return tuple(p for p in (self.mixer_norm, self.mixer, self.feed_forward, self.after) if p is not None)
+        return tuple(p for p in (self.mixer_norm, self.feed_forward_norm, self.mixer, self.feed_forward, self.after) if p is not None)
 
     def params(self) -> Dict[str, ParamSpec]:
         out: Dict[str, ParamSpec] = {}
         for p in self.parts():
             out.update(p.params())
+        if self.idle_norm is not None:
+            spec = next(iter(self.mixer_norm.params().values()))
+            out[self.idle_norm] = ParamSpec(spec.shape, role=spec.role, init=spec.init, optional=True)
         return out
 
     def libraries(self) -> set:
@@ -178,7 +227,63 @@ class ParallelBlock(Part):
         for p in self.parts():
             p.load(source)
 
+    def _norms(self, hs: torch.Tensor, owed):
+        """What the mixer reads, and what the feed-forward reads (in the activation dtype, and exactly when it asks for that),
+        of the same stream; partial sums owed to the stream are added first."""
+        a, b, ff = self.mixer_norm, self.feed_forward_norm, self.feed_forward
+        exact = getattr(ff, "needs_f32_input", False)
+        if (b is not None and not exact and isinstance(a, RMSNorm) and isinstance(b, RMSNorm) and a.eps == b.eps):
+            xa = torch.empty(hs.shape, dtype=self.runtime.act_dtype, device=hs.device)
+            xb = torch.empty_like(xa)
+            K.tag = "norms"
+            K.rmsnorm_pair(hs, a.weight, b.weight, a.eps, xa, xb, partials=owed)
+            K.tag = None
+            return xa, xb, None
+        if owed:
+            K.tag = "partial sums"
+            K.add_partials(hs, *owed)
+            K.tag = None
+        xa, _ = a.forward(hs)
+        if b is None:
+            return xa, None, None
+        wants_split = getattr(ff, "wants_split_input", None)
+        split = bool(wants_split and wants_split(hs.shape[0]))
+        xb, xb_exact = b.forward(hs, want_f32=exact and not split, want_split=split)
+        return xa, xb, xb_exact
+
+    def _forward_two_norms(self, hs: torch.Tensor, ctx, entry) -> None:
+        owed, ctx.owed = ctx.owed, ()
+        ff, rows = self.feed_forward, hs.shape[0]
+        x, xf, xf_exact = self._norms(hs, owed)
+        # both sublayers add to the same stream, so they may only run side by side when one of them does not: it hands
+        # back partial sums
+        beside = (ff is not None and self.overlap and hs.is_cuda
+                  and any(getattr(p, "defers", lambda n: False)(rows) for p in (self.mixer, ff)))
+        late = None
+        if beside:
+            # what the feed-forward allocates is its stream's; its result is read by the step's stream after the join, and the
+            # side stream's next work waits for the step's stream before it can reuse that memory.  A step that is being
+            # captured records the fork and the join as the graph's branches.
+            main = torch.cuda.current_stream()
+            if self._side is None:
+                self._side = side_stream(hs.device)
+            self._side.wait_stream(main)
+            with torch.cuda.stream(self._side):
+                late = ff.forward(xf, xf_exact, hs, ctx)
+            pending = self.mixer.forward(x, hs, ctx, entry)
+            main.wait_stream(self._side)
+        else:
+            pending = self.mixer.forward(x, hs, ctx, entry)
+            if ff is not None:
+                late = ff.forward(xf, xf_exact, hs, ctx)
+        ctx.owed = tuple(p for p in (pending, late) if p is not None)
+        if self.after is not None:
+            settle(hs, ctx)
+            self.after.forward(hs, ctx)
+
     def forward(self, hs: torch.Tensor, ctx, entry) -> None:
+        if self.two_norms:
+            return self._forward_two_norms(hs, ctx, entry)
         ff = self.feed_forward
         wants_split = getattr(ff, "wants_split_input", None)
         split = bool(wants_split and wants_split(hs.shape[0]))

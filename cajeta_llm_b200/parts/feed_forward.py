@@ -6,7 +6,9 @@
 ``gate``, ``up`` and ``down`` under the part's prefix).
 
 ``dense_relu2``: ``W_d max(W_u x, 0)^2``, a feed-forward without a gate whose activation is the square of the
-rectified sum.  Parameters: ``hidden_size``, ``intermediate_size``, ``names`` (``up``, ``down``).  On the tensor-core
+rectified sum.  Parameters: ``hidden_size``, ``intermediate_size``, ``names`` (``up``, ``down``), ``bias`` (optional: both products
+have a bias, under the weight's name with ``.b`` added).  A block may set ``out_scale`` (multiplies the result as it is added)
+and ``allow_pending`` (few rows: partial sums are handed back instead of added).  On the tensor-core
 path the square is the up-product's epilogue (the float32 sum squared, then rounded); elsewhere a kernel of its own.
 
 ``sparse_moe``: router logits ``l_e = Wr[e] . x`` in float32, softmax over all experts,
@@ -55,7 +57,7 @@ import torch
 
 from ..csrc import kernels as K
 from .base import Part, register_part
-from .linear import project, relu2_fused
+from .linear import project, project_split, relu2_fused, splits_few_rows
 from .plan import ParamSpec
 
 
@@ -112,10 +114,17 @@ class DenseRelu2(Part):
         names = dict(spec.get("names") or {})
         self.n_up = self.name(names.get("up", "up_proj.weight"))
         self.n_down = self.name(names.get("down", "down_proj.weight"))
-        self.w_up = self.w_down = None
+        self.bias = bool(spec.get("bias", False))
+        self.out_scale = 1.0
+        self.allow_pending = False         # a block that takes partial sums from its feed-forward sets this True
+        self.w_up = self.w_down = self.b_up = self.b_down = None
 
     def params(self) -> Dict[str, ParamSpec]:
-        return {self.n_up: ParamSpec((self.inter, self.hidden)), self.n_down: ParamSpec((self.hidden, self.inter))}
+        p = {self.n_up: ParamSpec((self.inter, self.hidden)), self.n_down: ParamSpec((self.hidden, self.inter))}
+        if self.bias:
+            p[self.n_up + ".b"] = ParamSpec((self.inter,), role="vector")
+            p[self.n_down + ".b"] = ParamSpec((self.hidden,), role="vector")
+        return p
 
     def libraries(self) -> set:
         libs = {"gemm_simt", "recurrent"}
@@ -126,22 +135,31 @@ class DenseRelu2(Part):
     def load(self, source) -> None:
         self.w_up = self.fetch(source, self.n_up)
         self.w_down = self.fetch(source, self.n_down)
+        if self.bias:
+            self.b_up = self.fetch(source, self.n_up + ".b")
+            self.b_down = self.fetch(source, self.n_down + ".b")
 
-    def forward(self, x: torch.Tensor, x_f32: Optional[torch.Tensor], residual: torch.Tensor, ctx) -> None:
+    def defers(self, rows: int) -> bool:
+        return self.allow_pending and splits_few_rows(self.runtime, rows, self.w_down)
+
+    def forward(self, x: torch.Tensor, x_f32: Optional[torch.Tensor], residual: torch.Tensor, ctx) -> Optional[torch.Tensor]:
         rt = self.runtime
         T = x.shape[0]
         act = torch.empty((T, self.inter), dtype=rt.act_dtype, device=x.device)
         K.tag = "dense up"
         if relu2_fused(rt, x, self.w_up, act.dtype):
-            project(rt, x, self.w_up, act, relu2=True)
+            project(rt, x, self.w_up, act, bias=self.b_up, relu2=True)
         else:
             pre = torch.empty((T, self.inter), dtype=torch.float32, device=x.device)
-            project(rt, x, self.w_up, pre)
+            project(rt, x, self.w_up, pre, bias=self.b_up)
             K.tag = "dense activation"
             K.relu2_rows(pre, act)
         K.tag = "dense down"
-        project(rt, act, self.w_down, residual, accumulate=True)
+        parts = project_split(rt, act, self.w_down, bias=self.b_down, out_scale=self.out_scale) if self.allow_pending else None
+        if parts is None:
+            project(rt, act, self.w_down, residual, bias=self.b_down, accumulate=True, out_scale=self.out_scale)
         K.tag = None
+        return parts
 
 
 @register_part("feed_forward", "sparse_moe")

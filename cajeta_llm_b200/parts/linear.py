@@ -79,7 +79,8 @@ def _pair_tile(runtime, rows: int, w: torch.Tensor, swiglu: bool, grouped: bool)
 def project(runtime, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Optional[torch.Tensor] = None,
             accumulate: bool = False, w_up: Optional[torch.Tensor] = None, group_offsets: Optional[torch.Tensor] = None,
             a_row_index: Optional[torch.Tensor] = None, max_group_rows: Optional[int] = None,
-            offsets_settled: bool = False, act_limit: float = 0.0, act_alpha: float = 1.0, relu2: bool = False) -> None:
+            offsets_settled: bool = False, act_limit: float = 0.0, act_alpha: float = 1.0, relu2: bool = False,
+            out_scale: float = 1.0) -> None:
     """``x``: [tokens, K]; ``w``: [features, K] or, with ``group_offsets``, [groups, features, K]
     where output row s belongs to the group whose range holds s and reads row
     ``a_row_index[s]`` of ``x`` (or row s).  ``w_up`` selects the SwiGLU form (``out`` in the
@@ -89,12 +90,15 @@ def project(runtime, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bia
     row gather does); the product may then read the offsets before it waits for that kernel.
     ``act_limit`` > 0 (with ``w_up``): the capped gate g = min(g, limit), u = clamp(u, +-limit),
     g * sigmoid(act_alpha g) * (u + 1) instead of silu(g) * u.  ``relu2`` (tensor-core path, ``out`` bfloat16, no ``w_up``):
-    ``out = max(x w^T, 0)^2``, the float32 sum squared before it is rounded; ask :func:`relu2_fused` first."""
+    ``out = max(x w^T (+ bias), 0)^2``, the float32 sum squared before it is rounded; ask :func:`relu2_fused` first.
+    ``out_scale`` multiplies the sum (bias included) before it is stored in or added to a float32 ``out``."""
+    if out_scale != 1.0 and (out.dtype != torch.float32 or w_up is not None):
+        raise ValueError("project: out_scale goes with a float32 result of one weight")
     if relu2 and (w_up is not None or out.dtype != torch.bfloat16 or not _tc_ok(runtime, x, w)):
         raise ValueError("project: relu2 is the tensor-core product's epilogue (bfloat16 out, no second weight)")
     if not _tc_ok(runtime, x, w):
         K.gemm(x, w, out, bias=bias, accumulate=accumulate, w_up=w_up, group_offsets=group_offsets, a_row_index=a_row_index,
-               act_limit=act_limit, act_alpha=act_alpha)
+               act_limit=act_limit, act_alpha=act_alpha, out_scale=out_scale)
         return
     rows = out.shape[0]
     if w_up is not None:
@@ -125,14 +129,14 @@ def project(runtime, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bia
     if pair_tile:
         # many rows: tiles of 256 features on pairs of SMs, each loading half of the token rows
         K.gemm_tc2(x, w, out, epi, pair_tile, bias=bias, w_up=w_up, group_offsets=group_offsets, tokens=rows,
-                    act_limit=act_limit, act_alpha=act_alpha)
+                    act_limit=act_limit, act_alpha=act_alpha, out_scale=out_scale)
     elif tile:
         K.gemm_tc(x, w, out, epi, True, tile, bias=bias, w_up=w_up, group_offsets=group_offsets, tokens=rows,
-                  offsets_settled=offsets_settled, act_limit=act_limit, act_alpha=act_alpha)
+                  offsets_settled=offsets_settled, act_limit=act_limit, act_alpha=act_alpha, out_scale=out_scale)
     else:
         n_mma = 256 if (w_up is None and w.shape[-2] >= 512) else 128
         K.gemm_tc(x, w, out, epi, False, n_mma, bias=bias, w_up=w_up, group_offsets=group_offsets, tokens=rows,
-                  offsets_settled=offsets_settled, act_limit=act_limit, act_alpha=act_alpha)
+                  offsets_settled=offsets_settled, act_limit=act_limit, act_alpha=act_alpha, out_scale=out_scale)
 
 
 def relu2_fused(runtime, x: torch.Tensor, w: torch.Tensor, out_dtype) -> bool:
@@ -140,25 +144,38 @@ def relu2_fused(runtime, x: torch.Tensor, w: torch.Tensor, out_dtype) -> bool:
     return out_dtype == torch.bfloat16 and _tc_ok(runtime, x, w)
 
 
-def project_split(runtime, x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
-    """For a few rows and a weight with few output features: the product cut along K into
-    enough pieces to occupy the machine.  Returns the partial sums [S, tokens, features]
-    (float32; the bias is in the first), to be added by the consumer in order - or None
-    when the shapes do not call for it (the caller then uses :func:`project`)."""
-    if not _tc_ok(runtime, x, w):
-        return None
-    rows = x.shape[0]
+def split_count(runtime, rows: int, w: torch.Tensor) -> int:
+    """Pieces along K that :func:`project_split` cuts a product of ``rows`` rows with ``w`` into; below 2: it does not."""
     tile = _token_tile(rows)
     if not tile:
-        return None
+        return 0
     features, Kd = w.shape[-2], w.shape[-1]
     feature_tiles = -(-features // 128) * -(-rows // tile)
     k_blocks = -(-Kd // 64)
     # as many pieces as it takes to give (nearly) every SM a block; 7/8 of them, so that a
     # product of 16 tiles is cut into 8 pieces of equal length rather than 9 ragged ones
-    splits = min(8, max(1, (runtime.sm_count * 7 // 8) // feature_tiles), max(1, k_blocks // 4))
+    return min(8, max(1, (runtime.sm_count * 7 // 8) // feature_tiles), max(1, k_blocks // 4))
+
+
+def splits_few_rows(runtime, rows: int, w: Optional[torch.Tensor]) -> bool:
+    """Whether a part whose last product is with ``w`` (its input dense activations of the engine's dtype) hands back partial
+    sums for a step of ``rows`` rows instead of adding its result itself."""
+    return (runtime.fast_kernels and w is not None and w.dtype == torch.bfloat16 and w.shape[-1] >= MIN_K and w.shape[-1] % 8 == 0
+            and w.shape[-2] >= MIN_FEATURES and split_count(runtime, rows, w) >= 2)
+
+
+def project_split(runtime, x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
+                  out_scale: float = 1.0) -> Optional[torch.Tensor]:
+    """For a few rows and a weight with few output features: the product cut along K into
+    enough pieces to occupy the machine.  Returns the partial sums [S, tokens, features]
+    (float32; the bias is in the first; ``out_scale`` in all), to be added by the consumer in order - or None
+    when the shapes do not call for it (the caller then uses :func:`project`)."""
+    if not _tc_ok(runtime, x, w):
+        return None
+    rows = x.shape[0]
+    splits = split_count(runtime, rows, w)
     if splits < 2:
         return None
-    parts = torch.empty((splits, rows, features), dtype=torch.float32, device=x.device)
-    K.gemm_tc(x, w, parts, K.EPI_STORE_F32, True, tile, bias=bias, k_splits=splits)
+    parts = torch.empty((splits, rows, w.shape[-2]), dtype=torch.float32, device=x.device)
+    K.gemm_tc(x, w, parts, K.EPI_STORE_F32, True, _token_tile(rows), bias=bias, k_splits=splits, out_scale=out_scale)
     return parts

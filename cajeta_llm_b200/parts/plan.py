@@ -55,6 +55,7 @@ class ParamSpec:
     role: str = "matrix"
     init: str = "normal"
     std: float = 0.02
+    optional: bool = False      # the file may hold it or not; nothing reads it (the norm of a sublayer that a layer does not have)
 
 
 @dataclass(frozen=True)

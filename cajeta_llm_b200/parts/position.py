@@ -18,6 +18,9 @@ out in float64 and rounded once.
 the wavelength ``l = 2 pi / f``, a frequency stays where ``l < original / high``, becomes ``f / factor`` where
 ``l > original / low``, and in between ``(1 - s) f / factor + s f`` with ``s = (original / l - low) / (high - low)``;
 the magnitude stays 1.  Worked out in float64 and rounded once.
+``pairs`` (optional, default false): entries 2i and 2i + 1 of a head rotate together with angle i, instead of entries i and
+i + rotary_dim / 2; a mixer reads it from the part.  ``float64_table`` (optional, default false): the unscaled table is worked out
+in float64 and rounded once.
 ``none``: no rotation.
 """
 from __future__ import annotations
@@ -43,6 +46,9 @@ class RotaryEncoding(Part):
         d = np.arange(half, dtype=np.float32)
         exponent = (np.float32(0.0) - np.float32(2.0) * d) / np.float32(self.rotary_dim)
         inv = np.power(np.float32(self.theta), exponent).astype(np.float32)
+        if spec.get("float64_table"):
+            inv = np.power(self.theta, -2.0 * np.arange(half, dtype=np.float64) / self.rotary_dim).astype(np.float32)
+        self.pairs = bool(spec.get("pairs", False))
         self.magnitude = 1.0
         scaling = spec.get("scaling")
         if scaling and scaling.get("kind") == "wavelength":
@@ -79,4 +85,5 @@ class NoPosition(Part):
         super().__init__(spec, prefix, runtime)
         self.rotary_dim = 0
         self.inv_freq = None
+        self.pairs = False
         self.magnitude = 1.0

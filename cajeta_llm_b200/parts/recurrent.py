@@ -59,6 +59,14 @@ entries), times ``sigmoid(W_g x)``, then ``W_o``.  Parameters: ``hidden_size``, 
 ``gate_cap``, ``floor`` (default 1e-6), ``eps``.  Tensors: ``q``, ``k``, ``v``, ``g``, ``i``, ``i.b``, ``f``,
 ``f.b``, ``norm``, ``o``.
 
+``mingru`` (minGRU, a gated recurrence whose gates read the current token alone).  Channel by channel over ``width``
+entries, ``z = sigmoid(W_z x + b_z)``, ``u = W_x x + b_x``, ``c = u + 1/2`` where ``u >= 0`` and ``sigmoid(u)`` below::
+
+    S_t = (1 - z_t) S_(t-1) + z_t c_t
+
+and the result is ``W_o (S_t * silu(W_g x))``.  The state is ``width`` float32 entries a request.  Gates, candidate and
+state are float32.  Parameters: ``hidden_size``, ``width``.  Tensors: ``z``, ``z.b``, ``x``, ``x.b``, ``g``, ``o``.
+
 A mixer inside another part (a block that keeps state of its own before the mixer's, a mixer that runs two
 side by side) finds its share of the request's state vector at ``entry.state_offset``.
 """
@@ -70,7 +78,7 @@ import torch
 
 from ..csrc import kernels as K
 from .base import Part, StateNeed, register_part
-from .linear import project
+from .linear import project, project_split, splits_few_rows
 from .plan import ParamSpec
 
 
@@ -358,3 +366,56 @@ class MatrixMemoryMixer(_StateMixer):
         project(rt, gated, self.w_o, residual, accumulate=True)
         K.tag = None
         return None
+
+
+@register_part("mixer", "mingru")
+class MinGRUMixer(_StateMixer):
+    def __init__(self, spec, prefix, runtime):
+        super().__init__(spec, prefix, runtime)
+        self.hidden = int(spec["hidden_size"])
+        self.width = int(spec["width"])
+        if self.width < 1:
+            raise ValueError(f"width must be >= 1, found {self.width}")
+        self.out_scale = 1.0               # a block with a residual multiplier sets this
+        self.allow_pending = False         # a block that takes partial sums from its mixer sets this True
+        self.w_in = self.b_in = self.w_o = None
+
+    def state_need(self) -> Optional[StateNeed]:
+        return StateNeed((self.width,), torch.float32)
+
+    def params(self) -> Dict[str, ParamSpec]:
+        return {
+            self.name("z"): ParamSpec((self.width, self.hidden)),
+            self.name("z.b"): ParamSpec((self.width,), role="vector", init="normal", std=1.0),
+            self.name("x"): ParamSpec((self.width, self.hidden)),
+            self.name("x.b"): ParamSpec((self.width,), role="vector", init="normal", std=1.0),
+            self.name("g"): ParamSpec((self.width, self.hidden)),
+            self.name("o"): ParamSpec((self.hidden, self.width)),
+        }
+
+    def load(self, source) -> None:
+        # one product: z | x | g, the two biases in its epilogue (the output gate has none)
+        self.w_in = torch.cat([self.fetch(source, self.name(n)) for n in ("z", "x", "g")], dim=0).contiguous()
+        bz, bx = self.fetch(source, self.name("z.b")), self.fetch(source, self.name("x.b"))
+        self.b_in = torch.cat([bz, bx, torch.zeros_like(bz)], dim=0).contiguous()
+        self.w_o = self.fetch(source, self.name("o"))
+
+    def defers(self, rows: int) -> bool:
+        return self.allow_pending and splits_few_rows(self.runtime, rows, self.w_o)
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, entry) -> Optional[torch.Tensor]:
+        rt = self.runtime
+        T, W = x.shape[0], self.width
+        proj = torch.empty((T, 3 * W), dtype=torch.float32, device=x.device)
+        K.tag = "mixer in"
+        project(rt, x, self.w_in, proj, bias=self.b_in)
+        gated = torch.empty((T, W), dtype=rt.act_dtype, device=x.device)
+        K.tag = "scan"
+        K.gated_scan(proj, 0, W, 2 * W, W, entry.state, getattr(entry, "state_offset", 0), ctx.req_start, ctx.req_slot,
+                     ctx.n_requests, gated, single=getattr(ctx, "all_single", False))
+        K.tag = "o"
+        parts = project_split(rt, gated, self.w_o, out_scale=self.out_scale) if self.allow_pending else None
+        if parts is None:
+            project(rt, gated, self.w_o, residual, accumulate=True, out_scale=self.out_scale)
+        K.tag = None
+        return parts

@@ -30,7 +30,7 @@ class WeightError(ValueError):
 
 
 def check_schema(schema: Mapping[str, ParamSpec], have: Mapping[str, Tuple[int, ...]], where: str) -> None:
-    missing = [n for n in schema if n not in have]
+    missing = [n for n in schema if n not in have and not schema[n].optional]
     unexpected = [n for n in have if n not in schema]
     wrong = [(n, tuple(schema[n].shape), tuple(have[n])) for n in schema
              if n in have and tuple(have[n]) != tuple(schema[n].shape)]
@@ -123,6 +123,6 @@ def write_model_folder(model_dir: str, config, schema: Mapping[str, ParamSpec], 
     with open(os.path.join(model_dir, "config.json"), "w", encoding="utf-8") as f:
         json.dump(config.to_json_dict(), f, indent=2)
     src = RandomWeights(seed, store_dtype=store_dtype, device="cpu")
-    tensors: Dict[str, torch.Tensor] = {name: src.get(name, spec) for name, spec in schema.items()}
+    tensors: Dict[str, torch.Tensor] = {name: src.get(name, spec) for name, spec in schema.items() if not spec.optional}
     write_safetensors(os.path.join(model_dir, "model.safetensors"), tensors,
                       metadata={"format": "pt", "seed": str(seed)})
