@@ -1,9 +1,11 @@
-"""Throughput of a Balalorn, a Saropel, a Govuvik or a Dimuvik model at layer sizes that resemble real models', beside the
+"""Throughput of a Balalorn, a Saropel, a Govuvik, a Dimuvik or a Rugezen model at layer sizes that resemble real models', beside the
 engine's Qwen2-MoE model at equal width, depth, experts and feed-forward sizes (Govuvik: beside Balalorn, the
 engine's other model with recurrent state, at equal width, depth and experts; Dimuvik: beside Balalorn, the engine's
-other model with attention over a latent and a borrowed cache, at equal width, depth, heads, latent and experts).
+other model with attention over a latent and a borrowed cache, at equal width, depth, heads, latent and experts; Rugezen:
+beside a Saropel of dense layers alone, the engine's other model of parallel blocks with capped attention and a looped
+stretch, at equal width, depth, heads and feed-forward, and beside Balalorn for its recurrent layers).
 
-``python bench.py --design balalorn|saropel|govuvik|dimuvik [--sizes small,medium,large]`` prints one JSON line per
+``python bench.py --design balalorn|saropel|govuvik|dimuvik|rugezen [--sizes small,medium,large]`` prints one JSON line per
 (size, model): prefill tokens a second (one prompt of 2,048 tokens), decode tokens a second
 (8 requests of 512 tokens each, steps replayed from CUDA graphs), and where the time of both
 steps goes by class of work (launches serialised, an event behind each), with the bytes or
@@ -101,6 +103,32 @@ def dimuvik_config(s):
             "layers": [kinds[i % 4](i) for i in range(s["layers"])]}
 
 
+RUGEZEN_RUNS = ("attention", "mingru", "mingru", "attention")      # three layers of weights; the middle one runs twice
+
+
+def rugezen_config(s):
+    """Three layers of weights, four layer runs: attention (H heads of 128 over H/4 key heads, half of each rotated) + dense,
+    minGRU of one and a half times the width + dense twice (a looped stretch), attention + dense."""
+    h, H = s["width"], s["heads"]
+    attn = {"type": "attention", "mlp": {"kind": "dense", "ff": s["ff"]},
+            "mixer": {"heads": H, "kv_heads": H // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0,
+                      "rot": {"base": 1000000.0, "dims": 64}}}
+    gru = {"type": "mingru", "mixer": {"width": 3 * h // 2}, "mlp": {"kind": "dense", "ff": s["ff"]}}
+    return {"architecture": "Rugezen", "width": h, "vocab": VOCAB, "norm": {"eps": 1e-6}, "residual_mult": 0.4,
+            "loop": {"start": 1, "stop": 2, "times": 2}, "layers": [attn, gru, attn]}
+
+
+def saropel_dense_config(s):
+    """The same shape of model from Saropel's parts: parallel blocks with dense feed-forwards and no side inputs, capped
+    attention, rotated and normed attention in a stretch that runs twice, capped attention; no windows, H/4 key heads."""
+    H = s["heads"]
+    base = {"heads": H, "kv_heads": H // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    capped = {"type": "attention", "mixer": dict(base, softcap=30.0), "mlp": {"kind": "dense", "ff": s["ff"]}}
+    rotated = {"type": "attention_2", "mixer": dict(base, rot={"base": 1000000.0, "dims": 64}), "mlp": {"kind": "dense", "ff": s["ff"]}}
+    return {"architecture": "Saropel", "width": s["width"], "vocab": VOCAB, "norm": {"eps": 1e-6},
+            "loop": {"start": 1, "stop": 2, "times": 2}, "layers": [capped, rotated, capped]}
+
+
 def qwen_config(s, shared=0):
     return {"architectures": ["Qwen2MoeForCausalLM"], "hidden_size": s["width"], "intermediate_size": s["ff"],
             "num_hidden_layers": s["layers"], "num_attention_heads": s["heads"], "num_key_value_heads": s["heads"], "head_dim": 128,
@@ -116,6 +144,23 @@ def needs(design, s, rows, ctx, prefill):
     if design == "qwen2_moe":
         kv = ctx * 2 * H * 128 * 2
         out["attention"] = (rows * kv * L if not prefill else 0, 4 * H * 128 * rows * (rows + 1) // 2 * L if prefill else 0)
+        return out
+    if design in ("rugezen", "saropel_dense"):
+        runs = RUGEZEN_RUNS if design == "rugezen" else ("attention",) * 4
+        n_attn, n_gru, G, W = runs.count("attention"), runs.count("mingru"), H // 4, 3 * s["width"] // 2
+        out["attention"] = (rows * ctx * 2 * G * 128 * 2 * n_attn if not prefill else 0,
+                            4 * H * 128 * rows * (rows + 1) // 2 * n_attn if prefill else 0)
+        # heads in float32, queries and cache entries out in bfloat16
+        out["heads + cache write"] = (rows * (H + 2 * G) * 128 * 6 * n_attn, 0)
+        # the stream once, two (one) normed copies out
+        out["norms" if design == "rugezen" else "rmsnorm"] = (rows * s["width"] * (8 if design == "rugezen" else 6) * len(runs), 0)
+        if n_gru:
+            reqs = 1 if prefill else rows
+            out["scan"] = ((rows * (3 * 4 + 2) * W + reqs * 2 * 4 * W) * n_gru, 0)
+        weights = {"dense up": 1, "dense gate/up": 2, "dense down": 1}
+        for k, n in weights.items():
+            w = n * s["width"] * s["ff"] * len(runs)
+            out[k] = (2 * w if not prefill else 0, 2 * rows * w if prefill else 0)
         return out
     if design == "saropel":
         by = fl = 0
@@ -181,6 +226,8 @@ def run(args, peaks) -> int:
             pair = (("govuvik", govuvik_config(s)), ("balalorn", balalorn_config(s)))
         elif args.design == "dimuvik":
             pair = (("dimuvik", dimuvik_config(s)), ("balalorn", balalorn_config(s)))
+        elif args.design == "rugezen":
+            pair = (("rugezen", rugezen_config(s)), ("saropel_dense", saropel_dense_config(s)), ("balalorn", balalorn_config(s)))
         else:
             pair = (("balalorn", balalorn_config(s)), ("qwen2_moe", qwen_config(s)))
         for design, cfg in pair:
@@ -229,6 +276,8 @@ def run(args, peaks) -> int:
                 for blk in r.model.blocks:
                     if hasattr(getattr(blk, "mixer", None), "overlap"):
                         blk.mixer.overlap = False
+                    if hasattr(blk, "overlap"):
+                        blk.overlap = False
                 spent = {}
                 for keep in (False, False, True):
                     held, entries = entries_of()

@@ -323,14 +323,19 @@ constexpr int TC_THREADS = 128;
 constexpr int TC_WARPS = TC_THREADS / 32;
 constexpr int TC_BLOCKS = 5;         // blocks an SM
 
-template <int HD>
+// HD: columns of a tile's rows, 64 or 128.  EXACT: keys and values have HD entries each; otherwise hd and vd (multiples of
+// eight, at most HD) are what they have, and the tiles' columns past them are filled with zeros, which add nothing to a score
+// and whose sums nobody reads.
+template <int HD, bool EXACT>
 __global__ void __launch_bounds__(TC_THREADS, TC_BLOCKS) decode_attention_tc_kernel(
     const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ kplane,
     const __nv_bfloat16* __restrict__ vplane, const int* __restrict__ positions, const int* __restrict__ row_req,
     const int* __restrict__ table, int table_stride, int page_tokens, int n_heads, int n_kv, int head_batches,
     int window, float scale, float* __restrict__ part_acc, float* __restrict__ part_ml, int* __restrict__ counters,
-    int max_splits, int merge_later, float softcap, const float* __restrict__ head_gate, int gate_ld, float sink) {
+    int max_splits, int merge_later, float softcap, const float* __restrict__ head_gate, int gate_ld, float sink,
+    int hd_given, int vd_given) {
     cj::release_successor();
+    const int hd = EXACT ? HD : hd_given, vd = EXACT ? HD : vd_given;
     constexpr int COLS = HD / 8;
     extern __shared__ __align__(128) unsigned char smem_raw[];
     __nv_bfloat16* kv = (__nv_bfloat16*)smem_raw;             // [128][HD] swizzled: the keys, then the values, then the warps' partial outputs
@@ -373,7 +378,8 @@ __global__ void __launch_bounds__(TC_THREADS, TC_BLOCKS) decode_attention_tc_ker
 #pragma unroll
     for (int j = 0; j < TC_CHUNK / ROWS_STEP; ++j) {
         const int r = r0 + j * ROWS_STEP;
-        cp_async16_zfill(kv + r * HD + ((c ^ (r & 7)) * 8), kplane + (size_t)bases[r] * HD + c * 8, r < count);
+        const bool there = r < count && (EXACT || c * 8 < hd);
+        cp_async16_zfill(kv + r * HD + ((c ^ (r & 7)) * 8), kplane + (there ? (size_t)bases[r] * hd + c * 8 : 0), there);
     }
     cp_async_commit();
     if (older_keys_only) cj::after_predecessor();
@@ -381,7 +387,7 @@ __global__ void __launch_bounds__(TC_THREADS, TC_BLOCKS) decode_attention_tc_ker
     if (r0 < TC_HEADS) {
         // the queries (the kernel before wrote them): q rows, zero below the heads taken
         uint4 qv = make_uint4(0u, 0u, 0u, 0u);
-        if (r0 < n_h) qv = __ldcg((const uint4*)(q + ((size_t)t * n_heads + h0 + r0) * HD + c * 8));
+        if (r0 < n_h && (EXACT || c * 8 < hd)) qv = __ldcg((const uint4*)(q + ((size_t)t * n_heads + h0 + r0) * hd + c * 8));
         *(uint4*)(qs + r0 * HD + ((c ^ (r0 & 7)) * 8)) = qv;
     }
     cp_async_wait<0>();
@@ -432,7 +438,8 @@ __global__ void __launch_bounds__(TC_THREADS, TC_BLOCKS) decode_attention_tc_ker
 #pragma unroll
     for (int j = 0; j < TC_CHUNK / ROWS_STEP; ++j) {
         const int r = r0 + j * ROWS_STEP;
-        cp_async16_zfill(kv + r * HD + ((c ^ (r & 7)) * 8), vplane + (size_t)bases[r] * HD + c * 8, r < count);
+        const bool there = r < count && (EXACT || c * 8 < vd);
+        cp_async16_zfill(kv + r * HD + ((c ^ (r & 7)) * 8), vplane + (there ? (size_t)bases[r] * vd + c * 8 : 0), there);
     }
     cp_async_commit();
     float m0 = smax[0][g];
@@ -479,6 +486,7 @@ __global__ void __launch_bounds__(TC_THREADS, TC_BLOCKS) decode_attention_tc_ker
     // ---- the chunk's result per head: warps added in order ---------------------------------------------
     for (int i = tid; i < n_h * (HD / 2); i += TC_THREADS) {
         const int row = i / (HD / 2), d2 = i % (HD / 2);
+        if (!EXACT && 2 * d2 >= vd) continue;
         float2 a = make_float2(0.0f, 0.0f);
         float l = 0.0f;
 #pragma unroll
@@ -495,7 +503,7 @@ __global__ void __launch_bounds__(TC_THREADS, TC_BLOCKS) decode_attention_tc_ker
             for (int w = 1; w < TC_WARPS; ++w) m = fmaxf(m, smax[w][row]);
             float inv = 1.0f / (l + expf(sink - m));          // the key without a value; sink = -inf: none
             if (head_gate) inv *= 1.0f / (1.0f + expf(-head_gate[(size_t)t * gate_ld + h]));
-            *(__nv_bfloat162*)(out + ((size_t)t * n_heads + h) * HD + 2 * d2) = __floats2bfloat162_rn(a.x * inv, a.y * inv);
+            *(__nv_bfloat162*)(out + ((size_t)t * n_heads + h) * vd + 2 * d2) = __floats2bfloat162_rn(a.x * inv, a.y * inv);
         } else {
             size_t slot = ((size_t)t * n_heads + h) * max_splits + split;
             *(float2*)(part_acc + slot * HD + 2 * d2) = a;
@@ -526,6 +534,7 @@ __global__ void __launch_bounds__(TC_THREADS, TC_BLOCKS) decode_attention_tc_ker
     if (!is_last) return;
     for (int i = tid; i < n_h * (HD / 2); i += TC_THREADS) {
         const int row = i / (HD / 2), d2 = i % (HD / 2);
+        if (!EXACT && 2 * d2 >= vd) continue;
         const int h = h0 + row;
         size_t slot0 = ((size_t)t * n_heads + h) * max_splits;
         float M = -INFINITY;
@@ -541,7 +550,7 @@ __global__ void __launch_bounds__(TC_THREADS, TC_BLOCKS) decode_attention_tc_ker
         }
         float inv = 1.0f / (L + expf(sink - M));
         if (head_gate) inv *= 1.0f / (1.0f + expf(-head_gate[(size_t)t * gate_ld + h]));
-        *(__nv_bfloat162*)(out + ((size_t)t * n_heads + h) * HD + 2 * d2) = __floats2bfloat162_rn(a.x * inv, a.y * inv);
+        *(__nv_bfloat162*)(out + ((size_t)t * n_heads + h) * vd + 2 * d2) = __floats2bfloat162_rn(a.x * inv, a.y * inv);
     }
 }
 
@@ -552,7 +561,7 @@ template <int HD>
 __global__ void __launch_bounds__(128) decode_merge_kernel(
     __nv_bfloat16* __restrict__ out, const float* __restrict__ part_acc, const float* __restrict__ part_ml,
     const int* __restrict__ positions, int T, int n_heads, int window, int max_splits, const float* __restrict__ head_gate,
-    int gate_ld, float sink) {
+    int gate_ld, float sink, int vd) {
     cj::release_successor();
     const int lane = threadIdx.x & 31;
     const long long idx = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -572,7 +581,7 @@ __global__ void __launch_bounds__(128) decode_merge_kernel(
     float M = -INFINITY;
     for (int sidx = 0; sidx < n_splits; ++sidx) M = fmaxf(M, part_ml[(slot0 + sidx) * 2]);
     const float gate = head_gate ? 1.0f / (1.0f + expf(-head_gate[(size_t)(idx / n_heads) * gate_ld + (int)(idx % n_heads)])) : 1.0f;
-    for (int d2 = lane; d2 < HD / 2; d2 += 32) {
+    for (int d2 = lane; d2 < vd / 2; d2 += 32) {
         float L = 0.0f;
         float2 a = make_float2(0.0f, 0.0f);
         for (int sidx = 0; sidx < n_splits; ++sidx) {
@@ -583,7 +592,7 @@ __global__ void __launch_bounds__(128) decode_merge_kernel(
             a.y = fmaf(v.y, f, a.y);
         }
         float inv = gate / (L + expf(sink - M));
-        *(__nv_bfloat162*)(out + (size_t)idx * HD + 2 * d2) = __floats2bfloat162_rn(a.x * inv, a.y * inv);
+        *(__nv_bfloat162*)(out + (size_t)idx * vd + 2 * d2) = __floats2bfloat162_rn(a.x * inv, a.y * inv);
     }
 }
 
@@ -630,17 +639,18 @@ CJ_EXPORT int cj_decode_attention(const void* q, void* out, const void* kplane, 
 }
 
 // The same on the tensor cores (chunks of 128 keys; up to 8 query heads of a kv head a block).
-// counters: int32 [T * n_heads] here (one per row, kv head and batch of 8 heads).
+// counters: int32 [T * n_heads] here (one per row, kv head and batch of 8 heads).  hd, vd: the keys' and the values' sizes,
+// multiples of eight up to 128; part_acc is laid out for rows of 64 (both at most 64) or 128.
 // sink: a constant score of one more key that has no value, exp(sink) in the divisor alone; -infinity: none.
 CJ_EXPORT int cj_decode_attention_tc(const void* q, void* out, const void* kplane, const void* vplane, const int* positions,
                                      const int* row_req, const int* table, int table_stride, int page_tokens, int T,
-                                     int n_heads, int n_kv, int hd, int window, float scale, int max_context,
+                                     int n_heads, int n_kv, int hd, int vd, int window, float scale, int max_context,
                                      float* part_acc, float* part_ml, int* counters, int max_splits, int merge_later,
                                      float softcap, const float* head_gate, int gate_ld, float sink, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (!q || !out || !kplane || !vplane || !positions || !row_req || !table || !part_acc || !part_ml || !counters) return CJ_ERR_ARG;
     if (n_heads <= 0 || n_kv <= 0 || n_heads % n_kv != 0 || page_tokens <= 0) return CJ_ERR_SIZE;
-    if (hd != 64 && hd != 128) return CJ_ERR_SIZE;
+    if (hd <= 0 || vd <= 0 || hd > 128 || vd > 128 || hd % 8 != 0 || vd % 8 != 0) return CJ_ERR_SIZE;
     int span = window > 0 ? min(window, max_context) : max_context;
     int splits = (span + TC_CHUNK - 1) / TC_CHUNK;
     if (splits < 1) splits = 1;
@@ -648,26 +658,29 @@ CJ_EXPORT int cj_decode_attention_tc(const void* q, void* out, const void* kplan
     const int head_batches = (group + TC_HEADS - 1) / TC_HEADS;
     if (splits > max_splits || splits > 65535 || (long long)n_kv * head_batches > 65535) return CJ_ERR_SIZE;
     dim3 grid(T, n_kv * head_batches, splits);
-#define LAUNCH(HD)                                                                                                     \
+#define LAUNCH(HD, EXACT)                                                                                              \
     {                                                                                                                  \
         constexpr int smem = (TC_CHUNK + TC_HEADS) * HD * (int)sizeof(__nv_bfloat16);                                  \
         static_assert(TC_WARPS * TC_HEADS * HD * 4 <= TC_CHUNK * HD * 2, "the warps' partial outputs must fit the tile"); \
         static bool configured = false;                                                                                \
         if (!configured) {                                                                                             \
-            cudaError_t e = cudaFuncSetAttribute(decode_attention_tc_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem); \
+            cudaError_t e = cudaFuncSetAttribute(decode_attention_tc_kernel<HD, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem); \
             if (e != cudaSuccess) return (int)e;                                                                       \
             configured = true;                                                                                         \
         }                                                                                                              \
-        cj::launch(decode_attention_tc_kernel<HD>, dim3(grid), dim3(TC_THREADS), smem, stream, (const __nv_bfloat16*)q, \
+        cj::launch(decode_attention_tc_kernel<HD, EXACT>, dim3(grid), dim3(TC_THREADS), smem, stream, (const __nv_bfloat16*)q, \
             (__nv_bfloat16*)out, (const __nv_bfloat16*)kplane, (const __nv_bfloat16*)vplane, positions, row_req, table, \
             table_stride, page_tokens, n_heads, n_kv, head_batches, window, scale, part_acc, part_ml, counters,        \
-            max_splits, merge_later && splits > 1 ? 1 : 0, softcap, head_gate, gate_ld, sink);                         \
+            max_splits, merge_later && splits > 1 ? 1 : 0, softcap, head_gate, gate_ld, sink, hd, vd);                 \
         if (merge_later && splits > 1)                                                                                 \
             cj::launch(decode_merge_kernel<HD>, dim3((unsigned)(((long long)T * n_heads + 3) / 4)), dim3(128), 0, stream, \
                 (__nv_bfloat16*)out, (const float*)part_acc, (const float*)part_ml, positions, T, n_heads, window, max_splits, \
-                head_gate, gate_ld, sink);                                                                             \
+                head_gate, gate_ld, sink, vd);                                                                         \
     }
-    if (hd == 128) LAUNCH(128) else LAUNCH(64)
+    if (hd == 128 && vd == 128) LAUNCH(128, true)
+    else if (hd == 64 && vd == 64) LAUNCH(64, true)
+    else if (hd > 64 || vd > 64) LAUNCH(128, false)
+    else LAUNCH(64, false)
 #undef LAUNCH
     return launch_status();
 }

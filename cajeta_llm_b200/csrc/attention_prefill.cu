@@ -61,12 +61,16 @@ __device__ __forceinline__ __nv_bfloat16* tile_ptr(__nv_bfloat16* base, int row,
 // HD: head size; BM: query rows a block; BN: keys a tile; MT: 16-row tiles a warp owns.  A
 // warp that owns two row tiles uses every key/value fragment it reads from shared memory
 // twice, which is what the legacy tensor path needs to stay ahead of shared-memory bandwidth.
-template <int HD, int HS, int BM, int BN, int MT>
+// EXACT: keys and values have HD entries each; otherwise hd and vd (multiples of eight, at most HD) are what they have, and
+// the tiles' columns past them are filled with zeros.
+template <int HD, int HS, int BM, int BN, int MT, bool EXACT>
 __global__ void __launch_bounds__(BM / (16 * MT) * 32) prefill_attention_kernel(
     const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ kplane,
     const __nv_bfloat16* __restrict__ vplane, const int* __restrict__ req_start, const int* __restrict__ req_prior,
     int n_requests, const int* __restrict__ table, int table_stride, int page_tokens, int n_heads, int n_kv, int window,
-    float scale, float softcap, const float* __restrict__ head_gate, int gate_ld, float sink_log2) {
+    float scale, float softcap, const float* __restrict__ head_gate, int gate_ld, float sink_log2,
+    int hd_given, int vd_given) {
+    const int hd = EXACT ? HD : hd_given, vd = EXACT ? HD : vd_given;
     cj::after_predecessor();
     cj::release_successor();
     extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -105,26 +109,29 @@ __global__ void __launch_bounds__(BM / (16 * MT) * 32) prefill_attention_kernel(
     // ---- loads -----------------------------------------------------------------------------
     auto load_kv = [&](int kt, int buf) {
         __nv_bfloat16* kd = ks + buf * BN * HS;
-        __nv_bfloat16* vd = vs + buf * BN * HS;
+        __nv_bfloat16* vdst = vs + buf * BN * HS;
         for (int i = tid; i < BN * CH; i += THREADS) {
             int r = i / CH, c = i % CH;
             int key = kt * BN + r;
             bool valid = key <= p_last && key >= key_from;
-            long long off = 0;
+            long long off = 0, voff = 0;
             if (valid) {
                 int page = tab[key / page_tokens];
                 valid = page >= 0;
-                off = (((long long)(valid ? page : 0) * n_kv + kvh) * page_tokens + key % page_tokens) * HD + c * 8;
+                const long long place = ((long long)(valid ? page : 0) * n_kv + kvh) * page_tokens + key % page_tokens;
+                off = place * hd + c * 8;
+                voff = EXACT ? off : place * vd + c * 8;
             }
             int pc = c ^ (r & 7);
-            cp_async16(kd + r * HS + pc * 8, kplane + off, valid);
-            cp_async16(vd + r * HS + pc * 8, vplane + off, valid);
+            const bool k_there = valid && (EXACT || c * 8 < hd), v_there = valid && (EXACT || c * 8 < vd);
+            cp_async16(kd + r * HS + pc * 8, kplane + (k_there ? off : 0), k_there);
+            cp_async16(vdst + r * HS + pc * 8, vplane + (v_there ? voff : 0), v_there);
         }
     };
     for (int i = tid; i < BM * CH; i += THREADS) {
         int r = i / CH, c = i % CH;
-        bool valid = r < rows;
-        const __nv_bfloat16* src = q + ((size_t)(row0 + (valid ? r : 0)) * n_heads + h) * HD + c * 8;
+        bool valid = r < rows && (EXACT || c * 8 < hd);
+        const __nv_bfloat16* src = q + ((size_t)(row0 + (valid ? r : 0)) * n_heads + h) * hd + (valid ? c * 8 : 0);
         cp_async16(qs + r * HS + (c ^ (r & 7)) * 8, src, valid);
     }
     load_kv(kt_begin, 0);
@@ -269,8 +276,9 @@ __global__ void __launch_bounds__(BM / (16 * MT) * 32) prefill_attention_kernel(
 #pragma unroll
         for (int i = 0; i < HD / 8; ++i) {
             int col = i * 8 + 2 * t4;
-            if (r0 < rows) *(unsigned*)(out + ((size_t)(row0 + r0) * n_heads + h) * HD + col) = pack_bf16(o[mt][i][0] * i0, o[mt][i][1] * i0);
-            if (r1 < rows) *(unsigned*)(out + ((size_t)(row0 + r1) * n_heads + h) * HD + col) = pack_bf16(o[mt][i][2] * i1, o[mt][i][3] * i1);
+            if (!EXACT && col >= vd) continue;
+            if (r0 < rows) *(unsigned*)(out + ((size_t)(row0 + r0) * n_heads + h) * vd + col) = pack_bf16(o[mt][i][0] * i0, o[mt][i][1] * i0);
+            if (r1 < rows) *(unsigned*)(out + ((size_t)(row0 + r1) * n_heads + h) * vd + col) = pack_bf16(o[mt][i][2] * i1, o[mt][i][3] * i1);
         }
     }
 }
@@ -278,39 +286,46 @@ __global__ void __launch_bounds__(BM / (16 * MT) * 32) prefill_attention_kernel(
 }  // namespace
 
 // q, out: [T, n_heads, hd] bf16; planes [pages, n_kv, page_tokens, hd] bf16; req_start
-// [n_requests + 1], req_prior [n_requests] as the step function lays them out.  hd must be
-// 32, 64, 96 or 128.  block_rows: 64 or 128 query rows a block, 0 = chosen from the step's shape.  softcap 0: none.
+// [n_requests + 1], req_prior [n_requests] as the step function lays them out.  hd and vd: the keys' and the values'
+// sizes, multiples of eight up to 128.  block_rows: 64 or 128 query rows a block, 0 = chosen from the step's shape.  softcap 0: none.
 // head_gate: null, or float32 with row stride gate_ld whose entry [t, h] gates head h of row t.
 // sink: a constant score of one more key that has no value, exp(sink) in the divisor alone; -infinity: none.
 CJ_EXPORT int cj_prefill_attention(const void* q, void* out, const void* kplane, const void* vplane, const int* req_start,
                                    const int* req_prior, int n_requests, int total_rows, const int* table, int table_stride,
-                                   int page_tokens, int n_heads, int n_kv, int hd, int window, float scale,
+                                   int page_tokens, int n_heads, int n_kv, int hd, int vd, int window, float scale,
                                    int block_rows, float softcap, const float* head_gate, int gate_ld, float sink, cudaStream_t stream) {
     if (total_rows <= 0 || n_requests <= 0) return 0;
     if (!q || !out || !kplane || !vplane || !req_start || !req_prior || !table) return CJ_ERR_ARG;
     if (n_heads <= 0 || n_kv <= 0 || n_heads % n_kv != 0 || page_tokens <= 0 || n_heads > 65535) return CJ_ERR_SIZE;
-    if (hd != 32 && hd != 64 && hd != 96 && hd != 128) return CJ_ERR_SIZE;
+    if (hd <= 0 || vd <= 0 || hd > 128 || vd > 128 || hd % 8 != 0 || vd % 8 != 0) return CJ_ERR_SIZE;
+    const int wide = (hd > vd ? hd : vd), size = wide <= 32 ? 32 : wide <= 64 ? 64 : wide <= 96 ? 96 : 128;
+    const bool exact = hd == size && vd == size;
     // long portions: 128 query rows a block, every warp two row tiles; short ones: 64 rows, one tile a warp
     const int bm = (block_rows == 128 || (block_rows == 0 && total_rows >= 128 * n_requests)) ? 128 : 64;
-#define LAUNCH(HD, HS, BM, BN, MT)                                                                                      \
+#define LAUNCH_AS(HD, HS, BM, BN, MT, EXACT)                                                                            \
     {                                                                                                                   \
         dim3 grid((total_rows + BM - 1) / BM + n_requests, n_heads);                                                    \
         size_t smem = (size_t)(BM + 4 * BN) * HS * sizeof(__nv_bfloat16);                                               \
         static bool configured = false;                                                                                 \
         if (!configured) {                                                                                              \
-            cudaError_t e = cudaFuncSetAttribute(prefill_attention_kernel<HD, HS, BM, BN, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            cudaError_t e = cudaFuncSetAttribute(prefill_attention_kernel<HD, HS, BM, BN, MT, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (e != cudaSuccess) return (int)e;                                                                        \
             configured = true;                                                                                          \
         }                                                                                                               \
-        cj::launch(prefill_attention_kernel<HD, HS, BM, BN, MT>, dim3(grid), dim3(BM / (16 * MT) * 32), smem, stream,                           \
+        cj::launch(prefill_attention_kernel<HD, HS, BM, BN, MT, EXACT>, dim3(grid), dim3(BM / (16 * MT) * 32), smem, stream,                           \
             (const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)kplane, (const __nv_bfloat16*)vplane,   \
             req_start, req_prior, n_requests, table, table_stride, page_tokens, n_heads, n_kv, window, scale, softcap,  \
-            head_gate, gate_ld, sink * 1.4426950408889634f);                                                            \
+            head_gate, gate_ld, sink * 1.4426950408889634f, hd, vd);                                                    \
     }
-    if (hd == 128) { if (bm == 128) LAUNCH(128, 128, 128, 32, 2) else LAUNCH(128, 128, 64, 64, 1) }
-    else if (hd == 96) { if (bm == 128) LAUNCH(96, 128, 128, 32, 2) else LAUNCH(96, 128, 64, 64, 1) }
-    else if (hd == 64) { if (bm == 128) LAUNCH(64, 64, 128, 64, 2) else LAUNCH(64, 64, 64, 64, 1) }
+#define LAUNCH(HD, HS, BM, BN, MT)                                                                                      \
+    {                                                                                                                   \
+        if (exact) LAUNCH_AS(HD, HS, BM, BN, MT, true) else LAUNCH_AS(HD, HS, BM, BN, MT, false)                        \
+    }
+    if (size == 128) { if (bm == 128) LAUNCH(128, 128, 128, 32, 2) else LAUNCH(128, 128, 64, 64, 1) }
+    else if (size == 96) { if (bm == 128) LAUNCH(96, 128, 128, 32, 2) else LAUNCH(96, 128, 64, 64, 1) }
+    else if (size == 64) { if (bm == 128) LAUNCH(64, 64, 128, 64, 2) else LAUNCH(64, 64, 64, 64, 1) }
     else { if (bm == 128) LAUNCH(32, 64, 128, 64, 2) else LAUNCH(32, 64, 64, 64, 1) }
 #undef LAUNCH
+#undef LAUNCH_AS
     return launch_status();
 }

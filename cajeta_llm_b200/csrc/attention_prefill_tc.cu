@@ -149,14 +149,16 @@ __device__ __forceinline__ float capped_score(float s, float in_cap, float cap_l
     return s == -INFINITY ? -INFINITY : y;
 }
 
-// Capped scores in full float32.  CAP_POLY: every |s| scale / cap is known to be at most CAP_POLY_REACH (queries and keys of
-// known length), where tanh(x) = x P(x^2) with the P below, whose relative error over that reach is 1.1e-7 (a minimax fit of
-// tanh(x) / x in x^2 with five terms); the arguments' scaling and the cap are folded into the terms by the host, so a score
-// costs three packed multiply-adds and no second special function.  CAP_EXP: any score, tanh(x) = 1 - 2 / (e^2x + 1).
-constexpr int CAP_NONE = 0, CAP_APPROX = 1, CAP_POLY = 2, CAP_EXP = 3;
-constexpr float CAP_POLY_REACH = 0.625f;
-constexpr int CAP_TERMS = 5;
-constexpr double CAP_P[CAP_TERMS] = {0.9999998931, -0.3333195425, 0.1330452599, -0.05182186644, 0.01505094485};
+// Capped scores in full float32.  CAP_POLY + n: every |s| scale / cap is known to be at most cap_reach(n) (queries and keys of
+// known length), where tanh(x) = x P(x^2) with n terms of the P below, whose relative error over that reach is at most 1.1e-7
+// (minimax fits of tanh(x) / x in x^2); the arguments' scaling and the cap are folded into the terms by the host, so a pair of
+// scores costs n + 1 packed operations and no second special function.  CAP_EXP: any score, tanh(x) = 1 - 2 / (e^2x + 1).
+constexpr int CAP_NONE = 0, CAP_APPROX = 1, CAP_EXP = 2, CAP_POLY = 10;
+constexpr int CAP_TERMS = 5;                           // at most; at least three
+inline float cap_reach(int terms) { return terms == 3 ? 0.21f : terms == 4 ? 0.40f : 0.625f; }
+constexpr double CAP_P[3][CAP_TERMS] = {{0.9999998594, -0.3332758288, 0.1298347298, 0, 0},
+                                        {0.9999999019, -0.3333136246, 0.1327097676, -0.04755360348, 0},
+                                        {0.9999998931, -0.3333195425, 0.1330452599, -0.05182186644, 0.01505094485}};
 
 __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
     f32x2 d;
@@ -490,13 +492,14 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
                     for (int c = 0; c < HC; c += 4) {
                         float2 t0, t1;
-                        if (CAP == CAP_POLY) {
+                        if (CAP > CAP_POLY) {
+                            constexpr int N = CAP > CAP_POLY ? CAP - CAP_POLY : CAP_TERMS;
                             const f32x2 s0 = pack2(__uint_as_float(v[c]), __uint_as_float(v[c + 1]));
                             const f32x2 s1 = pack2(__uint_as_float(v[c + 2]), __uint_as_float(v[c + 3]));
                             const f32x2 x0 = mul2(s0, s0), x1 = mul2(s1, s1);
-                            f32x2 p0 = pack2(p.cap_p[CAP_TERMS - 1], p.cap_p[CAP_TERMS - 1]), p1 = p0;
+                            f32x2 p0 = pack2(p.cap_p[N - 1], p.cap_p[N - 1]), p1 = p0;
 #pragma unroll
-                            for (int k = CAP_TERMS - 2; k >= 0; --k) {
+                            for (int k = N - 2; k >= 0; --k) {
                                 const f32x2 ck = pack2(p.cap_p[k], p.cap_p[k]);
                                 p0 = fma2(p0, x0, ck);
                                 p1 = fma2(p1, x1, ck);
@@ -648,7 +651,11 @@ CJ_EXPORT int cj_prefill_attention_tc(const void* q, void* out, const void* kpla
         if (e == cudaSuccess)
             e = cudaFuncSetAttribute(prefill_attention_tc_kernel<CAP_APPROX>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
         if (e == cudaSuccess)
-            e = cudaFuncSetAttribute(prefill_attention_tc_kernel<CAP_POLY>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
+            e = cudaFuncSetAttribute(prefill_attention_tc_kernel<CAP_POLY + 3>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
+        if (e == cudaSuccess)
+            e = cudaFuncSetAttribute(prefill_attention_tc_kernel<CAP_POLY + 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
+        if (e == cudaSuccess)
+            e = cudaFuncSetAttribute(prefill_attention_tc_kernel<CAP_POLY + 5>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
         if (e == cudaSuccess)
             e = cudaFuncSetAttribute(prefill_attention_tc_kernel<CAP_EXP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
         if (e != cudaSuccess) return (int)e;
@@ -674,11 +681,13 @@ CJ_EXPORT int cj_prefill_attention_tc(const void* q, void* out, const void* kpla
            softcap > 0.0f ? scale / softcap : 0.0f, {}, sink * 1.4426950408889634f, head_gate, gate_ld, (int)plane_rows, block_rows};
     int cap = softcap > 0.0f ? CAP_APPROX : CAP_NONE;
     if (softcap > 0.0f && exact_cap) {
-        cap = score_bound > 0.0f && score_bound <= CAP_POLY_REACH * softcap ? CAP_POLY : CAP_EXP;
+        cap = CAP_EXP;
+        for (int n = CAP_TERMS; n >= 3; --n)
+            if (score_bound > 0.0f && score_bound <= cap_reach(n) * softcap) cap = CAP_POLY + n;
         // cap log2(e) tanh(x), x = s scale / cap: the k-th term carries x^(2k + 1)
         const double x = (double)scale / (double)softcap;
         double f = (double)softcap * 1.4426950408889634 * x;
-        for (int k = 0; k < CAP_TERMS; ++k, f *= x * x) a.cap_p[k] = (float)(CAP_P[k] * f);
+        for (int k = 0; k < CAP_TERMS; ++k, f *= x * x) a.cap_p[k] = (float)(CAP_P[cap > CAP_POLY ? cap - CAP_POLY - 3 : 0][k] * f);
     }
     // heads run fastest, so that blocks start in the order of their length (the last rows of a
     // request see the most keys) and the heads of one group read the same keys one after another
@@ -686,7 +695,8 @@ CJ_EXPORT int cj_prefill_attention_tc(const void* q, void* out, const void* kpla
     if (row_blocks > 65535) return CJ_ERR_SIZE;
     dim3 grid(n_heads, (unsigned)row_blocks);
     auto kern = cap == CAP_NONE ? prefill_attention_tc_kernel<CAP_NONE> : cap == CAP_APPROX ? prefill_attention_tc_kernel<CAP_APPROX>
-                : cap == CAP_POLY ? prefill_attention_tc_kernel<CAP_POLY> : prefill_attention_tc_kernel<CAP_EXP>;
+                : cap == CAP_POLY + 3 ? prefill_attention_tc_kernel<CAP_POLY + 3> : cap == CAP_POLY + 4 ? prefill_attention_tc_kernel<CAP_POLY + 4>
+                : cap == CAP_POLY + 5 ? prefill_attention_tc_kernel<CAP_POLY + 5> : prefill_attention_tc_kernel<CAP_EXP>;
     cj::launch(kern, dim3(grid), dim3(THREADS), SMEM_TOTAL, stream, mq, mk, mv, a);
     return cj::launch_status();
 }

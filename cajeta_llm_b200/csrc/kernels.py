@@ -1207,8 +1207,9 @@ def decode_attention(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor, 
                      n_heads: int, n_kv: int, head_dim: int, window: int, scale: float, max_context: int,
                      scratch: "DecodeScratch", chunk: int = 0, tensor_cores: Optional[bool] = None,
                      merge_later: Optional[bool] = None, softcap: float = 0.0, head_gate: Optional[torch.Tensor] = None,
-                     gate_offset: int = 0, sink: float = NO_SINK) -> None:
-    """Split-KV attention of few bfloat16 query rows over their cached keys (head_dim 64 or 128).
+                     gate_offset: int = 0, sink: float = NO_SINK, value_dim: int = 0) -> None:
+    """Split-KV attention of few bfloat16 query rows over their cached keys (the tensor-core form: sizes that
+    :func:`tile_sizes` takes, ``value_dim`` = the values' when it is not the keys'; the other: head_dim 64 or 128).
     ``tensor_cores``: scores and weighted values of a chunk by mma.sync (the default) or on the
     FMA pipe (``chunk`` 64 or 128 applies to that form only).  ``merge_later``: the chunks of a
     row are merged by a kernel of its own instead of the row's last block (the default for steps
@@ -1221,15 +1222,16 @@ def decode_attention(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor, 
     span = min(window, max_context) if window > 0 else max_context
     gate_ptr, gate_ld = _gate(head_gate, gate_offset)
     if tensor_cores is None:
-        tensor_cores = (DECODE_TENSOR_CORES and chunk == 0) or softcap > 0.0 or head_gate is not None or sink != NO_SINK
+        tensor_cores = (DECODE_TENSOR_CORES and chunk == 0) or softcap > 0.0 or head_gate is not None or sink != NO_SINK or value_dim not in (0, head_dim) or head_dim not in (64, 128)
+    vd = value_dim or head_dim
     if tensor_cores:
         splits = max(1, -(-span // 128))
-        scratch.ensure(T, n_heads, n_kv, head_dim, splits, q.device)
+        scratch.ensure(T, n_heads, n_kv, 64 if max(head_dim, vd) <= 64 else 128, splits, q.device)
         if merge_later is None:
             merge_later = T * n_heads >= MERGE_LATER_MIN_ROW_HEADS
         st = library("attention_decode").cj_decode_attention_tc(
             _ptr(q), _ptr(out), _ptr(k_plane), _ptr(v_plane), _ptr(positions), _ptr(row_req), _ptr(table),
-            _i(table.stride(0)), _i(page_tokens), _i(T), _i(n_heads), _i(n_kv), _i(head_dim), _i(window), _f(scale),
+            _i(table.stride(0)), _i(page_tokens), _i(T), _i(n_heads), _i(n_kv), _i(head_dim), _i(vd), _i(window), _f(scale),
             _i(max_context), _ptr(scratch.acc), _ptr(scratch.ml), _ptr(scratch.counters), _i(scratch.splits),
             _i(1 if merge_later else 0), _f(softcap), gate_ptr, _i(gate_ld), _f(sink), _stream())
         _check(st, "decode_attention")
@@ -1237,7 +1239,7 @@ def decode_attention(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor, 
             global launches
             launches += 1                  # the merge kernel
         return
-    if softcap > 0.0 or head_gate is not None or sink != NO_SINK:
+    if softcap > 0.0 or head_gate is not None or sink != NO_SINK or vd != head_dim:
         raise KernelError("decode_attention: capped scores, gated heads and a sink are built into the tensor-core form only")
     chunk = chunk or decode_chunk(span)
     splits = max(1, -(-span // chunk))
@@ -1247,6 +1249,11 @@ def decode_attention(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor, 
         _i(page_tokens), _i(T), _i(n_heads), _i(n_kv), _i(head_dim), _i(window), _f(scale), _i(max_context),
         _ptr(scratch.acc), _ptr(scratch.ml), _ptr(scratch.counters), _i(scratch.splits), _i(chunk), _stream())
     _check(st, "decode_attention")
+
+
+def tile_sizes(head_dim: int, value_dim: int) -> bool:
+    """Whether the tiled attention kernels on ``mma.sync`` (prompt portions, decode) take these sizes of keys and values."""
+    return head_dim % 8 == 0 and value_dim % 8 == 0 and 0 < head_dim <= 128 and 0 < value_dim <= 128
 
 
 class DecodeScratch:
@@ -1271,9 +1278,10 @@ def prefill_attention(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor,
                       req_start: torch.Tensor, req_prior: torch.Tensor, table: torch.Tensor, page_tokens: int,
                       n_heads: int, n_kv: int, head_dim: int, window: int, scale: float, block_rows: int = 0,
                       softcap: float = 0.0, head_gate: Optional[torch.Tensor] = None, gate_offset: int = 0,
-                      sink: float = NO_SINK) -> None:
+                      sink: float = NO_SINK, value_dim: int = 0) -> None:
     """Tensor-core attention of a step's rows (request r owns rows req_start[r]..req_start[r+1]
-    at positions req_prior[r] + i) over the paged cache; bfloat16, head_dim 32, 64, 96 or 128.
+    at positions req_prior[r] + i) over the paged cache; bfloat16, sizes that :func:`tile_sizes` takes
+    (``value_dim``: the values' when it is not the keys').
     ``softcap``, ``head_gate`` and ``sink`` as in ``paged_attention``."""
     for n, t in (("q", q), ("out", out), ("k_plane", k_plane), ("v_plane", v_plane)):
         _need(t, n, torch.bfloat16)
@@ -1281,8 +1289,8 @@ def prefill_attention(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor,
     gate_ptr, gate_ld = _gate(head_gate, gate_offset)
     st = library("attention_prefill").cj_prefill_attention(
         _ptr(q), _ptr(out), _ptr(k_plane), _ptr(v_plane), _ptr(req_start), _ptr(req_prior), _i(req_prior.numel()),
-        _i(q.shape[0]), _ptr(table), _i(table.stride(0)), _i(page_tokens), _i(n_heads), _i(n_kv), _i(head_dim), _i(window),
-        _f(scale), _i(block_rows), _f(softcap), gate_ptr, _i(gate_ld), _f(sink), _stream())
+        _i(q.shape[0]), _ptr(table), _i(table.stride(0)), _i(page_tokens), _i(n_heads), _i(n_kv), _i(head_dim),
+        _i(value_dim or head_dim), _i(window), _f(scale), _i(block_rows), _f(softcap), gate_ptr, _i(gate_ld), _f(sink), _stream())
     _check(st, "prefill_attention")
 
 

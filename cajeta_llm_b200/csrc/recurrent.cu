@@ -538,7 +538,7 @@ __global__ void softcap_rows_kernel(float* __restrict__ x, float cap, long long 
 // zp, u and g are columns off_z + k, off_x + k, off_g + k of the step's projected rows (biases included).  Because the
 // gates do not read the state, a stretch of tokens is one affine map S -> A S + B, and stretches compose: a block takes
 // CT neighbouring channels of one request, a thread PER consecutive tokens of a channel (their a = 1 - z and b = z c in
-// registers), the threads of a channel compose their stretches' maps by a warp's prefix scan, and every thread
+// registers), a warp composes the maps of a channel's stretches by a prefix scan, and every thread
 // then walks its tokens from the state its stretch begins with.  A request is cut into tiles from its own first row of the
 // step; requests of a few tokens (single decoded ones) are walked by a thread a channel instead, in the leading blocks.
 // Everything is float32 but the result.
@@ -550,32 +550,68 @@ struct GatedScanArgs {
     long long slot_stride;
     const int* req_start;
     const int* req_slot;
+    int vec;         // rows and column offsets on 16-byte boundaries
+    int single;      // every request brings one token
 };
 
+// e^x, 1 / x: CUDA's own for float32 results; FAST (results rounded to bfloat16): the special-function unit's, a few units in
+// the last place of float32
+template <bool FAST> __device__ __forceinline__ float gs_exp(float x) {
+    if (!FAST) return expf(x);
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x * 1.4426950408889634f));
+    return y;
+}
+template <bool FAST> __device__ __forceinline__ float gs_rcp(float x) {
+    if (!FAST) return 1.0f / x;
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+template <bool FAST> __device__ __forceinline__ float gs_silu(float x) { return x * gs_rcp<FAST>(1.0f + gs_exp<FAST>(-fmaxf(x, -80.0f))); }
+
 // a = 1 - z and b = z c; both sides of the sigmoid come from one exponential, so neither loses digits near 0 or 1
+template <bool FAST>
 __device__ __forceinline__ void gated_step(float zp, float u, float& a, float& b) {
-    const float e = expf(-fabsf(zp)), big = 1.0f / (1.0f + e), small = e * big;
+    const float e = gs_exp<FAST>(-fabsf(zp)), big = gs_rcp<FAST>(1.0f + e), small = e * big;
     const float z = zp >= 0.0f ? big : small;
     a = zp >= 0.0f ? small : big;
-    b = z * (u >= 0.0f ? u + 0.5f : sigmoid_f(u));
+    const float below = gs_rcp<FAST>(1.0f + gs_exp<FAST>(fminf(-u, 80.0f)));      // sigmoid(u); the bound keeps e^(-u) finite
+    b = z * (u >= 0.0f ? u + 0.5f : below);
 }
 
-constexpr int GS_PER = 16;           // tokens a thread takes in a tile; a request of at most this many is walked by a thread a channel
-constexpr int GS_THREADS = 512;
+constexpr int GS_WALK = 16;          // a request of at most this many tokens is walked by a thread a channel
 
-template <typename TO, int CT>
-__global__ void __launch_bounds__(GS_THREADS) gated_scan_kernel(GatedScanArgs p, TO* __restrict__ out) {
+// 16 bytes, or four times 4 where the rows are not aligned for that, on their way to shared memory
+__device__ __forceinline__ void cp_async16(float* smem, const float* gmem) {
+    unsigned s = (unsigned)__cvta_generic_to_shared(smem);
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(s), "l"(gmem) : "memory");
+}
+
+// A block takes CT (8, 16 or 32) neighbouring channels and 32 CT threads: 32 stretches of PER tokens each make a tile.  The
+// next tile's pre-activations travel to shared memory (cp.async) while this one is worked on; a stretch's tokens lie CT floats
+// apart and stretches CT (PER + 1), which keeps the reads of a warp (CT channels of 32 / CT stretches) in different banks.
+constexpr int GS_SEG = 32;
+template <int CT, int PER> struct GatedScanTile {
+    static constexpr int TOKENS = GS_SEG * PER, PLANE = GS_SEG * CT * (PER + 1), FLOATS = 3 * PLANE, BYTES = 2 * FLOATS * 4;
+};
+
+template <typename TO, int CT, int PER, int BLOCKS>
+__global__ void __launch_bounds__(32 * CT, BLOCKS) gated_scan_kernel(GatedScanArgs p, TO* __restrict__ out) {
     cj::after_predecessor();
     cj::release_successor();
-    constexpr int NSEG = GS_THREADS / CT;          // stretches of a tile, one a thread
-    constexpr int PL = NSEG / 32;                  // stretches a lane of the composing warp holds
-    static_assert(NSEG % 32 == 0 && CT <= GS_THREADS / 32, "a warp composes a channel's stretches");
+    constexpr bool FAST = sizeof(TO) == 2;
+    using Tile = GatedScanTile<CT, PER>;
+    constexpr int THREADS = 32 * CT;
+    extern __shared__ __align__(16) float gs_buf[];             // [2][z | x | g]
+    __shared__ float As[GS_SEG][CT + 1], Bs[GS_SEG][CT + 1];      // a stretch's map, then (in Bs) the state it begins with
+    __shared__ float carry[CT];
     const int req = blockIdx.y;
     const int slot = p.req_slot[req];
     const int first = p.req_start[req], n = p.req_start[req + 1] - first;
     if (slot < 0 || n <= 0) return;
     float* st = p.state + (size_t)slot * p.slot_stride;
-    if (n <= GS_PER || blockDim.x != GS_THREADS) {
+    if (n <= GS_WALK || p.single) {
         // a thread a channel: the launch has at least enough blocks of its size for all channels
         const int c = blockIdx.x * blockDim.x + threadIdx.x;
         if (c >= p.width) return;
@@ -584,53 +620,73 @@ __global__ void __launch_bounds__(GS_THREADS) gated_scan_kernel(GatedScanArgs p,
             const float* row = p.x + (size_t)(first + t) * p.ld;
             const float g = row[p.off_g + c];
             float a, b;
-            gated_step(row[p.off_z + c], row[p.off_x + c], a, b);
+            gated_step<FAST>(row[p.off_z + c], row[p.off_x + c], a, b);
             S = fmaf(a, S, b);
-            out[(size_t)(first + t) * p.width + c] = from_f32<TO>(S * silu(g));
+            out[(size_t)(first + t) * p.width + c] = from_f32<TO>(S * gs_silu<FAST>(g));
         }
         st[c] = S;
         return;
     }
-    __shared__ float As[NSEG][CT + 1], Bs[NSEG][CT + 1];        // a stretch's map, then (in Bs) the state it begins with
-    __shared__ float carry[CT];
+    const int c0 = blockIdx.x * CT, nch = min(CT, p.width - c0);
     const int ch = threadIdx.x % CT, seg = threadIdx.x / CT;
-    const int c = blockIdx.x * CT + ch;
-    const bool live = c < p.width;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    if (threadIdx.x < CT) carry[threadIdx.x] = live ? st[c] : 0.0f;
-    for (int tile0 = 0; tile0 < n; tile0 += NSEG * GS_PER) {
-        const int t0 = tile0 + seg * GS_PER;
-        const int mine = live ? max(0, min(GS_PER, n - t0)) : 0;
-        const float* row = p.x + (size_t)(first + t0) * p.ld + c;
-        float a[GS_PER], b[GS_PER];
-#pragma unroll
-        for (int i = 0; i < GS_PER; ++i) {
-            a[i] = i < mine ? row[(size_t)i * p.ld + p.off_z] : 0.0f;
-            b[i] = i < mine ? row[(size_t)i * p.ld + p.off_x] : 0.0f;
+    const bool live = ch < nch;
+    auto fetch = [&](int tile0, float* buf) {
+        const int rows = min(Tile::TOKENS, n - tile0);
+        const float* src = p.x + (size_t)(first + tile0) * p.ld + c0;
+        if (p.vec && nch == CT) {
+            for (int e = threadIdx.x; e < Tile::TOKENS * (CT / 4); e += THREADS) {
+                const int t = e / (CT / 4), h = (e % (CT / 4)) * 4;
+                if (t >= rows) break;
+                const float* r = src + (size_t)t * p.ld + h;
+                float* d = buf + (t + t / PER) * CT + h;
+                cp_async16(d, r + p.off_z);
+                cp_async16(d + Tile::PLANE, r + p.off_x);
+                cp_async16(d + 2 * Tile::PLANE, r + p.off_g);
+            }
+        } else {
+            for (int e = threadIdx.x; e < Tile::TOKENS * CT; e += THREADS) {
+                const int t = e / CT, k = e % CT;
+                if (t >= rows) break;
+                if (k >= nch) continue;
+                const float* r = src + (size_t)t * p.ld + k;
+                float* d = buf + (t + t / PER) * CT + k;
+                cp_async4(d, r + p.off_z);
+                cp_async4(d + Tile::PLANE, r + p.off_x);
+                cp_async4(d + 2 * Tile::PLANE, r + p.off_g);
+            }
         }
+    };
+    if (threadIdx.x < CT) carry[threadIdx.x] = live ? st[c0 + ch] : 0.0f;
+    fetch(0, gs_buf);
+    cp_async_commit();
+    int cur = 0;
+    for (int tile0 = 0; tile0 < n; tile0 += Tile::TOKENS, cur ^= 1) {
+        if (tile0 + Tile::TOKENS < n) fetch(tile0 + Tile::TOKENS, gs_buf + (cur ^ 1) * Tile::FLOATS);
+        cp_async_commit();
+        cp_async_wait<1>();
+        __syncthreads();
+        const float* mine = gs_buf + cur * Tile::FLOATS + seg * CT * (PER + 1) + ch;
+        const int t0 = tile0 + seg * PER;
+        const int have = live ? min(PER, n - t0) : 0;           // tokens of this stretch (none: zero or below)
+        float a[PER], b[PER];
         float A = 1.0f, B = 0.0f;
 #pragma unroll
-        for (int i = 0; i < GS_PER; ++i) {
+        for (int i = 0; i < PER; ++i) {
             float ai, bi;
-            gated_step(a[i], b[i], ai, bi);
-            a[i] = i < mine ? ai : 1.0f;                        // past the end: the map that changes nothing
-            b[i] = i < mine ? bi : 0.0f;
+            gated_step<FAST>(mine[i * CT], mine[Tile::PLANE + i * CT], ai, bi);
+            a[i] = i < have ? ai : 1.0f;                        // past the end (whatever lies there): the map that changes nothing
+            b[i] = i < have ? bi : 0.0f;
             A *= a[i];
             B = fmaf(a[i], B, b[i]);
         }
         As[seg][ch] = A;
         Bs[seg][ch] = B;
         __syncthreads();
-        if (warp < CT) {
-            // this warp composes channel `warp`: a lane its PL stretches in order, then a prefix scan over the lanes
-            float la[PL], lb[PL], ta = 1.0f, tb = 0.0f;
-#pragma unroll
-            for (int k = 0; k < PL; ++k) {
-                la[k] = As[lane * PL + k][warp];
-                lb[k] = Bs[lane * PL + k][warp];
-                tb = fmaf(la[k], tb, lb[k]);
-                ta *= la[k];
-            }
+        {
+            // a warp a channel: its 32 stretches' maps composed by a prefix scan over the lanes
+            float ta = As[lane][warp], tb = Bs[lane][warp];
+            const float S0 = carry[warp];
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
                 const float pa = __shfl_up_sync(0xffffffffu, ta, o), pb = __shfl_up_sync(0xffffffffu, tb, o);
@@ -639,32 +695,24 @@ __global__ void __launch_bounds__(GS_THREADS) gated_scan_kernel(GatedScanArgs p,
                     ta *= pa;
                 }
             }
-            const float S0 = carry[warp];
-            float pa = __shfl_up_sync(0xffffffffu, ta, 1), pb = __shfl_up_sync(0xffffffffu, tb, 1);
-            float S = lane == 0 ? S0 : fmaf(pa, S0, pb);        // the state this lane's first stretch begins with
-#pragma unroll
-            for (int k = 0; k < PL; ++k) {
-                Bs[lane * PL + k][warp] = S;
-                S = fmaf(la[k], S, lb[k]);
-            }
+            const float end = fmaf(ta, S0, tb);                 // the state after this lane's stretch
+            float begin = __shfl_up_sync(0xffffffffu, end, 1);
+            if (lane == 0) begin = S0;
+            Bs[lane][warp] = begin;
             __syncwarp();
-            if (lane == 31) carry[warp] = S;
+            if (lane == 31) carry[warp] = end;
         }
         __syncthreads();
         float S = Bs[seg][ch];
-        const float* grow = row + p.off_g;
-        float g[GS_PER];
+        TO* dst = out + (size_t)(first + t0) * p.width + c0 + ch;
 #pragma unroll
-        for (int i = 0; i < GS_PER; ++i) g[i] = i < mine ? grow[(size_t)i * p.ld] : 0.0f;
-        TO* dst = out + (size_t)(first + t0) * p.width + c;
-#pragma unroll
-        for (int i = 0; i < GS_PER; ++i) {
+        for (int i = 0; i < PER; ++i) {
             S = fmaf(a[i], S, b[i]);
-            if (i < mine) dst[(size_t)i * p.width] = from_f32<TO>(S * silu(g[i]));
+            if (i < have) dst[(size_t)i * p.width] = from_f32<TO>(S * gs_silu<FAST>(mine[2 * Tile::PLANE + i * CT]));
         }
-        __syncthreads();                                        // Bs is read before the next tile writes it
+        __syncthreads();                                        // this buffer and Bs are read before the next tile writes them
     }
-    if (threadIdx.x < CT && live) st[c] = carry[threadIdx.x];
+    if (threadIdx.x < nch) st[c0 + threadIdx.x] = carry[threadIdx.x];
 }
 
 }  // namespace
@@ -848,25 +896,33 @@ CJ_EXPORT int cj_gated_scan(const float* x, int ld, int off_z, int off_x, int of
     if (requests <= 0) return 0;
     if (!x || !state || !req_start || !req_slot || !out) return CJ_ERR_ARG;
     if (width <= 0 || ld < width || slot_stride < width || requests > 65535) return CJ_ERR_SIZE;
-    GatedScanArgs p{x, ld, off_z, off_x, off_g, width, state, slot_stride, req_start, req_slot};
-    // single tokens: small blocks, a thread a channel.  Otherwise tiles of 16 channels (64-byte pieces of a row), or of 8
-    // when tiles of 16 would leave SMs idle.
-    if (single) {
-        const dim3 grid((width + 127) / 128, requests);
-        if (out_dtype == CJ_F32) cj::launch(gated_scan_kernel<float, 16>, grid, dim3(128), 0, stream, p, (float*)out);
-        else if (out_dtype == CJ_BF16) cj::launch(gated_scan_kernel<__nv_bfloat16, 16>, grid, dim3(128), 0, stream, p, (__nv_bfloat16*)out);
-        else return CJ_ERR_DTYPE;
-        return launch_status();
-    }
-    const int ct = (long long)((width + 15) / 16) * requests >= 132 ? 16 : 8;
-    const dim3 grid((width + ct - 1) / ct, requests);
-#define LAUNCH(TO)                                                                                            \
-    if (ct == 16) cj::launch(gated_scan_kernel<TO, 16>, grid, dim3(GS_THREADS), 0, stream, p, (TO*)out);      \
-    else cj::launch(gated_scan_kernel<TO, 8>, grid, dim3(GS_THREADS), 0, stream, p, (TO*)out)
-    if (out_dtype == CJ_F32) { LAUNCH(float); }
-    else if (out_dtype == CJ_BF16) { LAUNCH(__nv_bfloat16); }
+    const int vec = (ld | off_z | off_x | off_g) % 4 == 0 && ((uintptr_t)x & 15) == 0;
+    GatedScanArgs p{x, ld, off_z, off_x, off_g, width, state, slot_stride, req_start, req_slot, vec, single};
+    // single tokens: small blocks, a thread a channel, no tile.  Otherwise 16 channels a block (64-byte pieces of a row; measured
+    // on 2,048 and 8,192 rows of 6,144 channels 55 / 184 us against 64 / 217 us with 8), or 8 where that leaves room on the SMs
+    // (3,072 channels: 37 / 118 us against 41 / 127 us)
+    const bool wide = (long long)((width + 15) / 16) * requests >= 2 * 148;
+#define LAUNCH_CT(TO, CT, BLOCKS)                                                                                       \
+    do {                                                                                                                \
+        constexpr int bytes = GatedScanTile<CT, 8>::BYTES;                                                              \
+        static bool sized = false;                                                                                      \
+        if (!sized) {                                                                                                   \
+            cudaFuncSetAttribute(gated_scan_kernel<TO, CT, 8, BLOCKS>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes); \
+            sized = true;                                                                                               \
+        }                                                                                                               \
+        const dim3 grid(single ? (width + 127) / 128 : (width + CT - 1) / CT, requests);                                \
+        cj::launch(gated_scan_kernel<TO, CT, 8, BLOCKS>, grid, dim3(single ? 128 : 32 * CT), single ? 0 : bytes, stream, p, (TO*)out); \
+    } while (0)
+#define LAUNCH(TO)                                                                                                      \
+    do {                                                                                                                \
+        if (wide) LAUNCH_CT(TO, 16, 2);                                                                                 \
+        else LAUNCH_CT(TO, 8, 3);                                                                                       \
+    } while (0)
+    if (out_dtype == CJ_F32) LAUNCH(float);
+    else if (out_dtype == CJ_BF16) LAUNCH(__nv_bfloat16);
     else return CJ_ERR_DTYPE;
 #undef LAUNCH
+#undef LAUNCH_CT
     return launch_status();
 }
 

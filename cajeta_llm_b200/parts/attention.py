@@ -193,11 +193,8 @@ class PagedAttention(Part):
                 libs.add("attention_mixed")
         elif self.general:
             libs.add("attention_paged")
-            if self.runtime.fast_kernels and self.value_dim == self.head_dim:
-                if self.head_dim in (64, 128):
-                    libs.add("attention_decode")
-                if self.head_dim in (32, 64, 96, 128):
-                    libs.add("attention_prefill_tc" if self.head_dim == 128 else "attention_prefill")
+            if self.runtime.fast_kernels and K.tile_sizes(self.head_dim, self.value_dim):
+                libs |= {"attention_decode", "attention_prefill_tc" if self.head_dim == self.value_dim == 128 else "attention_prefill"}
         elif self.runtime.fast_kernels and self.head_dim in (64, 128):
             libs |= {"attention_decode", "attention_prefill_tc" if self.head_dim == 128 else "attention_prefill"}
         else:
@@ -301,24 +298,24 @@ class PagedAttention(Part):
         out = torch.empty((T, self.heads, self.value_dim), dtype=rt.act_dtype, device=x.device)
         K.tag = "attention"
         gate = qkv if gate_cols else None
-        fast = rt.fast_kernels and self.value_dim == self.head_dim
-        if fast and getattr(ctx, "all_single", False) and self.head_dim in (64, 128):
+        fast = rt.fast_kernels and K.tile_sizes(self.head_dim, self.value_dim)
+        if fast and getattr(ctx, "all_single", False):
             # every request brings one token: the split-KV decode kernel
             K.decode_attention(q, out, entry.k_plane, entry.v_plane, ctx.positions, ctx.row_req, entry.block_table,
                                entry.page_tokens, self.heads, self.kv_heads, self.head_dim, self.window, self.scale,
                                ctx.max_context, getattr(ctx, "decode_scratch", None) or rt.decode_scratch,
-                               softcap=self.softcap, head_gate=gate, gate_offset=g_off, sink=self.sink_score)
-        elif fast and self.head_dim == 128 and entry.page_tokens == 16 and hasattr(ctx, "req_start"):
+                               softcap=self.softcap, head_gate=gate, gate_offset=g_off, sink=self.sink_score, value_dim=self.value_dim)
+        elif fast and self.head_dim == 128 and self.value_dim == 128 and entry.page_tokens == 16 and hasattr(ctx, "req_start"):
             # portions of prompts (and whatever single tokens ride along): both products on tcgen05
             K.prefill_attention_tc(q, out, entry.k_plane, entry.v_plane, ctx.req_start, ctx.req_prior, entry.block_table,
                                    entry.page_tokens, self.heads, self.kv_heads, self.head_dim, self.window, self.scale,
                                    softcap=self.softcap, head_gate=gate, gate_offset=g_off, sink=self.sink_score,
                                    exact_cap=self.exact_cap, score_bound=self.score_bound)
-        elif fast and self.head_dim in (32, 64, 96, 128) and hasattr(ctx, "req_start"):
+        elif fast and hasattr(ctx, "req_start"):
             # portions of prompts (and whatever single tokens ride along): query tiles on the tensor cores
             K.prefill_attention(q, out, entry.k_plane, entry.v_plane, ctx.req_start, ctx.req_prior, entry.block_table,
                                 entry.page_tokens, self.heads, self.kv_heads, self.head_dim, self.window, self.scale,
-                                softcap=self.softcap, head_gate=gate, gate_offset=g_off, sink=self.sink_score)
+                                softcap=self.softcap, head_gate=gate, gate_offset=g_off, sink=self.sink_score, value_dim=self.value_dim)
         else:
             K.paged_attention(q, out, entry.k_plane, entry.v_plane, ctx.positions, ctx.row_req, entry.block_table, entry.page_tokens,
                               self.heads, self.kv_heads, self.head_dim, self.window, self.scale, value_dim=self.value_dim,
