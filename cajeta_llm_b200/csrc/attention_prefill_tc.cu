@@ -172,12 +172,11 @@ __device__ __forceinline__ float ex2(float x) {       // 2^x, 0 for -inf
     return y;
 }
 
-__device__ __forceinline__ float capped_score_exp(float s, float in_cap, float cap_log2, float neg_sub) {
+__device__ __forceinline__ float capped_score_exp(float s, float in_cap, float cap_log2) {
     const float e = ex2(s * in_cap * 2.8853900817779268f);                   // e^2x
     float r;
     asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.0f));
-    const float y = fmaf(r, -2.0f * cap_log2, cap_log2 + neg_sub);
-    return s == -INFINITY ? -INFINITY : y;
+    return fmaf(r, -2.0f * cap_log2, cap_log2);
 }
 
 // 32 consecutive 32-bit columns of this thread's lane into v[OFF .. OFF + 31]
@@ -204,7 +203,7 @@ struct Args {
     const int* req_prior;
     const int* table;
     int n_requests, table_stride, page_tokens, n_heads, n_kv, window;
-    float scale_log2;
+    float scale_log2;          // scores to units of log 2 (1 where the cap has done that)
     float cap_log2, in_cap;    // capped scores: cap log2(e) and scale / cap (the kernel's CAP forms)
     float cap_p[CAP_TERMS];    // CAP_POLY: P's terms with both folded in, a score s becomes s P(s^2) in units of log 2
     float sink_log2;           // score of a key without a value in units of log 2; -infinity: none
@@ -468,8 +467,25 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 tmem_ld32<0>(s_addr + half * HC, v);
                 tmem_ld32<32>(s_addr + half * HC + 32, v);
                 tmem_ld_wait();
-                const bool partial = lo != 0 || span != BN - 1;
-                if (partial) {
+                // The exact forms of the cap turn the raw scores into capped ones where they lie, in units of log 2 (the host
+                // then gives 1 for the scale below): one pass whether or not the softmax pass is repeated.
+                if (CAP > CAP_POLY) {
+                    constexpr int N = CAP > CAP_POLY ? CAP - CAP_POLY : CAP_TERMS;
+#pragma unroll
+                    for (int c = 0; c < HC; c += 2) {
+                        const f32x2 s2 = pack2(__uint_as_float(v[c]), __uint_as_float(v[c + 1])), x2 = mul2(s2, s2);
+                        f32x2 y2 = pack2(p.cap_p[N - 1], p.cap_p[N - 1]);
+#pragma unroll
+                        for (int k = N - 2; k >= 0; --k) y2 = fma2(y2, x2, pack2(p.cap_p[k], p.cap_p[k]));
+                        const float2 t = unpack2(mul2(y2, s2));
+                        v[c] = __float_as_uint(t.x);
+                        v[c + 1] = __float_as_uint(t.y);
+                    }
+                } else if (CAP == CAP_EXP) {
+#pragma unroll
+                    for (int c = 0; c < HC; ++c) v[c] = __float_as_uint(capped_score_exp(__uint_as_float(v[c]), p.in_cap, p.cap_log2));
+                }
+                if (lo != 0 || span != BN - 1) {
 #pragma unroll
                     for (int c = 0; c < HC; ++c)
                         if (!((unsigned)(half * HC + c - lo) <= (unsigned)span && span >= 0)) v[c] = 0xff800000u;       // -inf
@@ -492,32 +508,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
                     for (int c = 0; c < HC; c += 4) {
                         float2 t0, t1;
-                        if (CAP > CAP_POLY) {
-                            constexpr int N = CAP > CAP_POLY ? CAP - CAP_POLY : CAP_TERMS;
-                            const f32x2 s0 = pack2(__uint_as_float(v[c]), __uint_as_float(v[c + 1]));
-                            const f32x2 s1 = pack2(__uint_as_float(v[c + 2]), __uint_as_float(v[c + 3]));
-                            const f32x2 x0 = mul2(s0, s0), x1 = mul2(s1, s1);
-                            f32x2 p0 = pack2(p.cap_p[N - 1], p.cap_p[N - 1]), p1 = p0;
-#pragma unroll
-                            for (int k = N - 2; k >= 0; --k) {
-                                const f32x2 ck = pack2(p.cap_p[k], p.cap_p[k]);
-                                p0 = fma2(p0, x0, ck);
-                                p1 = fma2(p1, x1, ck);
-                            }
-                            t0 = unpack2(fma2(p0, s0, sub2));
-                            t1 = unpack2(fma2(p1, s1, sub2));
-                            if (partial) {                     // a masked score (-inf) stays -inf
-                                t0.x = __uint_as_float(v[c]) == -INFINITY ? -INFINITY : t0.x;
-                                t0.y = __uint_as_float(v[c + 1]) == -INFINITY ? -INFINITY : t0.y;
-                                t1.x = __uint_as_float(v[c + 2]) == -INFINITY ? -INFINITY : t1.x;
-                                t1.y = __uint_as_float(v[c + 3]) == -INFINITY ? -INFINITY : t1.y;
-                            }
-                        } else if (CAP == CAP_EXP) {
-                            t0 = make_float2(capped_score_exp(__uint_as_float(v[c]), p.in_cap, p.cap_log2, neg_sub),
-                                             capped_score_exp(__uint_as_float(v[c + 1]), p.in_cap, p.cap_log2, neg_sub));
-                            t1 = make_float2(capped_score_exp(__uint_as_float(v[c + 2]), p.in_cap, p.cap_log2, neg_sub),
-                                             capped_score_exp(__uint_as_float(v[c + 3]), p.in_cap, p.cap_log2, neg_sub));
-                        } else if (CAP == CAP_APPROX) {
+                        if (CAP == CAP_APPROX) {
                             t0 = make_float2(capped_score(__uint_as_float(v[c]), p.in_cap, p.cap_log2, neg_sub),
                                              capped_score(__uint_as_float(v[c + 1]), p.in_cap, p.cap_log2, neg_sub));
                             t1 = make_float2(capped_score(__uint_as_float(v[c + 2]), p.in_cap, p.cap_log2, neg_sub),
@@ -540,8 +531,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     if (attempt == 1) break;
                     // scale > 0, and capping keeps the order: the largest raw score is the largest score
                     const float mx_raw = fmaxf(mx0, mx1);
-                    const float mx = CAP == CAP_NONE ? mx_raw * p.scale_log2 : CAP == CAP_APPROX ? capped_score(mx_raw, p.in_cap, p.cap_log2, 0.0f)
-                                     : capped_score_exp(mx_raw, p.in_cap, p.cap_log2, 0.0f);       // only a reference for the sums
+                    const float mx = CAP == CAP_APPROX ? capped_score(mx_raw, p.in_cap, p.cap_log2, 0.0f) : mx_raw * p.scale_log2;
                     float m_new = m_ref;
                     if (mx > m_ref + RESCALE_THRESHOLD || m_ref == -INFINITY) m_new = fmaxf(m_ref, mx);
                     if (!__any_sync(0xffffffffu, m_new != m_ref)) break;
@@ -687,6 +677,7 @@ CJ_EXPORT int cj_prefill_attention_tc(const void* q, void* out, const void* kpla
         // cap log2(e) tanh(x), x = s scale / cap: the k-th term carries x^(2k + 1)
         const double x = (double)scale / (double)softcap;
         double f = (double)softcap * 1.4426950408889634 * x;
+        a.scale_log2 = 1.0f;             // the capped scores come out in units of log 2
         for (int k = 0; k < CAP_TERMS; ++k, f *= x * x) a.cap_p[k] = (float)(CAP_P[cap > CAP_POLY ? cap - CAP_POLY - 3 : 0][k] * f);
     }
     // heads run fastest, so that blocks start in the order of their length (the last rows of a
