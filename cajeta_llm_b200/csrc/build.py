@@ -45,6 +45,7 @@ LIBRARIES: Dict[str, str] = {
     "attention_prefill_tc": "attention_prefill_tc.cu",
     "random_fill": "random_fill.cu",
     "recurrent": "recurrent.cu",
+    "decay_attention": "decay_attention.cu",
     "latent_attention": "latent_attention.cu",
     "latent_prefill": "latent_prefill.cu",
     "stream_ops": "stream_ops.cu",

@@ -48,24 +48,34 @@ __device__ __forceinline__ float warp_max(float v) {
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + expf(-x)); }
 
 // The gate of a gated feed-forward, from its two products g (gate) and u (up).  limit == 0:
-// silu(g) * u.  limit > 0, the capped form: g = min(g, limit), u = clamp(u, -limit, limit),
-// g * sigmoid(alpha g) * (u + 1).
-__device__ __forceinline__ float gated_act(float g, float u, float limit, float alpha) {
+// g * sigmoid(alpha g + cubic g^3) * u, which is silu(g) * u for (1, 0) and, because
+// (1 + tanh y) / 2 = sigmoid(2 y), the tanh form of gelu for (2 sqrt(2 / pi), 2 sqrt(2 / pi) 0.044715).
+// limit > 0, the capped form: g = min(g, limit), u = clamp(u, -limit, limit), g * sigmoid(alpha g) * (u + 1).
+__device__ __forceinline__ float gated_act(float g, float u, float limit, float alpha, float cubic) {
     if (limit > 0.0f) {
         g = fminf(g, limit);
         u = fminf(fmaxf(u, -limit), limit);
         return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
     }
-    return silu(g) * u;
+    return g / (1.0f + expf(-g * (alpha + cubic * g * g))) * u;
 }
 // the same with the fast exponential and division, for results that are rounded to bfloat16
-__device__ __forceinline__ float gated_act_fast(float g, float u, float limit, float alpha) {
+__device__ __forceinline__ float gated_act_fast(float g, float u, float limit, float alpha, float cubic) {
     if (limit > 0.0f) {
         g = fminf(g, limit);
         u = fminf(fmaxf(u, -limit), limit);
         return __fdividef(g, 1.0f + __expf(-alpha * g)) * (u + 1.0f);
     }
-    return __fdividef(g, 1.0f + __expf(-g)) * u;
+    return __fdividef(g, 1.0f + __expf(-g * (alpha + cubic * g * g))) * u;
+}
+
+// The activation of a product's result: max(v, 0)^2, v Phi(v) (gelu by the error function) or silu
+constexpr int ACT_NONE = 0, ACT_RELU2 = 1, ACT_GELU = 2, ACT_SILU = 3;
+__device__ __forceinline__ float plain_act(float v, int act) {
+    if (act == ACT_GELU) return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
+    if (act == ACT_SILU) return silu(v);
+    v = fmaxf(v, 0.0f);
+    return v * v;
 }
 
 // Launches overlap their neighbours in the stream (programmatic dependent launch): a kernel

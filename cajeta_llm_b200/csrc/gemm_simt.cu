@@ -7,7 +7,7 @@
 //
 // Variants, all one kernel template:
 //   * plain / accumulate into C (the residual add of an output projection);
-//   * SwiGLU: two weight matrices, C = silu(A.Wg^T) * (A.Wu^T)
+//   * gated: two weight matrices, C = act(A.Wg^T + bg) * (A.Wu^T + bu), act = silu (SwiGLU) or another gated_act takes
 //     (model/Prim.cajeta:1822-1847);
 //   * grouped: rows of A are "sorted slots" of a mixture of experts; group g owns slots
 //     [offsets[g], offsets[g+1]) and its own weight slab W + g * w_group_stride;
@@ -26,6 +26,7 @@ struct GemmArgs {
     const void* A; long long lda;
     const void* W; const void* W2; long long ldw;
     const float* bias;
+    const float* bias2;           // gated form: the second weight's bias (bias is then the first's); both before the activation
     void* C; long long ldc;
     int M, N, K;
     int accumulate;
@@ -33,7 +34,8 @@ struct GemmArgs {
     const int* a_row_index;       // [M] or null
     long long w_group_stride;
     int num_groups;
-    float act_limit, act_alpha;   // the gated form's activation (see gated_act)
+    float act_limit, act_alpha, act_cubic;   // the gated form's activation (see gated_act)
+    int act, act_feats;           // one weight: the activation of the sum (bias included) of the first act_feats features, ACT_NONE for none
     float out_scale;              // multiplies the sum (bias included) before it is stored or added; 1 = as it is
 };
 
@@ -143,8 +145,9 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(GemmArgs p) {
             int c = col_begin + tx * TN + j;
             if (c >= p.N) continue;
             float v = acc[i][j];
-            if (SWIGLU) v = gated_act(v, acc2[i][j], p.act_limit, p.act_alpha);
             if (p.bias) v += p.bias[c];
+            if (SWIGLU) v = gated_act(v, p.bias2 ? acc2[i][j] + p.bias2[c] : acc2[i][j], p.act_limit, p.act_alpha, p.act_cubic);
+            else if (p.act != ACT_NONE && c < p.act_feats) v = plain_act(v, p.act);
             v *= p.out_scale;
             size_t o = (size_t)r * p.ldc + c;
             if (p.accumulate) v += to_f32(C[o]);
@@ -166,15 +169,20 @@ int launch(const GemmArgs& p, bool swiglu, cudaStream_t stream) {
 }  // namespace
 
 // a_dtype / w_dtype / c_dtype: CJ_F32 or CJ_BF16.  Instantiated: (f32,f32,f32),
-// (bf16,bf16,f32), (bf16,bf16,bf16).  w2 non-null selects the SwiGLU form.
+// (bf16,bf16,f32), (bf16,bf16,bf16).  w2 non-null selects the gated form (bias and bias2: its weights' biases);
+// act (ACT_RELU2, ACT_GELU, ACT_SILU): the activation of a product of one weight, applied to the sum and its bias; with
+// act_feats > 0 to the first that many features alone.
 CJ_EXPORT int cj_gemm_simt(const void* A, long long lda, int a_dtype, const void* W, const void* W2, long long ldw,
-                           int w_dtype, const float* bias, void* C, long long ldc, int c_dtype, int M, int N, int K,
+                           int w_dtype, const float* bias, const float* bias2, void* C, long long ldc, int c_dtype, int M, int N, int K,
                            int accumulate, const int* group_offsets, int num_groups, long long w_group_stride,
-                           const int* a_row_index, float act_limit, float act_alpha, float out_scale, cudaStream_t stream) {
+                           const int* a_row_index, float act_limit, float act_alpha, float act_cubic, int act, int act_feats, float out_scale,
+                           cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (!A || !W || !C || K <= 0) return CJ_ERR_ARG;
     if (group_offsets && num_groups <= 0) return CJ_ERR_ARG;
-    GemmArgs p{A, lda, W, W2, ldw, bias, C, ldc, M, N, K, accumulate, group_offsets, a_row_index, w_group_stride, num_groups, act_limit, act_alpha, out_scale};
+    if ((bias2 && !W2) || (act != ACT_NONE && W2)) return CJ_ERR_ARG;
+    GemmArgs p{A, lda, W, W2, ldw, bias, bias2, C, ldc, M, N, K, accumulate, group_offsets, a_row_index, w_group_stride, num_groups,
+               act_limit, act_alpha, act_cubic, act, act_feats > 0 ? act_feats : N, out_scale};
     bool sw = W2 != nullptr;
     if (a_dtype == CJ_F32 && w_dtype == CJ_F32 && c_dtype == CJ_F32) return launch<float, float, float>(p, sw, stream);
     if (a_dtype == CJ_BF16 && w_dtype == CJ_BF16 && c_dtype == CJ_F32) return launch<__nv_bfloat16, __nv_bfloat16, float>(p, sw, stream);

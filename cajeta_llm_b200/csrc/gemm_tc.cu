@@ -41,8 +41,10 @@ constexpr int UMMA_K = 16;         // K of one tcgen05.mma of kind::f16
 constexpr int THREADS = 224;          // warps 0 and 6: loads; warp 1: products; warps 2-5: epilogue
 constexpr int LOADERS = 2;
 
-// EPI_RELU2_BF16: max(v, 0)^2 of the float32 sum (bias included), rounded to bfloat16: an expert without a gate
-enum Epilogue { EPI_STORE_F32 = 0, EPI_ACC_F32 = 1, EPI_SWIGLU_BF16 = 2, EPI_STORE_BF16 = 3, EPI_RELU2_BF16 = 4 };
+// EPI_ACT_BF16: Args::act (max(v, 0)^2, gelu or silu) of the float32 sum (bias included), rounded to bfloat16: an expert without a gate.
+// Callers name it EPI_RELU2_BF16, EPI_GELU_BF16 or EPI_SILU_BF16; one kernel serves all.
+enum Epilogue { EPI_STORE_F32 = 0, EPI_ACC_F32 = 1, EPI_SWIGLU_BF16 = 2, EPI_STORE_BF16 = 3, EPI_ACT_BF16 = 4 };
+constexpr int EPI_RELU2_BF16 = 4, EPI_GELU_BF16 = 5, EPI_SILU_BF16 = 6;
 
 struct Args {
     int tokens;                 // rows of X
@@ -51,12 +53,14 @@ struct Args {
     void* out;
     long long ldo;              // elements between output rows (tokens)
     const float* bias;          // [features] or null
+    const float* bias2;         // gated form: the second weight's bias (bias is the first's), both before the activation
     const int* group_offsets;   // [groups + 1] or null
     int groups;
     int k_splits;               // > 1: each split stores its partial at out + split * split_stride
     long long split_stride;
     int offsets_settled;        // the groups' offsets were complete before the kernel before this one began
-    float act_limit, act_alpha; // the gated form's activation (see gated_act)
+    float act_limit, act_alpha, act_cubic; // the gated form's activation (see gated_act)
+    int act, act_feats;         // EPI_ACT_BF16's activation (see plain_act), of the first act_feats features
     float out_scale;            // float32 store / accumulate: multiplies the sum (bias included); 1 = as it is
     int choose_height;          // grouped, weights on the rows: the tile's height is chosen in the kernel (see LowTiles)
 };
@@ -352,7 +356,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
             tcgen05_fence_after();
             const uint32_t lane_base = tmem_base + as * STAGE_COLS + ((uint32_t)(quarter * 32) << 16);
             const long long split_off = (long long)c.split * p.split_stride;
-            const bool add_bias = p.bias != nullptr && c.split == 0;
+            const bool add_bias = p.bias != nullptr && c.split == 0 && EPI != EPI_SWIGLU_BF16;
+            // the gated form's biases: with the weights on the rows this thread has one feature, else they are read by column
+            float bg = 0.0f, bu = 0.0f;
+            if (EPI == EPI_SWIGLU_BF16 && SWAP && c.feat0 + r < p.features) {
+                if (p.bias) bg = p.bias[c.feat0 + r];
+                if (p.bias2) bu = p.bias2[c.feat0 + r];
+            }
 #pragma unroll 1
             for (int c0 = 0; c0 < N_MMA; c0 += 16) {
                 if (SWAP && c.tok0 + c0 >= c.tok_end) break;           // no token left in these columns
@@ -370,7 +380,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
                 for (int j = 0; j < 16; ++j) {
                     v[j] = __uint_as_float(v0[j]);
                     // the result is rounded to bfloat16 (8 bits): the fast exponential and division (2 ulp of float32) do not show
-                    if (EPI == EPI_SWIGLU_BF16) v[j] = cj::gated_act_fast(v[j], __uint_as_float(v1[j]), p.act_limit, p.act_alpha);
+                    if (EPI == EPI_SWIGLU_BF16) {
+                        if (!SWAP) {
+                            const int f = min(c.feat0 + c0 + j, p.features - 1);
+                            bg = p.bias ? p.bias[f] : 0.0f;
+                            bu = p.bias2 ? p.bias2[f] : 0.0f;
+                        }
+                        v[j] = cj::gated_act_fast(v[j] + bg, __uint_as_float(v1[j]) + bu, p.act_limit, p.act_alpha, p.act_cubic);
+                    }
                 }
                 if (!SWAP) {
                     // this thread owns one token row and 16 consecutive features of it
@@ -382,9 +399,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
 #pragma unroll
                         for (int j = 0; j < 16; ++j) if (whole || feat + j < p.features) v[j] += p.bias[feat + j];
                     }
-                    if (EPI == EPI_RELU2_BF16) {
+                    if (EPI == EPI_ACT_BF16) {
 #pragma unroll
-                        for (int j = 0; j < 16; ++j) { const float t = fmaxf(v[j], 0.0f); v[j] = t * t; }
+                        for (int j = 0; j < 16; ++j) if (feat + j < p.act_feats) v[j] = cj::plain_act(v[j], p.act);
                     }
                     if (EPI == EPI_STORE_F32 || EPI == EPI_ACC_F32) {
 #pragma unroll
@@ -434,7 +451,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
                         if (token >= c.tok_end) break;
                         long long o = (long long)token * p.ldo + feat;
                         float val = v[j] + b;
-                        if (EPI == EPI_RELU2_BF16) { val = fmaxf(val, 0.0f); val *= val; }
+                        if (EPI == EPI_ACT_BF16 && feat < p.act_feats) val = cj::plain_act(val, p.act);
                         if (EPI == EPI_STORE_F32 || EPI == EPI_ACC_F32) val *= p.out_scale;
                         if (EPI == EPI_STORE_F32) ((float*)p.out)[o + split_off] = val;
                         else if (EPI == EPI_ACC_F32) ((float*)p.out)[o] += val;
@@ -540,21 +557,24 @@ int dispatch_n(int n_mma, const CUtensorMap& mx, const CUtensorMap& mw, const CU
 // x: [tokens, K] bf16 with row stride ldx; w (and w2 for SwiGLU): [groups * features, K] bf16,
 // contiguous.  swap: 0 = tokens on the product's rows (tile 128 tokens x n_mma features),
 // 1 = weights on the rows (tile 128 features x n_mma tokens).  epilogue: 0 float32 store,
-// 1 float32 accumulate, 2 SwiGLU to bf16 (needs w2), 3 bf16 store (0 and 1: out_scale multiplies the sum).  k_splits > 1 only with
+// 1 float32 accumulate, 2 gated to bf16 (needs w2; bias and bias2 are its weights'; SwiGLU, or what gated_act takes), 3 bf16 store,
+// 4 squared ReLU, 5 gelu (by the error function) and 6 silu of the sum to bf16, with act_feats > 0 of the first that many
+// features alone (0 and 1: out_scale multiplies the sum).  k_splits > 1 only with
 // epilogue 0: split s stores its partial sum at out + s * split_stride (the bias goes to
 // split 0).  offsets_settled: non-zero if group_offsets were complete before the kernel
 // before this launch began (not merely before this launch): the kernel then reads them, and
 // sends for its first weight tiles, while that kernel is still draining.  Refuses (negative
 // code) what it cannot run; never a wrong result.
-CJ_EXPORT int cj_gemm_tc(const void* x, long long ldx, const void* w, const void* w2, const float* bias, void* out,
+CJ_EXPORT int cj_gemm_tc(const void* x, long long ldx, const void* w, const void* w2, const float* bias, const float* bias2, void* out,
                          long long ldo, int tokens, int features, int K, int epilogue, int swap, int n_mma,
                          const int* group_offsets, int groups, int k_splits, long long split_stride,
-                         int offsets_settled, float act_limit, float act_alpha, float out_scale, cudaStream_t stream) {
+                         int offsets_settled, float act_limit, float act_alpha, float act_cubic, int act_feats, float out_scale,
+                         cudaStream_t stream) {
     if (tokens <= 0 || features <= 0) return 0;
     if (!x || !w || !out || K <= 0) return CJ_ERR_ARG;
     if (K % 8 != 0 || ldx % 8 != 0) return CJ_ERR_ALIGN;               // TMA: 16-byte strides
     if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)w2) & 15) return CJ_ERR_ALIGN;
-    if ((epilogue == EPI_SWIGLU_BF16) != (w2 != nullptr)) return CJ_ERR_ARG;
+    if ((epilogue == EPI_SWIGLU_BF16) != (w2 != nullptr) || (bias2 && !w2)) return CJ_ERR_ARG;
     if (k_splits < 1 || (k_splits > 1 && epilogue != EPI_STORE_F32)) return CJ_ERR_ARG;
     if (group_offsets && groups <= 0) return CJ_ERR_ARG;
     int total_w_rows = (group_offsets ? groups : 1) * features;
@@ -575,7 +595,9 @@ CJ_EXPORT int cj_gemm_tc(const void* x, long long ldx, const void* w, const void
             if (w2 && !make_map_bf16(&low.w2[i], w2, total_w_rows, K, K, low_height(i))) return CJ_ERR_ARG;
         }
     }
-    Args a{tokens, features, K, out, ldo, bias, group_offsets, groups, k_splits, split_stride, offsets_settled, act_limit, act_alpha, out_scale, choose_height};
+    const int act = epilogue == EPI_GELU_BF16 ? cj::ACT_GELU : epilogue == EPI_SILU_BF16 ? cj::ACT_SILU : cj::ACT_RELU2;
+    Args a{tokens, features, K, out, ldo, bias, bias2, group_offsets, groups, k_splits, split_stride, offsets_settled, act_limit, act_alpha,
+           act_cubic, act, act_feats > 0 ? act_feats : features, out_scale, choose_height};
 #define CASE(EPI, DUAL)                                                                              \
     if (swap) return dispatch_n<true, DUAL, EPI>(n_mma, mx, mw, mw2, low, a, stream);                 \
     else return dispatch_n<false, DUAL, EPI>(n_mma, mx, mw, mw2, low, a, stream);
@@ -584,7 +606,9 @@ CJ_EXPORT int cj_gemm_tc(const void* x, long long ldx, const void* w, const void
         case EPI_ACC_F32: CASE(EPI_ACC_F32, false)
         case EPI_SWIGLU_BF16: CASE(EPI_SWIGLU_BF16, true)
         case EPI_STORE_BF16: CASE(EPI_STORE_BF16, false)
-        case EPI_RELU2_BF16: CASE(EPI_RELU2_BF16, false)
+        case EPI_RELU2_BF16:
+        case EPI_GELU_BF16:
+        case EPI_SILU_BF16: CASE(EPI_ACT_BF16, false)
     }
 #undef CASE
     return CJ_ERR_ARG;

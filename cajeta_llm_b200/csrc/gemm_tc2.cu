@@ -47,16 +47,19 @@ constexpr int FEAT_TILE = 256;      // feature rows a pair of blocks covers
 constexpr int MAX_GROUPS = 1024;
 constexpr int MAX_ACC_STAGES = 2;
 
-enum Epilogue { EPI_STORE_F32 = 0, EPI_ACC_F32 = 1, EPI_SWIGLU_BF16 = 2, EPI_STORE_BF16 = 3, EPI_RELU2_BF16 = 4 };
+enum Epilogue { EPI_STORE_F32 = 0, EPI_ACC_F32 = 1, EPI_SWIGLU_BF16 = 2, EPI_STORE_BF16 = 3, EPI_ACT_BF16 = 4 };
+constexpr int EPI_RELU2_BF16 = 4, EPI_GELU_BF16 = 5, EPI_SILU_BF16 = 6;      // they run as EPI_ACT_BF16 with Args::act
 
 struct Args {
     int tokens, features, K;
     void* out;
     long long ldo;
     const float* bias;
+    const float* bias2;          // gated form: the second weight's bias (bias is the first's), both before the activation
     const int* group_offsets;
     int groups;
-    float act_limit, act_alpha;  // the gated form's activation (see gated_act)
+    float act_limit, act_alpha, act_cubic;  // the gated form's activation (see gated_act)
+    int act, act_feats;          // EPI_ACT_BF16's activation (see plain_act), of the first act_feats features
     float out_scale;             // float32 store / accumulate: multiplies the sum (bias included); 1 = as it is
 };
 
@@ -269,7 +272,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant
                         for (int j = 0; j < 32; ++j) {
                             if (c0 + j >= n_cols) break;
                             float val = __uint_as_float(v[j]) + b;
-                            if (EPI == EPI_RELU2_BF16) { val = fmaxf(val, 0.0f); val *= val; }       // an expert without a gate
+                            if (EPI == EPI_ACT_BF16 && feat < p.act_feats) val = cj::plain_act(val, p.act);       // an expert without a gate
                             if (EPI == EPI_STORE_F32) ((float*)p.out)[o0 + j * p.ldo] = val * p.out_scale;
                             else ((__nv_bfloat16*)p.out)[o0 + j * p.ldo] = __float2bfloat16_rn(val);
                         }
@@ -447,8 +450,10 @@ swiglu_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_const
                     float v[16];
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
-                        float gv = __uint_as_float(g[j]);
-                        v[j] = cj::gated_act_fast(gv, __uint_as_float(u[j]), p.act_limit, p.act_alpha);
+                        const int f = min(c.feat0 + c0 + j, p.features - 1);
+                        const float gv = __uint_as_float(g[j]) + (p.bias ? p.bias[f] : 0.0f);
+                        const float uv = __uint_as_float(u[j]) + (p.bias2 ? p.bias2[f] : 0.0f);
+                        v[j] = cj::gated_act_fast(gv, uv, p.act_limit, p.act_alpha, p.act_cubic);
                     }
                     __nv_bfloat16* dst = dst_row + c0;
                     if (c.feat0 + c0 + 16 <= p.features && (((uintptr_t)dst) & 15) == 0) {
@@ -559,24 +564,27 @@ int launch_swiglu(const CUtensorMap& mx, const CUtensorMap& mwg, const CUtensorM
 
 // x: [tokens, K] bf16 with row stride ldx; w (and w2 for SwiGLU): [groups * features, K] bf16,
 // contiguous.  n_tok: tokens a tile covers, 128 or 256 (SwiGLU: always 256).  epilogue: 0 float32
-// store, 1 float32 accumulate, 2 SwiGLU to bf16 (needs w2), 3 bf16 store.
+// store, 1 float32 accumulate, 2 gated to bf16 (needs w2; bias and bias2 are its weights'), 3 bf16 store, 4 squared ReLU, 5 gelu
+// (by the error function) and 6 silu of the sum to bf16, with act_feats > 0 of the first that many features alone.
 // Refuses (negative code) what it cannot run; never a wrong result.
-CJ_EXPORT int cj_gemm_tc2(const void* x, long long ldx, const void* w, const void* w2, const float* bias, void* out,
+CJ_EXPORT int cj_gemm_tc2(const void* x, long long ldx, const void* w, const void* w2, const float* bias, const float* bias2, void* out,
                           long long ldo, int tokens, int features, int K, int epilogue, int n_tok,
-                          const int* group_offsets, int groups, float act_limit, float act_alpha, float out_scale, cudaStream_t stream) {
+                          const int* group_offsets, int groups, float act_limit, float act_alpha, float act_cubic, int act_feats, float out_scale,
+                          cudaStream_t stream) {
     if (tokens <= 0 || features <= 0) return 0;
     if (!x || !w || !out || K <= 0) return CJ_ERR_ARG;
     if (K % 8 != 0 || ldx % 8 != 0) return CJ_ERR_ALIGN;
     if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)w2) & 15) return CJ_ERR_ALIGN;
-    if ((epilogue == EPI_SWIGLU_BF16) != (w2 != nullptr)) return CJ_ERR_ARG;
-    if (epilogue == EPI_SWIGLU_BF16 && bias) return CJ_ERR_ARG;
+    if ((epilogue == EPI_SWIGLU_BF16) != (w2 != nullptr) || (bias2 && !w2)) return CJ_ERR_ARG;
     if (group_offsets && groups <= 0) return CJ_ERR_ARG;
     if (n_tok != 128 && n_tok != 256) return CJ_ERR_SIZE;
     if (group_offsets && groups > MAX_GROUPS) return CJ_ERR_SIZE;
     int total_w_rows = (group_offsets ? groups : 1) * features;
     CUtensorMap mx, mw, mw2;
     if (!make_map_bf16(&mw, w, total_w_rows, K, K, 128)) return CJ_ERR_ARG;
-    Args a{tokens, features, K, out, ldo, bias, group_offsets, groups, act_limit, act_alpha, out_scale};
+    const int act = epilogue == EPI_GELU_BF16 ? cj::ACT_GELU : epilogue == EPI_SILU_BF16 ? cj::ACT_SILU : cj::ACT_RELU2;
+    Args a{tokens, features, K, out, ldo, bias, bias2, group_offsets, groups, act_limit, act_alpha, act_cubic, act,
+           act_feats > 0 ? act_feats : features, out_scale};
     if (epilogue == EPI_SWIGLU_BF16) {
         // tokens on the rows: a block's box is 128 token rows whatever n_tok says
         if (!make_map_bf16(&mx, x, tokens, K, ldx, 128)) return CJ_ERR_ARG;
@@ -591,7 +599,9 @@ CJ_EXPORT int cj_gemm_tc2(const void* x, long long ldx, const void* w, const voi
         case EPI_STORE_F32: CASE(EPI_STORE_F32)
         case EPI_ACC_F32: CASE(EPI_ACC_F32)
         case EPI_STORE_BF16: CASE(EPI_STORE_BF16)
-        case EPI_RELU2_BF16: CASE(EPI_RELU2_BF16)
+        case EPI_RELU2_BF16:
+        case EPI_GELU_BF16:
+        case EPI_SILU_BF16: CASE(EPI_ACT_BF16)
     }
 #undef CASE
     return CJ_ERR_ARG;

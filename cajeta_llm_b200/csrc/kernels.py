@@ -7,6 +7,7 @@ no fallback: without a CUDA device and the built libraries these functions raise
 from __future__ import annotations
 
 import ctypes
+import math
 import os
 from typing import Dict, Optional
 
@@ -246,14 +247,37 @@ def dyt_add(hs: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, bias: torch
     _check(library("rowwise").cj_dyt_add(_ptr(hs), _ptr(y), _ptr(weight), _ptr(bias), _f(alpha), _i(rows), _i(H), _stream()), "dyt_add")
 
 
+# (act_alpha, act_cubic) of gelu's tanh form as a gate: g sigmoid(alpha g + cubic g^3)
+GELU_TANH = (2.0 * math.sqrt(2.0 / math.pi), 2.0 * math.sqrt(2.0 / math.pi) * 0.044715)
+ACTS = {"": 0, "relu2": 1, "gelu": 2, "silu": 3}        # activations of a product of one weight (gelu: by the error function)
+
+
+def _gate_biases(w: torch.Tensor, w_up: Optional[torch.Tensor], bias: Optional[torch.Tensor], bias_up: Optional[torch.Tensor],
+                 act: str) -> None:
+    for n, t in (("bias", bias), ("bias_up", bias_up)):
+        if t is not None:
+            _need(t, n, torch.float32)
+            if t.numel() != w.shape[-2]:
+                raise KernelError(f"{n} must hold {w.shape[-2]} entries, found {t.numel()}")
+    if bias_up is not None and w_up is None:
+        raise KernelError("bias_up goes with w_up")
+    if act not in ACTS or (act and w_up is not None):
+        raise KernelError(f"act must be one of {sorted(ACTS)} and goes with one weight, found '{act}'")
+
+
 def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
          accumulate: bool = False, w_up: Optional[torch.Tensor] = None, group_offsets: Optional[torch.Tensor] = None,
          a_row_index: Optional[torch.Tensor] = None, rows: Optional[int] = None, act_limit: float = 0.0,
-         act_alpha: float = 1.0, out_scale: float = 1.0) -> None:
+         act_alpha: float = 1.0, out_scale: float = 1.0, act_cubic: float = 0.0, bias_up: Optional[torch.Tensor] = None,
+         act: str = "", act_features: int = 0) -> None:
     """out[M, N] (+)= out_scale (a[M, K] . w[N, K]^T (+ bias)) on the float32 FMA pipe.
 
     ``w_up`` selects the gated form: silu(a.w^T) * (a.w_up^T), or with ``act_limit`` > 0 the capped one,
-    g = min(a.w^T, limit), u = clamp(a.w_up^T, +-limit), g * sigmoid(act_alpha g) * (u + 1).  With ``group_offsets``
+    g = min(a.w^T, limit), u = clamp(a.w_up^T, +-limit), g * sigmoid(act_alpha g) * (u + 1); without a limit
+    g * sigmoid(act_alpha g + act_cubic g^3) * u (GELU_TANH gives the two numbers of gelu's tanh form).  ``bias`` and ``bias_up``
+    are added to the two sums first.  ``act`` ("relu2", "gelu" or "silu"): the activation of a product of one weight, after its bias
+    (``act_features`` > 0: of its first that many features alone).
+    With ``group_offsets``
     ([G + 1] int32) ``w`` is [G, N, K], output row s belongs to the group whose range
     holds s, and ``a_row_index[s]`` names the row of ``a`` that feeds it.
     """
@@ -269,8 +293,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[tor
         _need(w_up, "w_up")
         if w_up.shape != w.shape or w_up.dtype != w.dtype:
             raise KernelError("gemm: w_up must match w")
-    if bias is not None:
-        _need(bias, "bias", torch.float32)
+    _gate_biases(w, w_up, bias, bias_up, act)
     G = 0
     if grouped:
         _need(group_offsets, "group_offsets", torch.int32)
@@ -280,9 +303,10 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[tor
     if a_row_index is not None:
         _need(a_row_index, "a_row_index", torch.int32)
     st = library("gemm_simt").cj_gemm_simt(
-        _ptr(a), _ll(a.stride(0)), _i(_code(a)), _ptr(w), _ptr(w_up), _ll(K), _i(_code(w)), _ptr(bias),
+        _ptr(a), _ll(a.stride(0)), _i(_code(a)), _ptr(w), _ptr(w_up), _ll(K), _i(_code(w)), _ptr(bias), _ptr(bias_up),
         _ptr(out), _ll(out.stride(0)), _i(_code(out)), _i(M), _i(N), _i(K), _i(1 if accumulate else 0),
-        _ptr(group_offsets), _i(G), _ll(N * K), _ptr(a_row_index), _f(act_limit), _f(act_alpha), _f(out_scale), _stream())
+        _ptr(group_offsets), _i(G), _ll(N * K), _ptr(a_row_index), _f(act_limit), _f(act_alpha), _f(act_cubic), _i(ACTS[act]), _i(act_features),
+        _f(out_scale), _stream())
     _check(st, "gemm")
 
 
@@ -510,10 +534,11 @@ def mixed_heads_attention(q: torch.Tensor, out: torch.Tensor, k_plane: torch.Ten
     _check(st, "mixed_heads_attention")
 
 
-def _route_mode(norm_topk: bool, sigmoid_scores: bool, groups) -> int:
-    """The selection's mode word: bit 0 renormalise the picked scores, bit 1 sigmoid scores, bits 4-15 the
-    number of expert groups and bits 16-27 how many of them stay eligible (``groups`` = (count, keep))."""
-    mode = (1 if norm_topk else 0) | (2 if sigmoid_scores else 0)
+def _route_mode(norm_topk: bool, sigmoid_scores: bool, groups, group_top2: bool = False) -> int:
+    """The selection's mode word: bit 0 renormalise the picked scores, bit 1 sigmoid scores, bit 2 a group's score is the
+    sum of its two largest, bits 4-15 the number of expert groups and bits 16-27 how many of them stay eligible
+    (``groups`` = (count, keep))."""
+    mode = (1 if norm_topk else 0) | (2 if sigmoid_scores else 0) | (4 if group_top2 else 0)
     if groups is not None and int(groups[0]) > 1:
         count, keep = int(groups[0]), int(groups[1])
         if not (1 <= keep <= count <= 0xfff):
@@ -545,13 +570,15 @@ def _correction(correction: Optional[torch.Tensor], num_experts: int, groups) ->
 def router_topk(x: torch.Tensor, router_w: torch.Tensor, shared_gate: Optional[torch.Tensor], top_k: int,
                 norm_topk: bool, sel: torch.Tensor, weights: torch.Tensor, shared_scale: Optional[torch.Tensor],
                 pin: Optional[torch.Tensor] = None, gap: Optional[torch.Tensor] = None, sigmoid_scores: bool = False,
-                groups=None, correction: Optional[torch.Tensor] = None, weight_scale: float = 1.0) -> None:
+                groups=None, correction: Optional[torch.Tensor] = None, weight_scale: float = 1.0, group_top2: bool = False,
+                norm_floor: float = 0.0) -> None:
     """Router logits, softmax over all experts (or, with ``sigmoid_scores``, each expert's own
     sigmoid), top-k and the shared expert's sigmoid gate.
     ``pin`` (int32 [T, k]): the experts are given, not chosen; the weights are still the row's own
     probabilities of them.  ``gap`` (float32 [T], not with ``pin``): each row's routing margin
     (p_k - p_{k+1}) / p_k out.  ``groups`` = (count, keep): the experts form ``count`` equal groups of
-    neighbours and only those of the ``keep`` groups with the largest best score can be picked.
+    neighbours and only those of the ``keep`` groups with the largest best score (``group_top2``: with the largest sum of
+    their two best) can be picked.  ``norm_floor`` > 0: a renormalisation divides by the picks' sum plus it.
     ``correction`` (float32 [E]): added to the scores for the choice alone, a pick's weight stays its score;
     ``weight_scale`` multiplies the picks' weights."""
     _need(x, "x", torch.float32), _need(router_w, "router_w", torch.float32)
@@ -571,9 +598,9 @@ def router_topk(x: torch.Tensor, router_w: torch.Tensor, shared_gate: Optional[t
     if tickets is None:
         tickets = _router_tickets[x.device] = torch.zeros((4,), dtype=torch.int32, device=x.device)
     st = library("moe_route").cj_router_topk(_ptr(x), _ptr(router_w), _ptr(shared_gate), _i(T), _i(H), _i(E), _i(top_k),
-                                             _i(_route_mode(norm_topk, sigmoid_scores, groups)), _ptr(sel), _ptr(weights),
+                                             _i(_route_mode(norm_topk, sigmoid_scores, groups, group_top2)), _ptr(sel), _ptr(weights),
                                              _ptr(shared_scale), _ptr(logits), _ptr(tickets), _ptr(pin), _ptr(gap),
-                                             _ptr(correction), _f(weight_scale), _stream())
+                                             _ptr(correction), _f(weight_scale), _f(norm_floor), _stream())
     _check(st, "router_topk")
     if T > 32:
         global launches
@@ -583,7 +610,8 @@ def router_topk(x: torch.Tensor, router_w: torch.Tensor, shared_gate: Optional[t
 def router_select(partials: torch.Tensor, num_experts: int, top_k: int, norm_topk: bool, sel: torch.Tensor,
                   weights: torch.Tensor, shared_scale: Optional[torch.Tensor], pin: Optional[torch.Tensor] = None,
                   gap: Optional[torch.Tensor] = None, sigmoid_scores: bool = False, groups=None,
-                  correction: Optional[torch.Tensor] = None, weight_scale: float = 1.0) -> None:
+                  correction: Optional[torch.Tensor] = None, weight_scale: float = 1.0, group_top2: bool = False,
+                  norm_floor: float = 0.0) -> None:
     """Softmax over all experts, top-k and the shared gate's sigmoid from router logits given
     as partial sums ``[S, T, ld]`` (float32; column ``num_experts`` holds the gate's dot when
     ``shared_scale`` is given); the partials of a row are added in order first."""
@@ -598,9 +626,9 @@ def router_select(partials: torch.Tensor, num_experts: int, top_k: int, norm_top
     if shared_scale is not None:
         _need(shared_scale, "shared_scale", torch.float32)
     st = library("moe_route").cj_router_select(_ptr(partials), _i(S), _ll(partials.stride(0)), _i(ld), _i(T), _i(num_experts),
-                                               _i(top_k), _i(_route_mode(norm_topk, sigmoid_scores, groups)), _ptr(sel),
+                                               _i(top_k), _i(_route_mode(norm_topk, sigmoid_scores, groups, group_top2)), _ptr(sel),
                                                _ptr(weights), _ptr(shared_scale), _ptr(pin), _ptr(gap), _ptr(correction),
-                                               _f(weight_scale), _stream())
+                                               _f(weight_scale), _f(norm_floor), _stream())
     _check(st, "router_select")
 
 
@@ -884,32 +912,95 @@ def rmsnorm_mix2(a: torch.Tensor, wa: torch.Tensor, b: torch.Tensor, wb: torch.T
     _check(st, "rmsnorm_mix2")
 
 
-def relu2_rows(x: torch.Tensor, out: torch.Tensor) -> None:
-    """out = max(x, 0)^2 in out's dtype; x float32."""
-    _need(x, "x", torch.float32), _need(out, "out")
-    if out.numel() != x.numel():
-        raise KernelError("relu2_rows: sizes differ")
-    _check(library("recurrent").cj_relu2_rows(_ptr(x), _ptr(out), _i(_code(out)), _ll(x.numel()), _stream()), "relu2_rows")
-
-
 def softcap_rows(x: torch.Tensor, cap: float) -> None:
     """x <- cap tanh(x / cap) in place; x float32."""
     _need(x, "x", torch.float32)
     _check(library("recurrent").cj_softcap_rows(_ptr(x), _f(cap), _ll(x.numel()), _stream()), "softcap_rows")
 
 
+# -- linear attention with a constant decay per head -----------------------------------------------------
+DECAY_WALK_ROWS = 32         # requests of a step with at most this many rows are walked token by token
+DECAY_CHUNK = 64             # tokens the tensor-core form takes at a time
+
+
+def decay_chunk_shape(dim: int, vdim: int) -> bool:
+    """Whether the tensor-core form of :func:`decay_attention` takes these sizes."""
+    return 0 < dim <= 128 and dim % 8 == 0 and vdim > 0 and vdim % 8 == 0
+
+
+def decay_segment(rows: int, heads: int, vdim: int) -> int:
+    """Tokens of a segment: as many segments of ``rows`` as give every SM a block, at least two chunks each."""
+    blocks = heads * (1 if vdim <= 64 else -(-vdim // 128))
+    want = max(1, -(-_sm_count() // blocks))
+    return max(2 * DECAY_CHUNK, -(-(-(-rows // want)) // DECAY_CHUNK) * DECAY_CHUNK)
+
+
+def decay_attention(x: torch.Tensor, off_q: int, off_k: int, off_v: int, decay: torch.Tensor, powers: torch.Tensor,
+                    log2_decay: torch.Tensor, state: torch.Tensor, state_offset: int, req_start: torch.Tensor, req_slot: torch.Tensor,
+                    requests: int, out: torch.Tensor, heads: int, dim: int, vdim: int, single: bool = False,
+                    segment: int = 0, chunked: Optional[bool] = None) -> None:
+    """Every request's rows of the step in order through its states: per head S = decay S + k v^T, out = S^T q.  x [T, ld]: q, k, v
+    at columns off_q, off_k (heads * dim) and off_v (heads * vdim); ``state[slot, state_offset:]``: heads * dim * vdim float32;
+    out float32 [T, heads * vdim].  ``decay`` float32 [heads], ``powers`` float32 [heads, 65] (decay^0 .. decay^64) and
+    ``log2_decay`` float64 [heads].  ``single``: every request of the step brings one token.  bfloat16 rows of requests with more
+    than ``DECAY_WALK_ROWS`` rows run on the tensor cores where the sizes allow it (``segment``: tokens of a segment instead
+    of the number that fills the machine; ``chunked`` false: walk everything)."""
+    _need(x, "x"), _need(decay, "decay", torch.float32), _need(state, "state", torch.float32), _need(out, "out", torch.float32)
+    _need(powers, "powers", torch.float32), _need(log2_decay, "log2_decay", torch.float64)
+    _need(req_start, "req_start", torch.int32), _need(req_slot, "req_slot", torch.int32)
+    T = x.shape[0]
+    need = heads * dim * vdim
+    if (tuple(out.shape) != (T, heads * vdim) or state[0].numel() < state_offset + need or decay.numel() != heads
+            or powers.numel() != heads * (DECAY_CHUNK + 1) or log2_decay.numel() != heads
+            or max(max(off_q, off_k) + heads * dim, off_v + heads * vdim) > x.shape[1]):
+        raise KernelError("decay_attention: sizes do not agree")
+    st_ptr = ctypes.c_void_p(state.data_ptr() + 4 * state_offset)
+    if chunked is None:
+        chunked = (x.dtype == torch.bfloat16 and decay_chunk_shape(dim, vdim) and not single and T > DECAY_WALK_ROWS
+                   and (x.stride(0) | off_q | off_k | off_v) % 8 == 0 and x.data_ptr() % 16 == 0)
+    lib = library("decay_attention")
+    # (a step's shape alone decides what is launched: which requests the two forms take is found on the device)
+    st = lib.cj_decay_walk(_ptr(x), _i(_code(x)), _i(x.stride(0)), _i(off_q), _i(off_k), _i(off_v), _ptr(decay), st_ptr, _ll(state.stride(0)),
+                           _ptr(req_start), _ptr(req_slot), _i(requests), _ptr(out), _i(heads), _i(dim), _i(vdim),
+                           _i(DECAY_WALK_ROWS if chunked else 0), _stream())
+    _check(st, "decay_attention (walk)")
+    if not chunked:
+        return
+    seg = segment or decay_segment(T, heads, vdim)
+    segments = T // seg + requests
+    added = torch.empty((segments, heads, dim, vdim), dtype=torch.float32, device=x.device) if T > seg else None
+    st = lib.cj_decay_chunk(_ptr(x), _i(x.stride(0)), _i(off_q), _i(off_k), _i(off_v), _ptr(powers), _ptr(log2_decay), st_ptr,
+                            _ll(state.stride(0)), _ptr(req_start), _ptr(req_slot), _i(requests), _ptr(out), _ptr(added), _i(segments),
+                            _i(heads), _i(dim), _i(vdim), _i(seg), _i(DECAY_WALK_ROWS), _stream())
+    _check(st, "decay_attention (chunks)")
+    if added is not None:
+        global launches
+        launches += 1                  # what the segments add is a kernel of its own
+
+
+def gated_row_norm(y: torch.Tensor, z: torch.Tensor, z_offset: int, weight: torch.Tensor, eps: float, out: torch.Tensor) -> None:
+    """out[r] = y[r] / rms(y[r]) * weight * sigmoid(z[r, z_offset:]); y float32 [T, n], z and out in one dtype."""
+    _need(y, "y", torch.float32), _need(z, "z"), _need(weight, "weight", torch.float32), _need(out, "out", z.dtype)
+    T, n = y.shape
+    if out.shape != y.shape or z.shape[1] < z_offset + n or weight.numel() != n:
+        raise KernelError("gated_row_norm: sizes do not agree")
+    st = library("decay_attention").cj_gated_row_norm(_ptr(y), _i(n), ctypes.c_void_p(z.data_ptr() + z.element_size() * z_offset), _i(_code(z)),
+                                                      _i(z.stride(0)), _ptr(weight), _f(eps), _ptr(out), _i(_code(out)), _i(T), _stream())
+    _check(st, "gated_row_norm")
+
+
 # -- attention over a compressed latent ---------------------------------------------------------------
 def latent_kv_write(d: torch.Tensor, d_offset: int, rank: int, rot: int, rotary: int, weight: torch.Tensor, eps: float, inv_freq: Optional[torch.Tensor],
                     positions: torch.Tensor, row_req: torch.Tensor, table: torch.Tensor, page_tokens: int,
-                    plane: torch.Tensor) -> None:
+                    plane: torch.Tensor, halves: bool = False, magnitude: float = 1.0) -> None:
     """Columns [d_offset, d_offset + rank + rot) of d (float32): the RMS-normed latent (times weight) and
-    the key part, its first ``rotary`` entries rotated in pairs (2i, 2i+1), go to the row's place in
-    the paged cache (entries of rank + rot)."""
+    the key part, its first ``rotary`` entries rotated in pairs (2i, 2i+1), or (i, i + rotary/2) when ``halves``, cos and
+    sin times ``magnitude``, go to the row's place in the paged cache (entries of rank + rot)."""
     _need(d, "d", torch.float32), _need(weight, "weight", torch.float32), _need(plane, "plane")
     _need(positions, "positions", torch.int32), _need(row_req, "row_req", torch.int32), _need(table, "table", torch.int32)
     if d.shape[1] < d_offset + rank + rot or plane.shape[-1] != rank + rot:
         raise KernelError("latent_kv_write: sizes do not agree")
-    st = library("latent_attention").cj_latent_kv_write(ctypes.c_void_p(d.data_ptr() + 4 * d_offset), _i(d.stride(0)), _i(rank), _i(rot), _i(rotary), _ptr(weight), _f(eps),
+    st = library("latent_attention").cj_latent_kv_write(ctypes.c_void_p(d.data_ptr() + 4 * d_offset), _i(d.stride(0)), _i(rank), _i(rot), _i(rotary), _i(1 if halves else 0), _f(magnitude), _ptr(weight), _f(eps),
                                                         _ptr(inv_freq), _ptr(positions), _ptr(row_req), _ptr(table),
                                                         _i(table.stride(0)), _i(page_tokens), _ptr(plane), _i(_code(plane)),
                                                         _i(d.shape[0]), _stream())
@@ -917,14 +1008,15 @@ def latent_kv_write(d: torch.Tensor, d_offset: int, rank: int, rot: int, rotary:
 
 
 def latent_q_split(q: torch.Tensor, heads: int, dim: int, rot: int, rotary: int, inv_freq: Optional[torch.Tensor], positions: torch.Tensor,
-                   q_plain: torch.Tensor, q_rot: torch.Tensor) -> None:
-    """q float32 [T, >= heads * (dim + rot)] -> q_plain [heads, T, dim] and the rotated parts q_rot float32 [T, heads, rot]."""
+                   q_plain: torch.Tensor, q_rot: torch.Tensor, halves: bool = False, magnitude: float = 1.0) -> None:
+    """q float32 [T, >= heads * (dim + rot)] -> q_plain [heads, T, dim] and the rotated parts q_rot float32 [T, heads, rot]
+    (``halves``, ``magnitude`` as for :func:`latent_kv_write`)."""
     _need(q, "q", torch.float32), _need(q_plain, "q_plain"), _need(q_rot, "q_rot", torch.float32), _need(positions, "positions", torch.int32)
     T = q.shape[0]
     if q_plain.numel() != heads * T * dim or q_rot.numel() != T * heads * rot:
         raise KernelError("latent_q_split: sizes do not agree")
-    st = library("latent_attention").cj_latent_q_split(_ptr(q), _i(q.stride(0)), _i(heads), _i(dim), _i(rot), _i(rotary), _ptr(inv_freq),
-                                                       _ptr(positions), _i(T), _ptr(q_plain), _i(_code(q_plain)), _ptr(q_rot), _stream())
+    st = library("latent_attention").cj_latent_q_split(_ptr(q), _i(q.stride(0)), _i(heads), _i(dim), _i(rot), _i(rotary), _i(1 if halves else 0),
+                                                       _f(magnitude), _ptr(inv_freq), _ptr(positions), _i(T), _ptr(q_plain), _i(_code(q_plain)), _ptr(q_rot), _stream())
     _check(st, "latent_q_split")
 
 
@@ -934,12 +1026,13 @@ LATENT_FILL_BLOCKS = 592         # blocks that fill the machine (four an SM); fe
 
 def latent_attention(q_abs: torch.Tensor, q_rot: torch.Tensor, plane: torch.Tensor, rank: int, rot: int, heads: int,
                      positions: torch.Tensor, row_req: torch.Tensor, table: torch.Tensor, page_tokens: int, scale: float,
-                     out: torch.Tensor, max_context: int = 0, sink: Optional[torch.Tensor] = None) -> None:
+                     out: torch.Tensor, max_context: int = 0, sink: Optional[torch.Tensor] = None, window: int = 0) -> None:
     """Every (row, head): softmax over the row's keys [0, position] of (q_abs . c + q_rot . r) * scale,
     and the weighted sum of the latents.  q_abs float32 [heads, T, rank]; q_rot float32 [T, heads, rot];
     out [heads, T, rank] in the cache's dtype.  ``max_context`` (the longest row's keys, when the
     caller knows it): with few rows the keys of a row are cut into stretches that run side by side.
-    ``sink`` (float32 [heads]): the softmax's divisor also holds exp(sink[h])."""
+    ``sink`` (float32 [heads]): the softmax's divisor also holds exp(sink[h]).  ``window`` > 0: a row sees its last
+    ``window`` keys alone."""
     if sink is not None:
         _need(sink, "sink", torch.float32)
         if sink.numel() != heads:
@@ -951,6 +1044,8 @@ def latent_attention(q_abs: torch.Tensor, q_rot: torch.Tensor, plane: torch.Tens
         raise KernelError("latent_attention: sizes do not agree")
     blocks = T * -(-heads // 8)
     split_keys, splits, part_acc, part_ml = 0, 1, None, None
+    if window > 0:
+        max_context = min(max_context, window)
     if max_context > LATENT_SPLIT_MIN_KEYS and blocks < LATENT_FILL_BLOCKS:
         want = min(64, -(-LATENT_FILL_BLOCKS // blocks))
         split_keys = max(LATENT_SPLIT_MIN_KEYS, -(-(-(-max_context // want)) // 32) * 32)
@@ -962,7 +1057,7 @@ def latent_attention(q_abs: torch.Tensor, q_rot: torch.Tensor, plane: torch.Tens
             split_keys = 0
     st = library("latent_attention").cj_latent_attention(_ptr(q_abs), _ptr(q_rot), _ptr(plane), _i(_code(plane)), _i(rank), _i(rot),
                                                          _i(heads), _i(T), _ptr(positions), _ptr(row_req), _ptr(table),
-                                                         _i(table.stride(0)), _i(page_tokens), _f(scale), _ptr(out),
+                                                         _i(table.stride(0)), _i(page_tokens), _i(window), _f(scale), _ptr(out),
                                                          _i(split_keys), _i(splits), _ptr(part_acc), _ptr(part_ml), _ptr(sink), _stream())
     _check(st, "latent_attention")
     if split_keys:
@@ -998,21 +1093,24 @@ def latent_kv_pack(kp: torch.Tensor, vp: torch.Tensor, plane: torch.Tensor, rank
 
 
 def latent_q_pack(q: torch.Tensor, heads: int, dim: int, rot: int, rotary: int, inv_freq: Optional[torch.Tensor],
-                  positions: torch.Tensor, qx: torch.Tensor) -> None:
-    """qx[t, h] = [q[t, h, :dim] | rotate(q[t, h, dim:]) | 0] in bfloat16; q float32 [T, >= heads (dim + rot)]."""
+                  positions: torch.Tensor, qx: torch.Tensor, halves: bool = False, magnitude: float = 1.0) -> None:
+    """qx[t, h] = [q[t, h, :dim] | rotate(q[t, h, dim:]) | 0] in bfloat16; q float32 [T, >= heads (dim + rot)]
+    (``halves``, ``magnitude`` as for :func:`latent_kv_write`)."""
     _need(q, "q", torch.float32), _need(qx, "qx", torch.bfloat16), _need(positions, "positions", torch.int32)
-    st = library("latent_prefill").cj_latent_q_pack(_ptr(q), _i(q.stride(0)), _i(heads), _i(dim), _i(rot), _i(rotary), _ptr(inv_freq),
-                                                    _ptr(positions), _i(qx.shape[2]), _ptr(qx), _i(q.shape[0]), _stream())
+    st = library("latent_prefill").cj_latent_q_pack(_ptr(q), _i(q.stride(0)), _i(heads), _i(dim), _i(rot), _i(rotary), _i(1 if halves else 0),
+                                                   _f(magnitude), _ptr(inv_freq), _ptr(positions), _i(qx.shape[2]), _ptr(qx), _i(q.shape[0]), _stream())
     _check(st, "latent_q_pack")
 
 
 def latent_flash(qx: torch.Tensor, out: torch.Tensor, kx: torch.Tensor, vx: torch.Tensor, req_start: torch.Tensor,
                  req_prior: torch.Tensor, req_base: torch.Tensor, requests: int, heads: int, scale: float,
-                 sink: Optional[torch.Tensor] = None) -> None:
+                 sink: Optional[torch.Tensor] = None, window: int = 0, exact_weights: bool = False) -> None:
     """Causal attention of the step's rows (request i: rows [req_start[i], req_start[i+1]) at positions
     req_prior[i] + j) over the dense keys and values of their requests (request i's token p at
     req_base[i] + p).  qx [T, heads, DK], kx [N, heads, DK], vx [N, heads, DV], out [T, heads, DV], bfloat16.
-    ``sink`` (float32 [heads]): the softmax's divisor also holds exp(sink[h])."""
+    ``sink`` (float32 [heads]): the softmax's divisor also holds exp(sink[h]).  ``window`` > 0: a row sees its last ``window``
+    keys alone; kx and vx then need a request's tokens from req_prior[i] + 1 - window on only.  ``exact_weights``: the softmax's
+    weights enter the product with the values as two bfloat16 terms instead of one."""
     if sink is not None:
         _need(sink, "sink", torch.float32)
     for n, t in (("qx", qx), ("out", out), ("kx", kx), ("vx", vx)):
@@ -1020,18 +1118,20 @@ def latent_flash(qx: torch.Tensor, out: torch.Tensor, kx: torch.Tensor, vx: torc
     for n, t in (("req_start", req_start), ("req_prior", req_prior), ("req_base", req_base)):
         _need(t, n, torch.int32)
     st = library("latent_prefill").cj_latent_flash(_ptr(qx), _ptr(out), _ptr(kx), _ptr(vx), _ptr(req_start), _ptr(req_prior), _ptr(req_base),
-                                                   _i(requests), _i(qx.shape[0]), _i(heads), _i(qx.shape[2]), _i(vx.shape[2]), _f(scale),
-                                                   _ptr(sink), _stream())
+                                                   _i(requests), _i(qx.shape[0]), _i(heads), _i(qx.shape[2]), _i(vx.shape[2]), _i(window),
+                                                   _i(1 if exact_weights else 0), _f(scale), _ptr(sink), _stream())
     _check(st, "latent_flash")
 
 
-def latent_gate_rows(o: torch.Tensor, gate: Optional[torch.Tensor], gate_offset: int, heads: int, vdim: int, out: torch.Tensor) -> None:
+def latent_gate_rows(o: torch.Tensor, gate: Optional[torch.Tensor], gate_offset: int, heads: int, vdim: int, out: torch.Tensor,
+                     by_entry: bool = False) -> None:
     """out[t, h * vdim + e] = o[t, h, e] * sigmoid(gate[t, gate_offset + h]); o bfloat16 [T, heads, DV], gate float32
-    (None: no gate, the heads' entries are only moved out of their padding)."""
+    (None: no gate, the heads' entries are only moved out of their padding).  ``by_entry``: the gate has a column for every entry,
+    gate[t, gate_offset + h * vdim + e]."""
     _need(o, "o", torch.bfloat16), _need(out, "out", torch.bfloat16)
     gate_ptr, gate_ld = _gate(gate, gate_offset)
     st = library("latent_prefill").cj_latent_gate_rows(_ptr(o), _i(o.shape[2]), gate_ptr,
-                                                       _i(gate_ld), _i(heads), _i(vdim), _ptr(out), _i(o.shape[0]), _stream())
+                                                       _i(gate_ld), _i(1 if by_entry else 0), _i(heads), _i(vdim), _ptr(out), _i(o.shape[0]), _stream())
     _check(st, "latent_gate_rows")
 
 
@@ -1046,14 +1146,16 @@ def latent_q_norm(x: torch.Tensor, offset: int, n: int, weight: torch.Tensor, ep
     _check(st, "latent_q_norm")
 
 
-def latent_gate_out(o: torch.Tensor, gate: Optional[torch.Tensor], gate_offset: int, heads: int, vdim: int, out: torch.Tensor) -> None:
-    """out[t, h, :] = o[h, t, :] * sigmoid(gate[t, gate_offset + h]); o float32 [heads, T, vdim], gate float32 (None: no gate)."""
+def latent_gate_out(o: torch.Tensor, gate: Optional[torch.Tensor], gate_offset: int, heads: int, vdim: int, out: torch.Tensor,
+                    by_entry: bool = False) -> None:
+    """out[t, h, :] = o[h, t, :] * sigmoid(gate[t, gate_offset + h]); o float32 [heads, T, vdim], gate float32 (None: no gate;
+    ``by_entry`` as for :func:`latent_gate_rows`)."""
     _need(o, "o", torch.float32), _need(out, "out")
     T = out.shape[0]
     if o.numel() != heads * T * vdim or out.shape[1] != heads * vdim:
         raise KernelError("latent_gate_out: sizes do not agree")
     gate_ptr, gate_ld = _gate(gate, gate_offset)
-    st = library("latent_attention").cj_latent_gate_out(_ptr(o), gate_ptr, _i(gate_ld),
+    st = library("latent_attention").cj_latent_gate_out(_ptr(o), gate_ptr, _i(gate_ld), _i(1 if by_entry else 0),
                                                         _i(heads), _i(vdim), _i(T), _ptr(out), _i(_code(out)), _stream())
     _check(st, "latent_gate_out")
 
@@ -1096,19 +1198,23 @@ def random_fill(out: torch.Tensor, key: int, scale: float) -> None:
     _check(st, "random_fill")
 
 
-EPI_STORE_F32, EPI_ACC_F32, EPI_SWIGLU_BF16, EPI_STORE_BF16, EPI_RELU2_BF16 = 0, 1, 2, 3, 4
+EPI_STORE_F32, EPI_ACC_F32, EPI_SWIGLU_BF16, EPI_STORE_BF16, EPI_RELU2_BF16, EPI_GELU_BF16, EPI_SILU_BF16 = 0, 1, 2, 3, 4, 5, 6
+BF16_EPILOGUES = (EPI_SWIGLU_BF16, EPI_STORE_BF16, EPI_RELU2_BF16, EPI_GELU_BF16, EPI_SILU_BF16)
 
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, swap: bool, n_mma: int,
             bias: Optional[torch.Tensor] = None, w_up: Optional[torch.Tensor] = None,
             group_offsets: Optional[torch.Tensor] = None, tokens: Optional[int] = None, k_splits: int = 1,
-            offsets_settled: bool = False, act_limit: float = 0.0, act_alpha: float = 1.0, out_scale: float = 1.0) -> None:
+            offsets_settled: bool = False, act_limit: float = 0.0, act_alpha: float = 1.0, out_scale: float = 1.0,
+            act_cubic: float = 0.0, bias_up: Optional[torch.Tensor] = None, act_features: int = 0) -> None:
     """Tensor-core product out[token, feature] (+)= out_scale (x[token, :] . w[feature, :] (+ bias)) in
     bfloat16 with float32 accumulation (tcgen05, TMA).
 
     ``swap`` False: tiles of 128 tokens x ``n_mma`` (128 or 256) features; True: tiles of 128
     features x ``n_mma`` (16, 32, 64, 96, 128, 160, 192, 256) tokens.  ``epilogue``: EPI_STORE_F32, EPI_ACC_F32,
-    EPI_SWIGLU_BF16 (``w_up`` given), EPI_STORE_BF16, EPI_RELU2_BF16 (``max(sum, 0)^2`` rounded to bfloat16).  With ``group_offsets`` the rows of
+    EPI_SWIGLU_BF16 (``w_up`` given; ``bias``, ``bias_up``, ``act_alpha`` and ``act_cubic`` as in :func:`gemm`), EPI_STORE_BF16, EPI_RELU2_BF16
+    (``max(sum, 0)^2`` rounded to bfloat16), EPI_GELU_BF16 (gelu by the error function, likewise), EPI_SILU_BF16;
+    ``act_features`` > 0: the activation of the last three for the first that many features alone.  With ``group_offsets`` the rows of
     ``x`` are sorted by group and ``w`` is [groups, features, K].  ``k_splits`` > 1 (store
     only): ``out`` is [k_splits, tokens, features] of partial sums.  ``offsets_settled``: the
     kernel that wrote ``group_offsets`` is not the one launched just before this product but an
@@ -1122,13 +1228,12 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, 
     T = tokens if tokens is not None else x.shape[0]
     if x.shape[-1] != K or out.shape[-1] != features:
         raise KernelError(f"gemm_tc: shapes x {tuple(x.shape)} w {tuple(w.shape)} out {tuple(out.shape)} do not agree")
-    want = torch.bfloat16 if epilogue in (EPI_SWIGLU_BF16, EPI_STORE_BF16, EPI_RELU2_BF16) else torch.float32
+    want = torch.bfloat16 if epilogue in BF16_EPILOGUES else torch.float32
     if out.dtype != want:
         raise KernelError(f"gemm_tc: epilogue {epilogue} writes {want}, out is {out.dtype}")
     if w_up is not None:
         _need(w_up, "w_up", torch.bfloat16)
-    if bias is not None:
-        _need(bias, "bias", torch.float32)
+    _gate_biases(w, w_up, bias, bias_up, "")
     G = 0
     if group_offsets is not None:
         _need(group_offsets, "group_offsets", torch.int32)
@@ -1136,16 +1241,18 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, 
     split_stride = out.stride(0) if k_splits > 1 else 0
     ldo = out.stride(-2)
     st = library("gemm_tc").cj_gemm_tc(
-        _ptr(x), _ll(x.stride(0)), _ptr(w), _ptr(w_up), _ptr(bias), _ptr(out), _ll(ldo), _i(T), _i(features), _i(K),
+        _ptr(x), _ll(x.stride(0)), _ptr(w), _ptr(w_up), _ptr(bias), _ptr(bias_up), _ptr(out), _ll(ldo), _i(T), _i(features), _i(K),
         _i(epilogue), _i(1 if swap else 0), _i(n_mma), _ptr(group_offsets), _i(G), _i(k_splits), _ll(split_stride),
-        _i(1 if offsets_settled and group_offsets is not None else 0), _f(act_limit), _f(act_alpha), _f(out_scale), _stream())
+        _i(1 if offsets_settled and group_offsets is not None else 0), _f(act_limit), _f(act_alpha), _f(act_cubic), _i(act_features),
+        _f(out_scale), _stream())
     _check(st, "gemm_tc")
 
 
 def gemm_tc2(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, n_tok: int,
              bias: Optional[torch.Tensor] = None, w_up: Optional[torch.Tensor] = None,
              group_offsets: Optional[torch.Tensor] = None, tokens: Optional[int] = None, act_limit: float = 0.0,
-             act_alpha: float = 1.0, out_scale: float = 1.0) -> None:
+             act_alpha: float = 1.0, out_scale: float = 1.0, act_cubic: float = 0.0, bias_up: Optional[torch.Tensor] = None,
+             act_features: int = 0) -> None:
     """The same product as ``gemm_tc`` on pairs of SMs (tcgen05 cta_group::2): tiles of 256
     features x ``n_tok`` (128 or 256) tokens, each SM of a pair loading its own 128 weight rows
     and half of the token rows.  For steps with many rows."""
@@ -1156,20 +1263,20 @@ def gemm_tc2(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int,
     T = tokens if tokens is not None else x.shape[0]
     if x.shape[-1] != K or out.shape[-1] != features:
         raise KernelError(f"gemm_tc2: shapes x {tuple(x.shape)} w {tuple(w.shape)} out {tuple(out.shape)} do not agree")
-    want = torch.bfloat16 if epilogue in (EPI_SWIGLU_BF16, EPI_STORE_BF16, EPI_RELU2_BF16) else torch.float32
+    want = torch.bfloat16 if epilogue in BF16_EPILOGUES else torch.float32
     if out.dtype != want:
         raise KernelError(f"gemm_tc2: epilogue {epilogue} writes {want}, out is {out.dtype}")
     if w_up is not None:
         _need(w_up, "w_up", torch.bfloat16)
-    if bias is not None:
-        _need(bias, "bias", torch.float32)
+    _gate_biases(w, w_up, bias, bias_up, "")
     G = 0
     if group_offsets is not None:
         _need(group_offsets, "group_offsets", torch.int32)
         G = w.shape[0]
     st = library("gemm_tc2").cj_gemm_tc2(
-        _ptr(x), _ll(x.stride(0)), _ptr(w), _ptr(w_up), _ptr(bias), _ptr(out), _ll(out.stride(-2)), _i(T), _i(features), _i(K),
-        _i(epilogue), _i(n_tok), _ptr(group_offsets), _i(G), _f(act_limit), _f(act_alpha), _f(out_scale), _stream())
+        _ptr(x), _ll(x.stride(0)), _ptr(w), _ptr(w_up), _ptr(bias), _ptr(bias_up), _ptr(out), _ll(out.stride(-2)), _i(T), _i(features), _i(K),
+        _i(epilogue), _i(n_tok), _ptr(group_offsets), _i(G), _f(act_limit), _f(act_alpha), _f(act_cubic), _i(act_features),
+        _f(out_scale), _stream())
     _check(st, "gemm_tc2")
 
 

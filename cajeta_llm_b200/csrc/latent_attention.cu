@@ -12,14 +12,16 @@
 // latent_attention  scores, softmax and the weighted sum of latents for every (row, head);
 //                   q_abs [H, T, kv_rank] in, the summed latents [H, T, kv_rank] out (both head-major;
 //                   the sums leave in the cache's dtype, as the next product's input)
-// latent_gate_out   out[t, h, :] = o[h, t, :] * sigmoid(gate[t, h])  (back to token-major; without a gate: the move alone)
+// latent_gate_out   out[t, h, :] = o[h, t, :] * sigmoid(gate[t, h])  (back to token-major; without a gate: the move alone;
+//                   or a gate of its own for every entry, gate[t, h * vdim + e])
 // latent_q_norm     the queries' own latent: rms(x[:, offset : offset + n]) * w into the activation dtype
 //
 // A sink (optional, one float32 per head): the softmax's divisor also holds exp(sink[h]), a term without key or value
 // that is neither scaled nor rotated; the running maximum of a row's first stretch starts at it and the running sum at 1.
 //
-// The rotation pairs entries (2i, 2i+1); the angle p * inv_freq[i] is float32.  Scores,
-// softmax and sums are float32 whatever the cache holds.
+// The rotation pairs entries (2i, 2i+1), or (i, i + rotary / 2) when `halves`; the angle p * inv_freq[i] is float32, cos and
+// sin are multiplied by `mag`.  A window w > 0: a row at position p sees the keys p - w + 1 .. p alone (pages before them may
+// be gone).  Scores, softmax and sums are float32 whatever the cache holds.
 #define CJ_LIB "latent_attention"
 #include "common.cuh"
 
@@ -28,7 +30,8 @@ using namespace cj;
 namespace {
 
 template <typename TC>
-__global__ void latent_kv_write_kernel(const float* __restrict__ d, int ld, int rank, int rot, int rotary, const float* __restrict__ w,
+__global__ void latent_kv_write_kernel(const float* __restrict__ d, int ld, int rank, int rot, int rotary, int halves, float mag,
+                                       const float* __restrict__ w,
                                        float eps, const float* __restrict__ inv_freq, const int* __restrict__ positions,
                                        const int* __restrict__ row_req, const int* __restrict__ table, int table_stride,
                                        int page_tokens, TC* __restrict__ plane) {
@@ -52,17 +55,18 @@ __global__ void latent_kv_write_kernel(const float* __restrict__ d, int ld, int 
     for (int i = threadIdx.x; i < rank; i += blockDim.x) dst[i] = from_f32<TC>(src[i] * scale * w[i]);
     for (int i = threadIdx.x; i < rotary / 2; i += blockDim.x) {
         const float a = (float)pos * inv_freq[i];
-        const float c = cosf(a), s = sinf(a);
-        const float u = src[rank + 2 * i], v = src[rank + 2 * i + 1];
-        dst[rank + 2 * i] = from_f32<TC>(u * c - v * s);
-        dst[rank + 2 * i + 1] = from_f32<TC>(v * c + u * s);
+        const float c = mag * cosf(a), s = mag * sinf(a);
+        const int i0 = rank + (halves ? i : 2 * i), i1 = rank + (halves ? i + rotary / 2 : 2 * i + 1);
+        const float u = src[i0], v = src[i1];
+        dst[i0] = from_f32<TC>(u * c - v * s);
+        dst[i1] = from_f32<TC>(v * c + u * s);
     }
     for (int i = rotary + threadIdx.x; i < rot; i += blockDim.x) dst[rank + i] = from_f32<TC>(src[rank + i]);   // past the rotated dims: unchanged
 }
 
 template <typename TO>
-__global__ void latent_q_split_kernel(const float* __restrict__ q, int ld, int heads, int dim, int rot, int rotary,
-                                      const float* __restrict__ inv_freq, const int* __restrict__ positions, int T,
+__global__ void latent_q_split_kernel(const float* __restrict__ q, int ld, int heads, int dim, int rot, int rotary, int halves,
+                                      float mag, const float* __restrict__ inv_freq, const int* __restrict__ positions, int T,
                                       TO* __restrict__ q_plain, float* __restrict__ q_rot) {
     cj::after_predecessor();
     cj::release_successor();
@@ -77,11 +81,12 @@ __global__ void latent_q_split_kernel(const float* __restrict__ q, int ld, int h
     for (int i = threadIdx.x; i < heads * (rotary / 2); i += blockDim.x) {
         const int h = i / (rotary / 2), e = i % (rotary / 2);
         const float a = (float)pos * inv_freq[e];
-        const float c = cosf(a), s = sinf(a);
-        const float u = src[h * per + dim + 2 * e], v = src[h * per + dim + 2 * e + 1];
+        const float c = mag * cosf(a), s = mag * sinf(a);
+        const int e0 = halves ? e : 2 * e, e1 = halves ? e + rotary / 2 : 2 * e + 1;
+        const float u = src[h * per + dim + e0], v = src[h * per + dim + e1];
         float* dst = q_rot + ((size_t)r * heads + h) * rot;
-        dst[2 * e] = u * c - v * s;
-        dst[2 * e + 1] = v * c + u * s;
+        dst[e0] = u * c - v * s;
+        dst[e1] = v * c + u * s;
     }
     const int rest = rot - rotary;
     for (int i = threadIdx.x; i < heads * rest; i += blockDim.x) {
@@ -98,8 +103,8 @@ __global__ void latent_q_split_kernel(const float* __restrict__ q, int ld, int h
 // when the cache holds 16-bit entries: one 32-bit word a read).
 // With few rows in the step (decoding) the keys of a row are cut into stretches of split_keys,
 // one block each (blockIdx.z), which leave unnormalised sums, maxima and weights behind; a
-// second kernel merges them in stretch order.  How a row is cut depends on its position and
-// split_keys only.
+// second kernel merges them in stretch order.  How a row is cut depends on its position, the window
+// and split_keys only.
 constexpr int LA_KEYS = 32;
 constexpr int LA_HEADS = 8;
 
@@ -110,7 +115,7 @@ template <typename TC, int NACC>
 __global__ void __launch_bounds__(LA_HEADS * 32) latent_attention_kernel(
     const float* __restrict__ q_abs, const float* __restrict__ q_rot, const TC* __restrict__ plane, int rank, int rot,
     int heads, int T, const int* __restrict__ positions, const int* __restrict__ row_req, const int* __restrict__ table,
-    int table_stride, int page_tokens, float scale, TC* __restrict__ out, int row_words, int split_keys,
+    int table_stride, int page_tokens, int window, float scale, TC* __restrict__ out, int row_words, int split_keys,
     float* __restrict__ part_acc, float* __restrict__ part_ml, const float* __restrict__ sink) {
     cj::after_predecessor();
     cj::release_successor();
@@ -124,7 +129,8 @@ __global__ void __launch_bounds__(LA_HEADS * 32) latent_attention_kernel(
     const int head = blockIdx.y * LA_HEADS + warp;
     const bool has_head = head < heads;
     const int pos = positions[r];
-    const int key_begin = split_keys > 0 ? (int)blockIdx.z * split_keys : 0;
+    const int oldest = window > 0 ? max(0, pos + 1 - window) : 0;         // the first key the row sees
+    const int key_begin = oldest + (split_keys > 0 ? (int)blockIdx.z * split_keys : 0);
     const int key_end = split_keys > 0 ? min(pos + 1, key_begin + split_keys) : pos + 1;
     if (key_begin >= key_end) return;                            // this stretch lies past the row's position
     const int* pages = table + (size_t)row_req[r] * table_stride;
@@ -140,7 +146,7 @@ __global__ void __launch_bounds__(LA_HEADS * 32) latent_attention_kernel(
 #pragma unroll
     for (int i = 0; i < NACC; ++i) acc[i] = 0.0f;
     float m = -INFINITY, l = 0.0f;
-    if (sink && has_head && key_begin == 0) { m = sink[head]; l = 1.0f; }       // the sink counts once: in the row's first stretch
+    if (sink && has_head && key_begin == oldest) { m = sink[head]; l = 1.0f; }       // the sink counts once: in the row's first stretch
     const TC* krow_base = (const TC*)ks;
     const int row_elems = row_words * (int)(4 / sizeof(TC));
     for (int k0 = key_begin; k0 < key_end; k0 += LA_KEYS) {
@@ -260,11 +266,12 @@ __global__ void __launch_bounds__(LA_HEADS * 32) latent_attention_kernel(
 // the stretches of a row's keys, merged in order: out = sum_z e^(m_z - M) acc_z / sum_z e^(m_z - M) l_z
 template <typename TC>
 __global__ void latent_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml, int splits, int split_keys,
-                                    int rank, int heads, int T, const int* __restrict__ positions, TC* __restrict__ out) {
+                                    int window, int rank, int heads, int T, const int* __restrict__ positions, TC* __restrict__ out) {
     cj::after_predecessor();
     cj::release_successor();
     const int r = blockIdx.x, head = blockIdx.y;
-    const int nz = min(splits, (positions[r] + split_keys) / split_keys);
+    const int n_keys = window > 0 ? min(positions[r] + 1, window) : positions[r] + 1;
+    const int nz = min(splits, (n_keys + split_keys - 1) / split_keys);
     const size_t item = (size_t)r * heads + head;
     const float* ml = part_ml + item * splits * 2;
     float M = -INFINITY;
@@ -280,14 +287,14 @@ __global__ void latent_merge_kernel(const float* __restrict__ part_acc, const fl
 }
 
 template <typename TO>
-__global__ void latent_gate_out_kernel(const float* __restrict__ o, const float* __restrict__ gate, int ld_gate, int heads,
+__global__ void latent_gate_out_kernel(const float* __restrict__ o, const float* __restrict__ gate, int ld_gate, int by_entry, int heads,
                                        int vdim, int T, TO* __restrict__ out) {
     cj::after_predecessor();
     cj::release_successor();
     const int r = blockIdx.x;
     for (int i = threadIdx.x; i < heads * vdim; i += blockDim.x) {
         const int h = i / vdim, e = i % vdim;
-        const float g = gate ? 1.0f / (1.0f + expf(-gate[(size_t)r * ld_gate + h])) : 1.0f;
+        const float g = gate ? 1.0f / (1.0f + expf(-gate[(size_t)r * ld_gate + (by_entry ? i : h)])) : 1.0f;
         out[(size_t)r * heads * vdim + i] = from_f32<TO>(o[((size_t)h * T + r) * vdim + e] * g);
     }
 }
@@ -325,41 +332,42 @@ CJ_EXPORT int cj_latent_q_norm(const float* x, int ld, int offset, int n, const 
     return launch_status();
 }
 
-CJ_EXPORT int cj_latent_kv_write(const float* d, int ld, int rank, int rot, int rotary, const float* w, float eps, const float* inv_freq,
-                                 const int* positions, const int* row_req, const int* table, int table_stride, int page_tokens,
+CJ_EXPORT int cj_latent_kv_write(const float* d, int ld, int rank, int rot, int rotary, int halves, float mag, const float* w, float eps,
+                                 const float* inv_freq, const int* positions, const int* row_req, const int* table, int table_stride, int page_tokens,
                                  void* plane, int cache_dtype, int T, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (!d || !w || !positions || !row_req || !table || !plane || rank <= 0 || rot < 0 || page_tokens <= 0) return CJ_ERR_ARG;
     if ((rotary & 1) || rotary < 0 || rotary > rot || (rotary > 0 && !inv_freq)) return CJ_ERR_SIZE;
     int threads = rank >= 512 ? 256 : 128;
-    if (cache_dtype == CJ_F32) cj::launch(latent_kv_write_kernel<float>, dim3(T), dim3(threads), 0, stream, d, ld, rank, rot, rotary, w, eps, inv_freq, positions, row_req, table, table_stride, page_tokens, (float*)plane);
-    else if (cache_dtype == CJ_BF16) cj::launch(latent_kv_write_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, d, ld, rank, rot, rotary, w, eps, inv_freq, positions, row_req, table, table_stride, page_tokens, (__nv_bfloat16*)plane);
+    if (cache_dtype == CJ_F32) cj::launch(latent_kv_write_kernel<float>, dim3(T), dim3(threads), 0, stream, d, ld, rank, rot, rotary, halves, mag, w, eps, inv_freq, positions, row_req, table, table_stride, page_tokens, (float*)plane);
+    else if (cache_dtype == CJ_BF16) cj::launch(latent_kv_write_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, d, ld, rank, rot, rotary, halves, mag, w, eps, inv_freq, positions, row_req, table, table_stride, page_tokens, (__nv_bfloat16*)plane);
     else return CJ_ERR_DTYPE;
     return launch_status();
 }
 
-CJ_EXPORT int cj_latent_q_split(const float* q, int ld, int heads, int dim, int rot, int rotary, const float* inv_freq, const int* positions,
+CJ_EXPORT int cj_latent_q_split(const float* q, int ld, int heads, int dim, int rot, int rotary, int halves, float mag,
+                                const float* inv_freq, const int* positions,
                                 int T, void* q_plain, int plain_dtype, float* q_rot, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (!q || !positions || !q_plain || !q_rot || heads <= 0 || dim <= 0 || rot < 0) return CJ_ERR_ARG;
     if ((rotary & 1) || rotary < 0 || rotary > rot || (rotary > 0 && !inv_freq)) return CJ_ERR_SIZE;
     int threads = heads * dim >= 2048 ? 256 : 128;
-    if (plain_dtype == CJ_F32) cj::launch(latent_q_split_kernel<float>, dim3(T), dim3(threads), 0, stream, q, ld, heads, dim, rot, rotary, inv_freq, positions, T, (float*)q_plain, q_rot);
-    else if (plain_dtype == CJ_BF16) cj::launch(latent_q_split_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, q, ld, heads, dim, rot, rotary, inv_freq, positions, T, (__nv_bfloat16*)q_plain, q_rot);
+    if (plain_dtype == CJ_F32) cj::launch(latent_q_split_kernel<float>, dim3(T), dim3(threads), 0, stream, q, ld, heads, dim, rot, rotary, halves, mag, inv_freq, positions, T, (float*)q_plain, q_rot);
+    else if (plain_dtype == CJ_BF16) cj::launch(latent_q_split_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, q, ld, heads, dim, rot, rotary, halves, mag, inv_freq, positions, T, (__nv_bfloat16*)q_plain, q_rot);
     else return CJ_ERR_DTYPE;
     return launch_status();
 }
 
 // split_keys > 0: a row's keys are cut into stretches of that many (a multiple of 32), one block each;
 // part_acc [T, heads, splits, rank] and part_ml [T, heads, splits, 2] (float32) then hold the
-// stretches' results, splits = ceil(max_context / split_keys).  split_keys = 0: one block a row.
+// stretches' results, splits = ceil(the most keys a row sees / split_keys).  split_keys = 0: one block a row.  window: 0 = none.
 CJ_EXPORT int cj_latent_attention(const float* q_abs, const float* q_rot, const void* plane, int cache_dtype, int rank, int rot,
                                   int heads, int T, const int* positions, const int* row_req, const int* table, int table_stride,
-                                  int page_tokens, float scale, void* out, int split_keys, int splits, float* part_acc,
+                                  int page_tokens, int window, float scale, void* out, int split_keys, int splits, float* part_acc,
                                   float* part_ml, const float* sink, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (!q_abs || !q_rot || !plane || !positions || !row_req || !table || !out) return CJ_ERR_ARG;
-    if (rank <= 0 || rank > 1024 || rot < 0 || heads <= 0 || page_tokens <= 0) return CJ_ERR_SIZE;
+    if (rank <= 0 || rank > 1024 || rot < 0 || heads <= 0 || page_tokens <= 0 || window < 0) return CJ_ERR_SIZE;
     if (split_keys < 0 || split_keys % LA_KEYS != 0 || (split_keys > 0 && (splits < 1 || splits > 65535 || !part_acc || !part_ml))) return CJ_ERR_ARG;
     const int width = rank + rot;
     const int esize = cache_dtype == CJ_F32 ? 4 : 2;
@@ -380,11 +388,11 @@ CJ_EXPORT int cj_latent_attention(const float* q_abs, const float* q_rot, const 
             sized_##N = true;                                                                                          \
         }                                                                                                              \
         cj::launch(latent_attention_kernel<TC, N>, grid, dim3(LA_HEADS * 32), smem, stream, q_abs, q_rot, (const TC*)plane, \
-                   rank, rot, heads, T, positions, row_req, table, table_stride, page_tokens, scale, (TC*)out, row_words, \
+                   rank, rot, heads, T, positions, row_req, table, table_stride, page_tokens, window, scale, (TC*)out, row_words, \
                    split_keys, pa, pm, sink);                                                                          \
         if (split_keys > 0)                                                                                            \
             cj::launch(latent_merge_kernel<TC>, dim3(T, heads), dim3(128), 0, stream, (const float*)pa, (const float*)pm, splits, \
-                       split_keys, rank, heads, T, positions, (TC*)out);                                               \
+                       split_keys, window, rank, heads, T, positions, (TC*)out);                                               \
     } while (0)
 #define PICK(TC)                                  \
     do {                                          \
@@ -401,13 +409,14 @@ CJ_EXPORT int cj_latent_attention(const float* q_abs, const float* q_rot, const 
     return launch_status();
 }
 
-CJ_EXPORT int cj_latent_gate_out(const float* o, const float* gate, int ld_gate, int heads, int vdim, int T, void* out,
+// gate: one column per head, or (by_entry) one per entry of the heads side by side
+CJ_EXPORT int cj_latent_gate_out(const float* o, const float* gate, int ld_gate, int by_entry, int heads, int vdim, int T, void* out,
                                  int out_dtype, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (!o || !out || heads <= 0 || vdim <= 0) return CJ_ERR_ARG;
     int threads = heads * vdim >= 2048 ? 256 : 128;
-    if (out_dtype == CJ_F32) cj::launch(latent_gate_out_kernel<float>, dim3(T), dim3(threads), 0, stream, o, gate, ld_gate, heads, vdim, T, (float*)out);
-    else if (out_dtype == CJ_BF16) cj::launch(latent_gate_out_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, o, gate, ld_gate, heads, vdim, T, (__nv_bfloat16*)out);
+    if (out_dtype == CJ_F32) cj::launch(latent_gate_out_kernel<float>, dim3(T), dim3(threads), 0, stream, o, gate, ld_gate, by_entry, heads, vdim, T, (float*)out);
+    else if (out_dtype == CJ_BF16) cj::launch(latent_gate_out_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, o, gate, ld_gate, by_entry, heads, vdim, T, (__nv_bfloat16*)out);
     else return CJ_ERR_DTYPE;
     return launch_status();
 }

@@ -14,11 +14,14 @@
 //   latent_kv_pack  [N, H, DK] = [k_plain(h) | r | 0], [N, H, DV] = [v(h) | 0]   (DK, DV: padded to 64)
 //   latent_q_pack   [T, H, DK] = [q_plain(h) | rotate(q_rot(h)) | 0]
 //   latent_flash    out [T, H, DV]
-//   latent_gate_rows out[t, h vdim + e] = o[t, h, e] * sigmoid(gate[t, h])
+//   latent_gate_rows out[t, h vdim + e] = o[t, h, e] * sigmoid(gate[t, h])  (or gate[t, h vdim + e])
 //
 // Token n of the dense buffers is (request tok_req[n], position tok_pos[n]); request i's
 // tokens lie at req_base[i] + position.  Rows are the step's rows: request i owns rows
-// [req_start[i], req_start[i+1]) at positions req_prior[i] + j.
+// [req_start[i], req_start[i+1]) at positions req_prior[i] + j.  A window w > 0: a row at position p sees the keys
+// p - w + 1 .. p alone; the dense buffers then need a request's tokens from req_prior[i] - w + 1 on only (req_base[i] may be
+// negative: it is where position 0 would lie), and tiles of keys before a block's oldest one are never visited.
+// EXACT: the weights enter the second product as two bfloat16 terms (their float32 value to 2^-17) instead of one.
 #define CJ_LIB "latent_prefill"
 #include "common.cuh"
 
@@ -54,6 +57,11 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
     return *(unsigned*)&v;
 }
 
+// the pair's rests after the bfloat16 terms in `first` (lo in its low half)
+__device__ __forceinline__ unsigned pack_rest(float lo, float hi, unsigned first) {
+    return pack_bf16(lo - __uint_as_float(first << 16), hi - __uint_as_float(first & 0xffff0000u));
+}
+
 // element (row, col) of a [rows][D] bf16 tile whose 16-byte chunks are XOR-swizzled by row (D a multiple of 64)
 template <int D>
 __device__ __forceinline__ __nv_bfloat16* tile_ptr(__nv_bfloat16* base, int row, int col) {
@@ -63,11 +71,11 @@ __device__ __forceinline__ __nv_bfloat16* tile_ptr(__nv_bfloat16* base, int row,
 
 constexpr int BM = 64, BN = 64, THREADS = 128;
 
-template <int DK, int DV>
+template <int DK, int DV, bool EXACT>
 __global__ void __launch_bounds__(THREADS) latent_flash_kernel(
     const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ kx,
     const __nv_bfloat16* __restrict__ vx, const int* __restrict__ req_start, const int* __restrict__ req_prior,
-    const int* __restrict__ req_base, int n_requests, int n_heads, float scale_log2, const float* __restrict__ sink) {
+    const int* __restrict__ req_base, int n_requests, int n_heads, int window, float scale_log2, const float* __restrict__ sink) {
     cj::after_predecessor();
     cj::release_successor();
     extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -94,6 +102,9 @@ __global__ void __launch_bounds__(THREADS) latent_flash_kernel(
     const int p0 = req_prior[req] + (row0 - req_start[req]);
     const int p_last = p0 + rows - 1;
     const int kt_end = p_last / BN;
+    // the oldest key any row of the block sees (keys before it may lie in no buffer: they are not loaded), and its tile
+    const int oldest = window > 0 ? max(0, p0 + 1 - window) : 0;
+    const int kt_begin = oldest / BN;
     const long long base = req_base[req];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
 
@@ -103,14 +114,14 @@ __global__ void __launch_bounds__(THREADS) latent_flash_kernel(
         for (int i = tid; i < BN * CK; i += THREADS) {
             int r = i / CK, c = i % CK;
             int key = kt * BN + r;
-            bool valid = key <= p_last;
+            bool valid = key <= p_last && key >= oldest;
             long long off = valid ? ((base + key) * n_heads + h) * DK + c * 8 : 0;
             cp_async16(kd + r * DK + (c ^ (r & 7)) * 8, kx + off, valid);
         }
         for (int i = tid; i < BN * CV; i += THREADS) {
             int r = i / CV, c = i % CV;
             int key = kt * BN + r;
-            bool valid = key <= p_last;
+            bool valid = key <= p_last && key >= oldest;
             long long off = valid ? ((base + key) * n_heads + h) * DV + c * 8 : 0;
             cp_async16(vd + r * DV + (c ^ (r & 7)) * 8, vx + off, valid);
         }
@@ -121,7 +132,7 @@ __global__ void __launch_bounds__(THREADS) latent_flash_kernel(
         const __nv_bfloat16* src = q + ((size_t)(row0 + (valid ? r : 0)) * n_heads + h) * DK + c * 8;
         cp_async16(qs + r * DK + (c ^ (r & 7)) * 8, src, valid);
     }
-    load_kv(0, 0);
+    load_kv(kt_begin, kt_begin & 1);
     cp_async_commit();
 
     const int g = lane >> 2, t4 = lane & 3;
@@ -131,7 +142,7 @@ __global__ void __launch_bounds__(THREADS) latent_flash_kernel(
 #pragma unroll
     for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
 
-    for (int kt = 0; kt <= kt_end; ++kt) {
+    for (int kt = kt_begin; kt <= kt_end; ++kt) {
         const int buf = kt & 1;
         if (kt < kt_end) load_kv(kt + 1, buf ^ 1);
         cp_async_commit();
@@ -156,19 +167,20 @@ __global__ void __launch_bounds__(THREADS) latent_flash_kernel(
                 mma_bf16(s[2 * jp + 1], qf, b[2], b[3]);
             }
         }
-        // causal mask and running softmax
+        // causal mask, window and running softmax
         const int kbase = kt * BN;
-        unsigned pf[BN / 16][4];
+        unsigned pf[BN / 16][4], pl[EXACT ? BN / 16 : 1][4];
         {
             const int pos0 = p0 + wrow + g, pos1 = pos0 + 8;
+            const int from0 = window > 0 ? pos0 - window : -1, from1 = window > 0 ? pos1 - window : -1;      // keys after these
             float mx0 = mrun[0], mx1 = mrun[1];
 #pragma unroll
             for (int j = 0; j < BN / 8; ++j) {
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     int key = kbase + j * 8 + 2 * t4 + e;
-                    float a = key <= pos0 ? s[j][e] * scale_log2 : -INFINITY;
-                    float b = key <= pos1 ? s[j][2 + e] * scale_log2 : -INFINITY;
+                    float a = key <= pos0 && key > from0 ? s[j][e] * scale_log2 : -INFINITY;
+                    float b = key <= pos1 && key > from1 ? s[j][2 + e] * scale_log2 : -INFINITY;
                     s[j][e] = a;
                     s[j][2 + e] = b;
                     mx0 = fmaxf(mx0, a);
@@ -191,6 +203,11 @@ __global__ void __launch_bounds__(THREADS) latent_flash_kernel(
                 sum1 += e2 + e3;
                 pf[j >> 1][(j & 1) * 2] = pack_bf16(e0, e1);
                 pf[j >> 1][(j & 1) * 2 + 1] = pack_bf16(e2, e3);
+                if (EXACT) {
+                    // what the first term leaves over
+                    pl[j >> 1][(j & 1) * 2] = pack_rest(e0, e1, pf[j >> 1][(j & 1) * 2]);
+                    pl[j >> 1][(j & 1) * 2 + 1] = pack_rest(e2, e3, pf[j >> 1][(j & 1) * 2 + 1]);
+                }
             }
             lrun[0] = lrun[0] * c0 + sum0;
             lrun[1] = lrun[1] * c1 + sum1;
@@ -211,6 +228,10 @@ __global__ void __launch_bounds__(THREADS) latent_flash_kernel(
                 ldmatrix_x4_trans(b, tile_ptr<DV>((__nv_bfloat16*)vb, kk * 16 + (mi & 1) * 8 + (lane & 7), dp * 16 + (mi >> 1) * 8));
                 mma_bf16(o[2 * dp], pf[kk], b[0], b[1]);
                 mma_bf16(o[2 * dp + 1], pf[kk], b[2], b[3]);
+                if (EXACT) {
+                    mma_bf16(o[2 * dp], pl[kk], b[0], b[1]);
+                    mma_bf16(o[2 * dp + 1], pl[kk], b[2], b[3]);
+                }
             }
         }
         __syncthreads();
@@ -271,8 +292,8 @@ __global__ void latent_kv_pack_kernel(const __nv_bfloat16* __restrict__ kp, cons
     }
 }
 
-__global__ void latent_q_pack_kernel(const float* __restrict__ q, int ld, int heads, int dim, int rot, int rotary,
-                                     const float* __restrict__ inv_freq, const int* __restrict__ positions, int DK,
+__global__ void latent_q_pack_kernel(const float* __restrict__ q, int ld, int heads, int dim, int rot, int rotary, int halves,
+                                     float mag, const float* __restrict__ inv_freq, const int* __restrict__ positions, int DK,
                                      __nv_bfloat16* __restrict__ qx) {
     cj::after_predecessor();
     cj::release_successor();
@@ -287,11 +308,13 @@ __global__ void latent_q_pack_kernel(const float* __restrict__ q, int ld, int he
         if (e < dim) {
             v = src[h * per + e];
         } else if (e < dim + rotary) {
-            const int j = e - dim, pair = j >> 1;
+            const int j = e - dim, hr = rotary / 2;
+            const int pair = halves ? (j < hr ? j : j - hr) : j >> 1;
+            const bool second = halves ? j >= hr : (j & 1) != 0;
             const float a = (float)pos * inv_freq[pair];
-            const float c = cosf(a), s = sinf(a);
-            const float u = src[h * per + dim + 2 * pair], w = src[h * per + dim + 2 * pair + 1];
-            v = (j & 1) ? w * c + u * s : u * c - w * s;
+            const float c = mag * cosf(a), s = mag * sinf(a);
+            const float u = src[h * per + dim + (halves ? pair : 2 * pair)], w = src[h * per + dim + (halves ? pair + hr : 2 * pair + 1)];
+            v = second ? w * c + u * s : u * c - w * s;
         } else if (e < per) {
             v = src[h * per + e];
         }
@@ -300,13 +323,13 @@ __global__ void latent_q_pack_kernel(const float* __restrict__ q, int ld, int he
 }
 
 __global__ void latent_gate_rows_kernel(const __nv_bfloat16* __restrict__ o, int DV, const float* __restrict__ gate, int ld_gate,
-                                        int heads, int vdim, __nv_bfloat16* __restrict__ out) {
+                                        int by_entry, int heads, int vdim, __nv_bfloat16* __restrict__ out) {
     cj::after_predecessor();
     cj::release_successor();
     const int r = blockIdx.x;
     for (int i = threadIdx.x; i < heads * vdim; i += blockDim.x) {
         const int h = i / vdim, e = i % vdim;
-        const float g = gate ? 1.0f / (1.0f + expf(-gate[(size_t)r * ld_gate + h])) : 1.0f;
+        const float g = gate ? 1.0f / (1.0f + expf(-gate[(size_t)r * ld_gate + (by_entry ? i : h)])) : 1.0f;
         out[(size_t)r * heads * vdim + i] = __float2bfloat16_rn(__bfloat162float(o[((size_t)r * heads + h) * DV + e]) * g);
     }
 }
@@ -334,38 +357,40 @@ CJ_EXPORT int cj_latent_kv_pack(const void* kp, const void* vp, const void* plan
     return launch_status();
 }
 
-CJ_EXPORT int cj_latent_q_pack(const float* q, int ld, int heads, int dim, int rot, int rotary, const float* inv_freq,
+CJ_EXPORT int cj_latent_q_pack(const float* q, int ld, int heads, int dim, int rot, int rotary, int halves, float mag, const float* inv_freq,
                                const int* positions, int DK, void* qx, int T, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (!q || !positions || !qx || heads <= 0 || dim <= 0 || rot < 0 || DK < dim + rot) return CJ_ERR_ARG;
     if ((rotary & 1) || rotary < 0 || rotary > rot || (rotary > 0 && !inv_freq)) return CJ_ERR_SIZE;
-    cj::launch(latent_q_pack_kernel, dim3(T), dim3(256), 0, stream, q, ld, heads, dim, rot, rotary, inv_freq, positions, DK,
+    cj::launch(latent_q_pack_kernel, dim3(T), dim3(256), 0, stream, q, ld, heads, dim, rot, rotary, halves, mag, inv_freq, positions, DK,
                (__nv_bfloat16*)qx);
     return launch_status();
 }
 
+// window: 0 = none; exact: weights as two bfloat16 terms.
 // q [T, heads, DK], kx [N, heads, DK], vx [N, heads, DV], out [T, heads, DV], all bf16; DK in {64, 128, 192, 256}, DV in {64, 128}
 CJ_EXPORT int cj_latent_flash(const void* q, void* out, const void* kx, const void* vx, const int* req_start, const int* req_prior,
-                              const int* req_base, int n_requests, int total_rows, int heads, int DK, int DV, float scale,
-                              const float* sink, cudaStream_t stream) {
+                              const int* req_base, int n_requests, int total_rows, int heads, int DK, int DV, int window, int exact,
+                              float scale, const float* sink, cudaStream_t stream) {
     if (total_rows <= 0 || n_requests <= 0) return 0;
     if (!q || !out || !kx || !vx || !req_start || !req_prior || !req_base) return CJ_ERR_ARG;
-    if (heads <= 0 || heads > 65535) return CJ_ERR_SIZE;
+    if (heads <= 0 || heads > 65535 || window < 0) return CJ_ERR_SIZE;
     const float scale_log2 = scale * 1.4426950408889634f;
     dim3 grid((total_rows + BM - 1) / BM + n_requests, heads);
-#define LAUNCH(K_, V_)                                                                                                   \
+#define LAUNCH_ONE(K_, V_, E_)                                                                                                 \
     {                                                                                                                    \
         size_t smem = (size_t)(BM * K_ + 2 * BN * K_ + 2 * BN * V_) * sizeof(__nv_bfloat16);                             \
         static bool configured = false;                                                                                  \
         if (!configured) {                                                                                               \
-            cudaError_t e = cudaFuncSetAttribute(latent_flash_kernel<K_, V_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            cudaError_t e = cudaFuncSetAttribute(latent_flash_kernel<K_, V_, E_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (e != cudaSuccess) return (int)e;                                                                         \
             configured = true;                                                                                           \
         }                                                                                                                \
-        cj::launch(latent_flash_kernel<K_, V_>, grid, dim3(THREADS), smem, stream, (const __nv_bfloat16*)q, (__nv_bfloat16*)out, \
-                   (const __nv_bfloat16*)kx, (const __nv_bfloat16*)vx, req_start, req_prior, req_base, n_requests, heads, scale_log2, sink); \
+        cj::launch(latent_flash_kernel<K_, V_, E_>, grid, dim3(THREADS), smem, stream, (const __nv_bfloat16*)q, (__nv_bfloat16*)out, \
+                   (const __nv_bfloat16*)kx, (const __nv_bfloat16*)vx, req_start, req_prior, req_base, n_requests, heads, window, scale_log2, sink); \
         return launch_status();                                                                                          \
     }
+#define LAUNCH(K_, V_) { if (exact) LAUNCH_ONE(K_, V_, true) else LAUNCH_ONE(K_, V_, false) }
     if (DV == 64) {
         if (DK == 64) LAUNCH(64, 64)
         if (DK == 128) LAUNCH(128, 64)
@@ -378,14 +403,15 @@ CJ_EXPORT int cj_latent_flash(const void* q, void* out, const void* kx, const vo
         if (DK == 256) LAUNCH(256, 128)
     }
 #undef LAUNCH
+#undef LAUNCH_ONE
     return CJ_ERR_SIZE;
 }
 
-CJ_EXPORT int cj_latent_gate_rows(const void* o, int DV, const float* gate, int ld_gate, int heads, int vdim, void* out, int T,
+CJ_EXPORT int cj_latent_gate_rows(const void* o, int DV, const float* gate, int ld_gate, int by_entry, int heads, int vdim, void* out, int T,
                                   cudaStream_t stream) {
     if (T <= 0) return 0;
     if (!o || !out || heads <= 0 || vdim <= 0 || DV < vdim) return CJ_ERR_ARG;
     cj::launch(latent_gate_rows_kernel, dim3(T), dim3(heads * vdim >= 2048 ? 256 : 128), 0, stream, (const __nv_bfloat16*)o, DV, gate,
-               ld_gate, heads, vdim, (__nv_bfloat16*)out);
+               ld_gate, by_entry, heads, vdim, (__nv_bfloat16*)out);
     return launch_status();
 }

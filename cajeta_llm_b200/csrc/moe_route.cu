@@ -108,15 +108,19 @@ __global__ void __launch_bounds__(ROUTER_THREADS) router_logits_kernel(
 __device__ __forceinline__ void select_row(const float* row, int t, int E, int k, int norm_topk, int* __restrict__ sel,
                                            float* __restrict__ w, float* __restrict__ shared_scale, float* probs, int lane,
                                            const int* __restrict__ pin, float* __restrict__ gap,
-                                           const float* __restrict__ corr, float wscale) {
+                                           const float* __restrict__ corr, float wscale, float norm_floor) {
     if (shared_scale && lane == 0) shared_scale[t] = 1.0f / (1.0f + expf(-row[E]));
     // bit 1 of norm_topk: an expert's score is the sigmoid of its own logit instead of the
     // softmax over all experts (bit 0 still asks for the picked scores to be renormalised)
     const bool sigmoid_scores = (norm_topk & 2) != 0;
     // bits 4-15: the experts form that many equal groups of neighbours (0 or 1: no groups), bits 16-27:
     // only the experts of that many groups - those whose best score is largest - can be picked
+    // bit 2: a group's score is the sum of its two largest scores (a group of one: its only score)
     const int n_groups = (norm_topk >> 4) & 0xfff, keep_groups = (norm_topk >> 16) & 0xfff;
+    const bool group_top2 = (norm_topk & 4) != 0;
     norm_topk &= 1;
+    // norm_floor > 0: a renormalisation divides by the picks' sum plus it, else by the sum clamped at 2^-14
+    auto divisor = [norm_floor](float total) { return norm_floor > 0.0f ? total + norm_floor : (total < 0.00006103515625f ? 0.00006103515625f : total); };
     if (sigmoid_scores) {
         for (int e = lane; e < E; e += 32) probs[e] = 1.0f / (1.0f + expf(-row[e]));
     } else {
@@ -145,22 +149,27 @@ __device__ __forceinline__ void select_row(const float* row, int t, int E, int k
                 total += p;
             }
             if (norm_topk) {
-                if (total < 0.00006103515625f) total = 0.00006103515625f;
+                total = divisor(total);
                 for (int j = 0; j < k; ++j) w[t * k + j] = w[t * k + j] / total * wscale;
             }
         }
         return;
     }
     if (n_groups > 1 && keep_groups < n_groups) {
-        // the groups with the smallest best score leave one by one (of equal ones the later group
+        // the groups with the smallest score leave one by one (of equal ones the later group
         // first): their experts' scores become -1, which no pick takes
         const int per = E / n_groups;
         for (int drop = n_groups - keep_groups; drop > 0; --drop) {
             float wm = 0.0f;
             int worst = -1;
             for (int g = lane; g < n_groups; g += 32) {
-                float m = -1.0f;
-                for (int i = 0; i < per; ++i) m = fmaxf(m, probs[g * per + i]);
+                float m = -1.0f, second = -1.0f;
+                for (int i = 0; i < per; ++i) {
+                    const float p = probs[g * per + i];
+                    second = fmaxf(second, fminf(m, p));
+                    m = fmaxf(m, p);
+                }
+                if (group_top2 && second >= 0.0f) m += second;
                 if (m >= 0.0f && (worst < 0 || m <= wm)) { worst = g; wm = m; }
             }
 #pragma unroll
@@ -222,7 +231,7 @@ __device__ __forceinline__ void select_row(const float* row, int t, int E, int k
         if (lane == 0) gap[t] = (k < E && last > 0.0f) ? (last - next) / last : 1.0f;
     }
     if (norm_topk) {
-        if (wsum < 0.00006103515625f) wsum = 0.00006103515625f;
+        wsum = divisor(wsum);
         if (lane < k) w[t * k + lane] = mine / wsum * wscale;
         if (lane == 0)
             for (int j = 32; j < k; ++j) w[t * k + j] = w[t * k + j] / wsum * wscale;
@@ -241,7 +250,7 @@ __global__ void __launch_bounds__(SMALL_ROWS * 32) router_small_kernel(
     const float* __restrict__ x, const float* __restrict__ Wr, const float* __restrict__ shared_gate, int T, int H,
     int E, int k, int norm_topk, float* __restrict__ logits, int* __restrict__ sel, float* __restrict__ w,
     float* __restrict__ shared_scale, int* __restrict__ tickets, const int* __restrict__ pin, float* __restrict__ gap,
-    const float* __restrict__ corr, float wscale) {
+    const float* __restrict__ corr, float wscale, float norm_floor) {
     cj::release_successor();
     __shared__ float probs[SMALL_ROWS][MAX_EXPERTS];
     __shared__ int is_last;
@@ -307,18 +316,18 @@ __global__ void __launch_bounds__(SMALL_ROWS * 32) router_small_kernel(
     if (!is_last) return;
     __threadfence();
     if (t < T) {
-        select_row(logits + (size_t)t * n_cols, t, E, k, norm_topk, sel, w, shared_scale, probs[warp], lane, pin, gap, corr, wscale);
+        select_row(logits + (size_t)t * n_cols, t, E, k, norm_topk, sel, w, shared_scale, probs[warp], lane, pin, gap, corr, wscale, norm_floor);
     }
 }
 
 __global__ void __launch_bounds__(32) router_select_kernel(
     const float* __restrict__ logits, int E, int n_cols, int k, int norm_topk, int* __restrict__ sel,
     float* __restrict__ w, float* __restrict__ shared_scale, const int* __restrict__ pin, float* __restrict__ gap,
-    const float* __restrict__ corr, float wscale) {
+    const float* __restrict__ corr, float wscale, float norm_floor) {
     cj::after_predecessor();
     cj::release_successor();
     __shared__ float probs[MAX_EXPERTS];
-    select_row(logits + (size_t)blockIdx.x * n_cols, blockIdx.x, E, k, norm_topk, sel, w, shared_scale, probs, threadIdx.x, pin, gap, corr, wscale);
+    select_row(logits + (size_t)blockIdx.x * n_cols, blockIdx.x, E, k, norm_topk, sel, w, shared_scale, probs, threadIdx.x, pin, gap, corr, wscale, norm_floor);
 }
 
 // The selection from logits that a product split along K left as partial sums
@@ -329,7 +338,7 @@ __global__ void __launch_bounds__(SELECT_ROWS * 32) router_select_partials_kerne
     const float* __restrict__ partials, int n_partials, long long partial_stride, int ld, int T, int E, int k,
     int norm_topk, int* __restrict__ sel, float* __restrict__ w, float* __restrict__ shared_scale,
     const int* __restrict__ pin, float* __restrict__ gap,
-    const float* __restrict__ corr, float wscale) {
+    const float* __restrict__ corr, float wscale, float norm_floor) {
     cj::after_predecessor();
     cj::release_successor();
     __shared__ float probs[SELECT_ROWS][MAX_EXPERTS];
@@ -344,7 +353,7 @@ __global__ void __launch_bounds__(SELECT_ROWS * 32) router_select_partials_kerne
         row[warp][e] = v;
     }
     __syncwarp();
-    select_row(row[warp], t, E, k, norm_topk, sel, w, shared_scale, probs[warp], lane, pin, gap, corr, wscale);
+    select_row(row[warp], t, E, k, norm_topk, sel, w, shared_scale, probs[warp], lane, pin, gap, corr, wscale, norm_floor);
 }
 
 // Counting sort of the picks (token t, choice j) by expert, stable.  One block per
@@ -427,9 +436,10 @@ __global__ void __launch_bounds__(GROUP_WARPS * 32) moe_group_kernel(
 // tickets: int32 [4], zero before the first use (the kernel leaves them zero); may be null, the two-launch form is then used.
 // pin: int32 [T, k] experts given instead of chosen, or null.  gap: float32 [T] routing margins out, or null.
 // correction: float32 [E] added to the scores for the choice alone, or null.  weight_scale: multiplies the picks' weights.
+// norm_floor: see select_row.
 CJ_EXPORT int cj_router_topk(const float* x, const float* Wr, const float* shared_gate, int T, int H, int E, int k,
                              int norm_topk, int* sel, float* w, float* shared_scale, float* logits, int* tickets,
-                             const int* pin, float* gap, const float* correction, float weight_scale, cudaStream_t stream) {
+                             const int* pin, float* gap, const float* correction, float weight_scale, float norm_floor, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (!x || !Wr || !sel || !w || !logits || H <= 0) return CJ_ERR_ARG;
     if (shared_gate && !shared_scale) return CJ_ERR_ARG;
@@ -438,7 +448,7 @@ CJ_EXPORT int cj_router_topk(const float* x, const float* Wr, const float* share
     if (T <= 32 && tickets) {
         dim3 grid_small(n_cols, (T + SMALL_ROWS - 1) / SMALL_ROWS);
         cj::launch(router_small_kernel, dim3(grid_small), dim3(SMALL_ROWS * 32), 0, stream, x, Wr, shared_gate, T, H, E, k, norm_topk, logits, sel, w,
-                                                                         shared_gate ? shared_scale : nullptr, tickets, pin, gap, correction, weight_scale);
+                                                                         shared_gate ? shared_scale : nullptr, tickets, pin, gap, correction, weight_scale, norm_floor);
         return launch_status();
     }
     // rows of x staged per block: as many as fit 200 KB of shared memory, at most 8
@@ -465,19 +475,19 @@ CJ_EXPORT int cj_router_topk(const float* x, const float* Wr, const float* share
     int st = launch_status();
     if (st) return st;
     cj::launch(router_select_kernel, dim3(T), dim3(32), 0, stream, logits, E, n_cols, k, norm_topk, sel, w, shared_gate ? shared_scale : nullptr,
-               pin, gap, correction, weight_scale);
+               pin, gap, correction, weight_scale, norm_floor);
     return launch_status();
 }
 
 // partials: [n_partials][T][ld] float32 logits (column E the shared gate's dot when shared_scale is given).
 CJ_EXPORT int cj_router_select(const float* partials, int n_partials, long long partial_stride, int ld, int T, int E, int k,
                                int norm_topk, int* sel, float* w, float* shared_scale, const int* pin, float* gap,
-                               const float* correction, float weight_scale, cudaStream_t stream) {
+                               const float* correction, float weight_scale, float norm_floor, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (!partials || !sel || !w || n_partials < 1) return CJ_ERR_ARG;
     if (E < 1 || E > MAX_EXPERTS || k < 1 || k > E || ld < E + (shared_scale ? 1 : 0)) return CJ_ERR_SIZE;
     cj::launch(router_select_partials_kernel, dim3((T + SELECT_ROWS - 1) / SELECT_ROWS), dim3(SELECT_ROWS * 32), 0, stream, 
-        partials, n_partials, partial_stride, ld, T, E, k, norm_topk, sel, w, shared_scale, pin, gap, correction, weight_scale);
+        partials, n_partials, partial_stride, ld, T, E, k, norm_topk, sel, w, shared_scale, pin, gap, correction, weight_scale, norm_floor);
     return launch_status();
 }
 

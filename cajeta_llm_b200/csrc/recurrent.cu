@@ -20,7 +20,6 @@
 //                      o = S^T q / (max(|n . q|, e^(-m_t)) + floor)
 //   gated_scan         S_t = (1 - z_t) S_(t-1) + z_t c_t per channel, out = S_t silu(g_t) (minGRU: gates of the current token only)
 //   rmsnorm_mix2       out (+)= c (a / rms(a) * wa + b / rms(b) * wb)
-//   relu2_rows         max(x, 0)^2 into the activation dtype
 //   softcap_rows       x <- cap tanh(x / cap), float32 in place (a head whose logits are capped)
 //   gated_group_norm   y * silu(z) (or sigmoid(z)) and RMS over equal parts of a row, in either order
 //
@@ -513,17 +512,6 @@ __global__ void rmsnorm_mix2_kernel(const float* __restrict__ a, const float* __
     }
 }
 
-// max(x, 0)^2 into the activation dtype (the activation of an ungated expert whose product was stored in float32)
-template <typename TO>
-__global__ void relu2_rows_kernel(const float* __restrict__ x, TO* __restrict__ out, long long n) {
-    cj::after_predecessor();
-    cj::release_successor();
-    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
-        const float v = fmaxf(x[i], 0.0f);
-        out[i] = from_f32<TO>(v * v);
-    }
-}
-
 // x <- cap tanh(x / cap), in place, float32
 __global__ void softcap_rows_kernel(float* __restrict__ x, float cap, long long n) {
     cj::after_predecessor();
@@ -932,17 +920,6 @@ CJ_EXPORT int cj_rmsnorm_mix2(const float* a, const float* wa, const float* b, c
     if (!a || !wa || !b || !wb || !out || H <= 0) return CJ_ERR_ARG;
     int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
     cj::launch(rmsnorm_mix2_kernel, dim3(rows), dim3(threads), 0, stream, a, wa, b, wb, eps, c, accumulate, out, H);
-    return launch_status();
-}
-
-CJ_EXPORT int cj_relu2_rows(const float* x, void* out, int out_dtype, long long n, cudaStream_t stream) {
-    if (n <= 0) return 0;
-    if (!x || !out) return CJ_ERR_ARG;
-    long long blocks = (n + 255) / 256;
-    if (blocks > 148 * 16) blocks = 148 * 16;
-    if (out_dtype == CJ_F32) cj::launch(relu2_rows_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, x, (float*)out, n);
-    else if (out_dtype == CJ_BF16) cj::launch(relu2_rows_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(256), 0, stream, x, (__nv_bfloat16*)out, n);
-    else return CJ_ERR_DTYPE;
     return launch_status();
 }
 

@@ -4,7 +4,7 @@
 residual stream ``hs`` in float32 (model/DecoderLayer.cajeta:38-75,
 model/CausalLM.cajeta:1445-1446,1506,1512-1517,1575).  Parameters: the tensor-name
 pieces ``mixer_norm_name``, ``feed_forward_norm_name``, ``mixer_name``,
-``feed_forward_name`` under the layer's prefix.
+``feed_forward_name`` under the layer's prefix.  A layer may have no feed-forward (the file may then hold its norm or not).
 
 ``outnorm``: the norm sits on each sublayer's OUTPUT and the sublayers read the stream
 itself: ``hs += norm_1(mixer(hs)); hs += norm_2(feed_forward(hs))``.  A layer may have no
@@ -74,20 +74,30 @@ class PreNormBlock(Part):
         super().__init__(spec, prefix, runtime)
         self.mixer_norm = make_part("norm", layer.mixer_norm, self.name(spec["mixer_norm_name"]), runtime)
         self.mixer = make_part("mixer", layer.mixer, self.name(spec["mixer_name"]), runtime)
-        self.feed_forward_norm = make_part("norm", layer.feed_forward_norm, self.name(spec["feed_forward_norm_name"]), runtime)
-        self.feed_forward = make_part("feed_forward", layer.feed_forward, self.name(spec["feed_forward_name"]), runtime)
+        if hasattr(self.mixer, "allow_pending"):
+            self.mixer.allow_pending = True
+        self.feed_forward = self.feed_forward_norm = None
+        self.idle_norm = None              # the name of the second norm's weight in a layer without a feed-forward: nothing reads it
+        if layer.feed_forward is not None:
+            self.feed_forward_norm = make_part("norm", layer.feed_forward_norm, self.name(spec["feed_forward_norm_name"]), runtime)
+            self.feed_forward = make_part("feed_forward", layer.feed_forward, self.name(spec["feed_forward_name"]), runtime)
+        else:
+            self.idle_norm = self.name(spec["feed_forward_norm_name"])
 
     def parts(self):
-        return (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward)
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward) if p is not None)
 
     def params(self) -> Dict[str, ParamSpec]:
         out: Dict[str, ParamSpec] = {}
         for p in self.parts():
             out.update(p.params())
+        if self.idle_norm is not None:
+            spec = next(iter(self.mixer_norm.params().values()))
+            out[self.idle_norm] = ParamSpec(spec.shape, role=spec.role, init=spec.init, optional=True)
         return out
 
     def libraries(self) -> set:
-        out = set()
+        out = {"stream_ops"} if self.feed_forward is None else set()
         for p in self.parts():
             out |= p.libraries()
         return out
@@ -104,6 +114,12 @@ class PreNormBlock(Part):
         # the feed-forward may want its input once more in float32 (a router), or, for many
         # rows, as three bfloat16 terms that a tensor-core product can sum to the same grade
         ff = self.feed_forward
+        if ff is None:
+            if pending is not None:
+                K.tag = "partial sums"
+                K.add_partials(hs, pending)
+                K.tag = None
+            return
         wants_split = getattr(ff, "wants_split_input", None)
         split = bool(wants_split and wants_split(hs.shape[0]))
         x, x_exact = self.feed_forward_norm.forward(hs, want_f32=getattr(ff, "needs_f32_input", False) and not split,

@@ -1,15 +1,17 @@
-"""Feed-forward parts: the dense SwiGLU MLP, a dense one with a squared ReLU, and the sparse mixture of experts.
+"""Feed-forward parts: the dense gated MLP (SwiGLU and its like), a dense one with a squared ReLU, and the sparse mixture of experts.
 
 ``dense_swiglu``: ``W_d (silu(W_g x) * (W_u x))``, ``silu(x) = x / (1 + exp(-x))``
 (model/Prim.cajeta:1822-1847, model/CausalLM.cajeta:1556-1566).  Parameters:
 ``hidden_size``, ``intermediate_size``, ``names`` (optional: the tensor names of
-``gate``, ``up`` and ``down`` under the part's prefix).
+``gate``, ``up`` and ``down`` under the part's prefix).  ``dense_gated`` is the same part with its two options:
+``activation`` (``silu``, the default, or ``gelu_tanh``, gelu's tanh form) and ``bias`` (every projection has one, under its
+weight's name with ``.b`` added; gate's and up's are added before the activation, in the product's epilogue).
 
 ``dense_relu2``: ``W_d max(W_u x, 0)^2``, a feed-forward without a gate whose activation is the square of the
 rectified sum.  Parameters: ``hidden_size``, ``intermediate_size``, ``names`` (``up``, ``down``), ``bias`` (optional: both products
 have a bias, under the weight's name with ``.b`` added).  A block may set ``out_scale`` (multiplies the result as it is added)
-and ``allow_pending`` (few rows: partial sums are handed back instead of added).  On the tensor-core
-path the square is the up-product's epilogue (the float32 sum squared, then rounded); elsewhere a kernel of its own.
+and ``allow_pending`` (few rows: partial sums are handed back instead of added).  The square is the up-product's epilogue (the
+float32 sum squared, then rounded).
 
 ``sparse_moe``: router logits ``l_e = Wr[e] . x`` in float32, softmax over all experts,
 top-k by repeated strict-``>`` argmax (ties to the lower index), weights = the picked
@@ -37,12 +39,14 @@ the weight multiplying the float32 row before it is rounded for the products);
 ``u = clamp(W_u x, -L, L)``, ``W_d (g sigmoid(a g) (u + 1))`` instead of SwiGLU; ``shared_act_limit`` /
 ``shared_act_alpha``: the same for the shared expert (default: the experts');
 ``route_groups`` ``(count, keep)``: the experts form ``count`` equal groups of neighbours, a group's
-score is its largest score, and only experts of the ``keep`` best groups can be picked;
+score is its largest score (``group_score`` ``top2``: the sum of its two largest), and only experts of the ``keep`` best groups
+can be picked;
 ``activation`` ``relu2``: an expert has no gate, ``W_d max(W_u x, 0)^2`` (tensors ``up`` and ``down`` only;
-built without a shared expert and with the weight on the output);
+built with the weight on the output); ``gelu``: the same with gelu by the error function.  A shared expert has the experts' form;
 ``correction``: a tensor name, ``[num_experts]``: a number per expert that is added to its score for the CHOICE of the
 ``top_k`` experts alone, a pick's weight staying its score without it; ``route_scale``: multiplies the picks'
-weights (after a renormalisation, when one is asked for).
+weights (after a renormalisation, when one is asked for); ``norm_floor`` e > 0: a renormalisation divides by the picks' sum plus
+e instead of by the clamped sum.
 
 The file stores one tensor per expert and projection
 (``experts.{e}.gate_proj.weight`` ...); they are stacked into ``[E, I, H]`` and
@@ -57,10 +61,14 @@ import torch
 
 from ..csrc import kernels as K
 from .base import Part, register_part
-from .linear import project, project_split, relu2_fused, splits_few_rows
+from .linear import project, project_split, splits_few_rows
 from .plan import ParamSpec
 
 
+GATES = {"silu": (1.0, 0.0), "gelu_tanh": K.GELU_TANH}      # (alpha, cubic): g sigmoid(alpha g + cubic g^3)
+
+
+@register_part("feed_forward", "dense_gated")
 @register_part("feed_forward", "dense_swiglu")
 class DenseSwiGLU(Part):
     needs_f32_input = False
@@ -73,14 +81,25 @@ class DenseSwiGLU(Part):
         self.n_gate = self.name(names.get("gate", "gate_proj.weight"))
         self.n_up = self.name(names.get("up", "up_proj.weight"))
         self.n_down = self.name(names.get("down", "down_proj.weight"))
+        self.bias = bool(spec.get("bias", False))
+        activation = str(spec.get("activation", "silu"))
+        if activation not in GATES:
+            raise ValueError(f"activation must be one of {', '.join(sorted(GATES))}, found '{activation}'")
+        self.gate_alpha, self.gate_cubic = GATES[activation]
         self.w_gate = self.w_up = self.w_down = None
+        self.b_gate = self.b_up = self.b_down = None
 
     def params(self) -> Dict[str, ParamSpec]:
-        return {
+        p = {
             self.n_gate: ParamSpec((self.inter, self.hidden)),
             self.n_up: ParamSpec((self.inter, self.hidden)),
             self.n_down: ParamSpec((self.hidden, self.inter)),
         }
+        if self.bias:
+            for n in (self.n_gate, self.n_up):
+                p[n + ".b"] = ParamSpec((self.inter,), role="vector")
+            p[self.n_down + ".b"] = ParamSpec((self.hidden,), role="vector")
+        return p
 
     def libraries(self) -> set:
         libs = {"gemm_simt"}
@@ -92,14 +111,17 @@ class DenseSwiGLU(Part):
         self.w_gate = self.fetch(source, self.n_gate)
         self.w_up = self.fetch(source, self.n_up)
         self.w_down = self.fetch(source, self.n_down)
+        if self.bias:
+            self.b_gate, self.b_up, self.b_down = (self.fetch(source, n + ".b") for n in (self.n_gate, self.n_up, self.n_down))
 
     def forward(self, x: torch.Tensor, x_f32: Optional[torch.Tensor], residual: torch.Tensor, ctx) -> None:
         T = x.shape[0]
         act = torch.empty((T, self.inter), dtype=self.runtime.act_dtype, device=x.device)
         K.tag = "dense gate/up"
-        project(self.runtime, x, self.w_gate, act, w_up=self.w_up)
+        project(self.runtime, x, self.w_gate, act, w_up=self.w_up, bias=self.b_gate, bias_up=self.b_up, act_alpha=self.gate_alpha,
+                act_cubic=self.gate_cubic)
         K.tag = "dense down"
-        project(self.runtime, act, self.w_down, residual, accumulate=True)
+        project(self.runtime, act, self.w_down, residual, bias=self.b_down, accumulate=True)
         K.tag = None
 
 
@@ -127,7 +149,7 @@ class DenseRelu2(Part):
         return p
 
     def libraries(self) -> set:
-        libs = {"gemm_simt", "recurrent"}
+        libs = {"gemm_simt"}
         if self.runtime.fast_kernels and self.hidden >= 128:
             libs |= {"gemm_tc", "gemm_tc2"}
         return libs
@@ -147,13 +169,7 @@ class DenseRelu2(Part):
         T = x.shape[0]
         act = torch.empty((T, self.inter), dtype=rt.act_dtype, device=x.device)
         K.tag = "dense up"
-        if relu2_fused(rt, x, self.w_up, act.dtype):
-            project(rt, x, self.w_up, act, bias=self.b_up, relu2=True)
-        else:
-            pre = torch.empty((T, self.inter), dtype=torch.float32, device=x.device)
-            project(rt, x, self.w_up, pre, bias=self.b_up)
-            K.tag = "dense activation"
-            K.relu2_rows(pre, act)
+        project(rt, x, self.w_up, act, bias=self.b_up, act="relu2")
         K.tag = "dense down"
         parts = project_split(rt, act, self.w_down, bias=self.b_down, out_scale=self.out_scale) if self.allow_pending else None
         if parts is None:
@@ -187,11 +203,16 @@ class SparseMoE(Part):
         self.shared_act_limit = float(spec.get("shared_act_limit", self.act_limit) or 0.0)
         self.shared_act_alpha = float(spec.get("shared_act_alpha", self.act_alpha))
         self.activation = str(spec.get("activation", "swiglu"))
-        if self.activation not in ("swiglu", "relu2"):
-            raise ValueError(f"activation must be 'swiglu' or 'relu2', found '{self.activation}'")
+        if self.activation not in ("swiglu", "relu2", "gelu"):
+            raise ValueError(f"activation must be 'swiglu', 'relu2' or 'gelu', found '{self.activation}'")
         self.gated = self.activation == "swiglu"
-        if not self.gated and (self.shared_inter > 0 or self.weight_on != "output" or self.act_limit > 0.0):
-            raise ValueError("ungated experts are built without a shared expert, capped gates or the weight on the input")
+        if not self.gated and (self.weight_on != "output" or self.act_limit > 0.0):
+            raise ValueError("ungated experts are built without capped gates or the weight on the input")
+        self.projections = ("gate", "up", "down") if self.gated else ("up", "down")
+        self.group_score = str(spec.get("group_score", "largest"))
+        if self.group_score not in ("largest", "top2"):
+            raise ValueError(f"group_score must be 'largest' or 'top2', found '{self.group_score}'")
+        self.norm_floor = float(spec.get("norm_floor", 0.0) or 0.0)
         self.n_correction = self.name(str(spec["correction"])) if spec.get("correction") else None
         self.route_scale = float(spec.get("route_scale", 1.0))
         self.correction = None
@@ -232,7 +253,8 @@ class SparseMoE(Part):
             p[self.expert_name("up", e)] = ParamSpec((self.inter, self.hidden))
             p[self.expert_name("down", e)] = ParamSpec((self.hidden, self.inter))
         if self.shared_inter > 0:
-            p[self.n_shared["gate"]] = ParamSpec((self.shared_inter, self.hidden))
+            if self.gated:
+                p[self.n_shared["gate"]] = ParamSpec((self.shared_inter, self.hidden))
             p[self.n_shared["up"]] = ParamSpec((self.shared_inter, self.hidden))
             p[self.n_shared["down"]] = ParamSpec((self.hidden, self.shared_inter))
             if self.shared_gate:
@@ -243,7 +265,7 @@ class SparseMoE(Part):
         return self.name(self.n_expert[proj].format(e=e))
 
     def libraries(self) -> set:
-        libs = {"rowwise", "moe_route", "gemm_simt"} | ({"recurrent"} if self.weight_on == "input" or not self.gated else set())
+        libs = {"rowwise", "moe_route", "gemm_simt"} | ({"recurrent"} if self.weight_on == "input" else set())
         if self.runtime.fast_kernels and self.hidden >= 128:
             libs |= {"gemm_tc", "gemm_tc2"}
         return libs
@@ -266,12 +288,13 @@ class SparseMoE(Part):
         self.w_up = slab("up", I, self.hidden)
         self.w_down = slab("down", self.hidden, I)
         if self.shared_inter > 0:
-            ws_gate = self.fetch(source, self.n_shared["gate"])
+            ws_gate = self.fetch(source, self.n_shared["gate"]) if self.gated else None
             ws_up = self.fetch(source, self.n_shared["up"])
             ws_down = self.fetch(source, self.n_shared["down"])
             if C > 0:
                 # chunk c of the shared expert: rows [c I, (c + 1) I) of gate and up, columns of down
-                self.w_gate[E:].copy_(ws_gate.view(C, I, self.hidden))
+                if self.gated:
+                    self.w_gate[E:].copy_(ws_gate.view(C, I, self.hidden))
                 self.w_up[E:].copy_(ws_up.view(C, I, self.hidden))
                 self.w_down[E:].copy_(ws_down.view(self.hidden, C, I).permute(1, 0, 2))
                 if rt.fast_kernels:
@@ -337,11 +360,11 @@ class SparseMoE(Part):
                       k_splits=splits)
             K.router_select(logits, self.num_experts, k, self.norm_topk, sel, wts, shared_scale, pin=pin, gap=gap,
                             sigmoid_scores=self.score == "sigmoid", groups=self.route_groups, correction=self.correction,
-                            weight_scale=self.route_scale)
+                            weight_scale=self.route_scale, group_top2=self.group_score == "top2", norm_floor=self.norm_floor)
         else:
             K.router_topk(x_exact, self.router, self.shared_gate_w, k, self.norm_topk, sel, wts, shared_scale, pin=pin, gap=gap,
                           sigmoid_scores=self.score == "sigmoid", groups=self.route_groups, correction=self.correction,
-                          weight_scale=self.route_scale)
+                          weight_scale=self.route_scale, group_top2=self.group_score == "top2", norm_floor=self.norm_floor)
 
     def forward(self, x: torch.Tensor, x_exact: torch.Tensor, residual: torch.Tensor, ctx) -> None:
         rt = self.runtime
@@ -393,17 +416,10 @@ class SparseMoE(Part):
             project(rt, scaled, self.w_gate[:G], act, w_up=self.w_up[:G], group_offsets=offsets, max_group_rows=T,
                     offsets_settled=True, act_limit=self.act_limit, act_alpha=self.act_alpha)
             wts = torch.ones_like(wts)
-        elif not self.gated and relu2_fused(rt, x, self.w_up, act.dtype):
-            # an expert without a gate: the rectified float32 sum is squared in the product's epilogue, then rounded
-            K.tag = "experts up"
-            project(rt, x, self.w_up[:G], act, group_offsets=offsets, a_row_index=slot_token, max_group_rows=T, relu2=True)
         elif not self.gated:
-            # the float32 path: the product, then the activation, as two kernels
-            pre = torch.empty((n_slots, self.inter), dtype=torch.float32, device=dev)
+            # an expert without a gate: the activation of the float32 sum in the product's epilogue, then rounded
             K.tag = "experts up"
-            project(rt, x, self.w_up[:G], pre, group_offsets=offsets, a_row_index=slot_token, max_group_rows=T)
-            K.tag = "experts activation"
-            K.relu2_rows(pre, act)
+            project(rt, x, self.w_up[:G], act, group_offsets=offsets, a_row_index=slot_token, max_group_rows=T, act=self.activation)
         else:
             K.tag = "experts gate/up"
             project(rt, x, self.w_gate[:G], act, w_up=self.w_up[:G], group_offsets=offsets, a_row_index=slot_token,
@@ -418,12 +434,16 @@ class SparseMoE(Part):
         elif self.shared_inter > 0:
             sact = torch.empty((T, self.shared_inter), dtype=rt.act_dtype, device=dev)
             if shared_dense:
-                ws_gate = self.w_gate[E:].view(self.shared_inter, self.hidden)
+                ws_gate = self.w_gate[E:].view(self.shared_inter, self.hidden) if self.gated else None
                 ws_up = self.w_up[E:].view(self.shared_inter, self.hidden)
             else:
                 ws_gate, ws_up = self.ws_gate, self.ws_up
-            K.tag = "shared gate/up"
-            project(rt, x, ws_gate, sact, w_up=ws_up, act_limit=self.shared_act_limit, act_alpha=self.shared_act_alpha)
+            if self.gated:
+                K.tag = "shared gate/up"
+                project(rt, x, ws_gate, sact, w_up=ws_up, act_limit=self.shared_act_limit, act_alpha=self.shared_act_alpha)
+            else:
+                K.tag = "shared up"
+                project(rt, x, ws_up, sact, act=self.activation)
             shared = torch.empty((T, self.hidden), dtype=torch.float32, device=dev)
             K.tag = "shared down"
             project(rt, sact, self.ws_down, shared)

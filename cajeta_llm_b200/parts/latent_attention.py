@@ -13,7 +13,7 @@ entries, values of ``vdim``, latent of ``kv_rank``::
     (the gate is optional, and so are a latent of the queries' own and a sink in the softmax: see the parameters)
 
 The rotation pairs entries (2i, 2i+1) of the first ``rotary_dim`` entries of the rotated
-part (the position part's ``rotary_dim`` and ``inv_freq``).  Nothing per head is built from
+part (the position part's ``rotary_dim`` and ``inv_freq``; cos and sin times its ``magnitude``).  Nothing per head is built from
 the cache: ``W_uk[h]^T q`` is taken on the query's side and ``W_uv[h]`` applied to the
 weighted sum of latents, so the attention kernel reads each cache entry once for all
 heads.  Steps that carry long prompt portions on the bfloat16 path take the plain form
@@ -34,7 +34,12 @@ Optional, each off by default:
 ``q_rank`` n > 0: the queries pass a latent of their own, ``c_q = rms(W_dq x) * w`` (``dq``, ``dq.norm``; the layer's
 eps), ``q = W_uq c_q`` (``uq``), instead of one projection ``q``; ``W_dq`` rides in the mixer's one input product,
 a kernel norms its columns, a second product brings the heads up;
-``gate`` false: no sigmoid gate on the heads' outputs (no tensor ``g``);
+``gate`` false: no sigmoid gate on the heads' outputs (no tensor ``g``); ``"entries"``: a gate for every entry of the heads side by
+side (``g`` has ``heads * vdim`` rows) instead of one per head;
+``halves``: the rotation pairs entries i and i + rotary_dim / 2;
+``window`` n > 0: a row sees its last n positions alone; the cache group gives pages behind the window back, and the plain form
+gathers a request's tokens from the oldest one that its rows of the step still see;
+``exact_weights``: the plain form's softmax weights enter the product with the values as two bfloat16 terms (float32 to 2^-17);
 ``sink``: a tensor name, ``[heads]``: the softmax's divisor also holds ``exp(sink[h])``, a term without key or value
 that is neither scaled nor rotated and counts once.
 """
@@ -47,7 +52,7 @@ import torch
 
 from ..csrc import kernels as K
 from .base import KvNeed, Part, make_part, register_part
-from .linear import project
+from .linear import project, project_split
 from .plan import ParamSpec
 
 
@@ -67,11 +72,23 @@ class LatentAttention(Part):
         self.eps = float(spec["eps"])
         self.owns_cache = bool(spec.get("owns_cache", True))
         self.q_rank = int(spec.get("q_rank", 0) or 0)
-        self.gate = bool(spec.get("gate", True))
+        gate = spec.get("gate", True)
+        if gate not in (True, False, "entries"):
+            raise ValueError(f"gate must be true, false or 'entries', found {gate!r}")
+        self.gate = bool(gate)
+        self.gate_by_entry = gate == "entries"
+        self.gate_cols = 0 if not gate else (self.heads * self.vdim if self.gate_by_entry else self.heads)
+        self.halves = bool(spec.get("halves", False))
+        self.window = int(spec.get("window", 0) or 0)
+        if self.window < 0:
+            raise ValueError(f"window must be positive (or 0 for none), found {self.window}")
+        self.exact_weights = bool(spec.get("exact_weights", False))
+        self.allow_pending = False         # a block that takes partial sums from its mixer sets this True
         self.n_sink = self.name(str(spec["sink"])) if spec.get("sink") else None
         self.sink = self.w_qnorm = self.w_uq = None
         self.position = make_part("position", spec["position"], prefix, runtime)
         self.rotary = int(self.position.rotary_dim)
+        self.magnitude = float(getattr(self.position, "magnitude", 1.0))
         if self.rotary > self.rot:
             raise ValueError(f"the position part rotates {self.rotary} entries; the rotated part has {self.rot}")
         if self.rank > 1024:
@@ -90,7 +107,7 @@ class LatentAttention(Part):
         return self.EXPAND_MIN_ROWS - 1 if self.can_expand else 1 << 30
 
     def cache_need(self) -> Optional[KvNeed]:
-        return KvNeed(1, self.rank + self.rot, 0, values=False)
+        return KvNeed(1, self.rank + self.rot, self.window, values=False)
 
     def state_need(self):
         return None
@@ -108,7 +125,7 @@ class LatentAttention(Part):
         else:
             p[self.name("q")] = ParamSpec((self.nq, self.hidden))
         if self.gate:
-            p[self.name("g")] = ParamSpec((self.heads, self.hidden))
+            p[self.name("g")] = ParamSpec((self.gate_cols, self.hidden))
         if self.n_sink:
             p[self.n_sink] = ParamSpec((self.heads,), role="vector", std=1.0)
         if self.owns_cache:
@@ -143,7 +160,7 @@ class LatentAttention(Part):
         self.w_uv = self.fetch(source, self.name("uv")).view(self.heads, self.vdim, self.rank).contiguous()
         self.w_o = self.fetch(source, self.name("o"))
 
-    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, entry) -> None:
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, entry) -> Optional[torch.Tensor]:
         rt = self.runtime
         dev = x.device
         T, H = x.shape[0], self.heads
@@ -152,7 +169,7 @@ class LatentAttention(Part):
             raise ValueError(f"{self.prefix}: the plan lets this entry write a cache, but the part has no W_dkv")
         n_q = self.q_rank or self.nq
         gate_off = n_q
-        d_off = n_q + (H if self.gate else 0)
+        d_off = n_q + self.gate_cols
         n_out = d_off + ((self.rank + self.rot) if write else 0)
         proj = torch.empty((T, n_out), dtype=torch.float32, device=dev)
         K.tag = "mixer in"
@@ -170,15 +187,18 @@ class LatentAttention(Part):
         if write:
             K.tag = "latent norm + rope + cache write"
             K.latent_kv_write(proj, d_off, self.rank, self.rot, self.rotary, self.w_norm, self.eps, inv_freq,
-                              ctx.positions, ctx.row_req, entry.block_table, entry.page_tokens, entry.k_plane)
+                              ctx.positions, ctx.row_req, entry.block_table, entry.page_tokens, entry.k_plane, halves=self.halves,
+                              magnitude=self.magnitude)
         if self.can_expand and T >= self.EXPAND_MIN_ROWS and not ctx.all_single and len(ctx.h_req_prior) > 0:
             gated = self._plain_form(q, gate, ctx, entry)
         else:
             gated = self._absorbed_form(q, gate, ctx, entry)
         K.tag = "o"
-        project(rt, gated, self.w_o, residual, accumulate=True)
+        parts = project_split(rt, gated, self.w_o) if self.allow_pending else None
+        if parts is None:
+            project(rt, gated, self.w_o, residual, accumulate=True)
         K.tag = None
-        return None
+        return parts
 
     def _absorbed_form(self, proj: torch.Tensor, gate, ctx, entry) -> torch.Tensor:
         """``proj``: float32 rows whose first ``heads * (dim + rot_dim)`` columns are the queries; ``gate``: (matrix, column)
@@ -190,7 +210,8 @@ class LatentAttention(Part):
         q_plain = torch.empty((H * T, self.dim), dtype=rt.act_dtype, device=dev)
         q_rot = torch.empty((T, H, self.rot), dtype=torch.float32, device=dev)
         K.tag = "q split + rope"
-        K.latent_q_split(proj, H, self.dim, self.rot, self.rotary, inv_freq, ctx.positions, q_plain, q_rot)
+        K.latent_q_split(proj, H, self.dim, self.rot, self.rotary, inv_freq, ctx.positions, q_plain, q_rot, halves=self.halves,
+                         magnitude=self.magnitude)
         # rows are head-major: group h of the grouped products is head h's T rows
         offsets = torch.arange(0, (H + 1) * T, T, dtype=torch.int32, device=dev)
         q_abs = torch.empty((H * T, self.rank), dtype=torch.float32, device=dev)
@@ -204,31 +225,35 @@ class LatentAttention(Part):
         # stretches a row's keys are cut when the step has few rows.
         reach = ctx.max_context if ctx.all_single else entry.block_table.shape[1] * entry.page_tokens
         K.latent_attention(q_abs, q_rot, entry.k_plane, self.rank, self.rot, H, ctx.positions, ctx.row_req, entry.block_table,
-                           entry.page_tokens, self.scale, lat, max_context=reach, sink=self.sink)
+                           entry.page_tokens, self.scale, lat, max_context=reach, sink=self.sink, window=self.window)
         o = torch.empty((H * T, self.vdim), dtype=torch.float32, device=dev)
         K.tag = "value up"
         project(rt, lat, self.w_uv, o, group_offsets=offsets, max_group_rows=T, offsets_settled=True)
         gated = torch.empty((T, H * self.vdim), dtype=rt.act_dtype, device=dev)
         K.tag = "head gate" if gate[0] is not None else "heads out"
-        K.latent_gate_out(o, gate[0], gate[1], H, self.vdim, gated)
+        K.latent_gate_out(o, gate[0], gate[1], H, self.vdim, gated, by_entry=self.gate_by_entry)
         return gated
 
     def _plain_form(self, proj: torch.Tensor, gate, ctx, entry) -> torch.Tensor:
         rt = self.runtime
         dev = proj.device
         T, H = proj.shape[0], self.heads
-        layout = getattr(ctx, "_latent_tokens", None)
+        layouts = ctx.__dict__.setdefault("_latent_tokens", {})
+        layout = layouts.get(self.window)
         if layout is None:
-            # every token of the step's requests, cached and new, request after request (shared by the step's layers)
+            # the tokens of the step's requests, cached and new, that its rows see, request after request (shared by the
+            # step's layers of one window); base: where a request's position 0 lies, or would lie
             totals = [p + (ctx.h_req_start[i + 1] - ctx.h_req_start[i]) for i, p in enumerate(ctx.h_req_prior)]
+            firsts = [max(0, p + 1 - self.window) if self.window else 0 for p in ctx.h_req_prior]
+            counts = [t - f for t, f in zip(totals, firsts)]
             base = np.zeros(ctx.n_requests, dtype=np.int32)
-            base[:len(totals)] = np.concatenate([[0], np.cumsum(totals)[:-1]])
-            tok_req = np.repeat(np.arange(len(totals), dtype=np.int32), totals)
-            tok_pos = np.concatenate([np.arange(t, dtype=np.int32) for t in totals])
+            base[:len(totals)] = np.concatenate([[0], np.cumsum(counts)[:-1]]) - np.asarray(firsts)
+            tok_req = np.repeat(np.arange(len(totals), dtype=np.int32), counts)
+            tok_pos = np.concatenate([np.arange(f, t, dtype=np.int32) for f, t in zip(firsts, totals)])
             host = torch.from_numpy(np.concatenate([base, tok_req, tok_pos]).astype(np.int32))
             d = host.to(dev, non_blocking=False)
             R, N = ctx.n_requests, int(tok_req.size)
-            layout = ctx._latent_tokens = (d[:R], d[R:R + N], d[R + N:], N)
+            layout = layouts[self.window] = (d[:R], d[R:R + N], d[R + N:], N)
         req_base, tok_req, tok_pos, N = layout
         plane = entry.k_plane
         c_all = torch.empty((N, self.rank), dtype=torch.bfloat16, device=dev)
@@ -246,11 +271,13 @@ class LatentAttention(Part):
                          self.vdim, kx, vx)
         qx = torch.empty((T, H, self.dk_pad), dtype=torch.bfloat16, device=dev)
         K.tag = "q split + rope"
-        K.latent_q_pack(proj, H, self.dim, self.rot, self.rotary, self.position.inv_freq, ctx.positions, qx)
+        K.latent_q_pack(proj, H, self.dim, self.rot, self.rotary, self.position.inv_freq, ctx.positions, qx, halves=self.halves,
+                        magnitude=self.magnitude)
         ox = torch.empty((T, H, self.dv_pad), dtype=torch.bfloat16, device=dev)
         K.tag = "attention"
-        K.latent_flash(qx, ox, kx, vx, ctx.req_start, ctx.req_prior, req_base, ctx.n_requests, H, self.scale, sink=self.sink)
+        K.latent_flash(qx, ox, kx, vx, ctx.req_start, ctx.req_prior, req_base, ctx.n_requests, H, self.scale, sink=self.sink,
+                       window=self.window, exact_weights=self.exact_weights)
         gated = torch.empty((T, H * self.vdim), dtype=torch.bfloat16, device=dev)
         K.tag = "head gate" if gate[0] is not None else "heads out"
-        K.latent_gate_rows(ox, gate[0], gate[1], H, self.vdim, gated)
+        K.latent_gate_rows(ox, gate[0], gate[1], H, self.vdim, gated, by_entry=self.gate_by_entry)
         return gated

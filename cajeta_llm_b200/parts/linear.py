@@ -1,7 +1,7 @@
 """One place that decides which matrix-product kernel a part's projection runs on.
 
-``project`` computes ``out[token, feature] (+)= x[token, :] . w[feature, :]`` (+ bias), or
-the SwiGLU of two such products, for a dense weight or for the stacked weights of a
+``project`` computes ``out[token, feature] (+)= x[token, :] . w[feature, :]`` (+ bias, + an activation), or
+a gated activation of two such products (SwiGLU and its like), for a dense weight or for the stacked weights of a
 mixture of experts.  On the bfloat16 path it runs on the tensor cores (tcgen05 / TMA)
 when the shapes allow TMA (K a multiple of 8, 16-byte aligned rows) and are large
 enough to fill a tile; otherwise, and always on the float32 path, it runs on the FMA
@@ -79,8 +79,9 @@ def _pair_tile(runtime, rows: int, w: torch.Tensor, swiglu: bool, grouped: bool)
 def project(runtime, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bias: Optional[torch.Tensor] = None,
             accumulate: bool = False, w_up: Optional[torch.Tensor] = None, group_offsets: Optional[torch.Tensor] = None,
             a_row_index: Optional[torch.Tensor] = None, max_group_rows: Optional[int] = None,
-            offsets_settled: bool = False, act_limit: float = 0.0, act_alpha: float = 1.0, relu2: bool = False,
-            out_scale: float = 1.0) -> None:
+            offsets_settled: bool = False, act_limit: float = 0.0, act_alpha: float = 1.0, act: str = "",
+            out_scale: float = 1.0, act_cubic: float = 0.0, bias_up: Optional[torch.Tensor] = None,
+            act_features: int = 0) -> None:
     """``x``: [tokens, K]; ``w``: [features, K] or, with ``group_offsets``, [groups, features, K]
     where output row s belongs to the group whose range holds s and reads row
     ``a_row_index[s]`` of ``x`` (or row s).  ``w_up`` selects the SwiGLU form (``out`` in the
@@ -89,22 +90,25 @@ def project(runtime, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bia
     before this call's product (another kernel of this engine ran since, or this call's own
     row gather does); the product may then read the offsets before it waits for that kernel.
     ``act_limit`` > 0 (with ``w_up``): the capped gate g = min(g, limit), u = clamp(u, +-limit),
-    g * sigmoid(act_alpha g) * (u + 1) instead of silu(g) * u.  ``relu2`` (tensor-core path, ``out`` bfloat16, no ``w_up``):
-    ``out = max(x w^T (+ bias), 0)^2``, the float32 sum squared before it is rounded; ask :func:`relu2_fused` first.
+    g * sigmoid(act_alpha g) * (u + 1) instead of silu(g) * u; without a limit the gate is g * sigmoid(act_alpha g + act_cubic g^3)
+    (``K.GELU_TANH`` holds the two numbers of gelu's tanh form); ``bias`` and ``bias_up`` are added to the two sums before it.
+    ``act`` (``out`` in the activation dtype, no ``w_up``): ``"relu2"``, ``out = max(x w^T (+ bias), 0)^2``, ``"gelu"`` (by the error
+    function) or ``"silu"``, of the float32 sum before it is rounded (``act_features`` > 0: of the first that many features alone).
     ``out_scale`` multiplies the sum (bias included) before it is stored in or added to a float32 ``out``."""
     if out_scale != 1.0 and (out.dtype != torch.float32 or w_up is not None):
         raise ValueError("project: out_scale goes with a float32 result of one weight")
-    if relu2 and (w_up is not None or out.dtype != torch.bfloat16 or not _tc_ok(runtime, x, w)):
-        raise ValueError("project: relu2 is the tensor-core product's epilogue (bfloat16 out, no second weight)")
+    if act and (w_up is not None or out.dtype != runtime.act_dtype):
+        raise ValueError("project: act goes with one weight and a result in the activation dtype")
     if not _tc_ok(runtime, x, w):
         K.gemm(x, w, out, bias=bias, accumulate=accumulate, w_up=w_up, group_offsets=group_offsets, a_row_index=a_row_index,
-               act_limit=act_limit, act_alpha=act_alpha, out_scale=out_scale)
+               act_limit=act_limit, act_alpha=act_alpha, out_scale=out_scale, act_cubic=act_cubic, bias_up=bias_up, act=act,
+               act_features=act_features)
         return
     rows = out.shape[0]
     if w_up is not None:
         epi = K.EPI_SWIGLU_BF16
     elif out.dtype == torch.bfloat16:
-        epi = K.EPI_RELU2_BF16 if relu2 else K.EPI_STORE_BF16
+        epi = {"": K.EPI_STORE_BF16, "relu2": K.EPI_RELU2_BF16, "gelu": K.EPI_GELU_BF16, "silu": K.EPI_SILU_BF16}[act]
     else:
         epi = K.EPI_ACC_F32 if accumulate else K.EPI_STORE_F32
     bound = rows if max_group_rows is None else min(rows, max_group_rows)
@@ -129,19 +133,17 @@ def project(runtime, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bia
     if pair_tile:
         # many rows: tiles of 256 features on pairs of SMs, each loading half of the token rows
         K.gemm_tc2(x, w, out, epi, pair_tile, bias=bias, w_up=w_up, group_offsets=group_offsets, tokens=rows,
-                    act_limit=act_limit, act_alpha=act_alpha, out_scale=out_scale)
+                    act_limit=act_limit, act_alpha=act_alpha, out_scale=out_scale, act_cubic=act_cubic, bias_up=bias_up,
+                    act_features=act_features)
     elif tile:
         K.gemm_tc(x, w, out, epi, True, tile, bias=bias, w_up=w_up, group_offsets=group_offsets, tokens=rows,
-                  offsets_settled=offsets_settled, act_limit=act_limit, act_alpha=act_alpha, out_scale=out_scale)
+                  offsets_settled=offsets_settled, act_limit=act_limit, act_alpha=act_alpha, out_scale=out_scale, act_cubic=act_cubic,
+                  bias_up=bias_up, act_features=act_features)
     else:
         n_mma = 256 if (w_up is None and w.shape[-2] >= 512) else 128
         K.gemm_tc(x, w, out, epi, False, n_mma, bias=bias, w_up=w_up, group_offsets=group_offsets, tokens=rows,
-                  offsets_settled=offsets_settled, act_limit=act_limit, act_alpha=act_alpha, out_scale=out_scale)
-
-
-def relu2_fused(runtime, x: torch.Tensor, w: torch.Tensor, out_dtype) -> bool:
-    """Whether :func:`project` can square the rectified sum in its own epilogue for these operands."""
-    return out_dtype == torch.bfloat16 and _tc_ok(runtime, x, w)
+                  offsets_settled=offsets_settled, act_limit=act_limit, act_alpha=act_alpha, out_scale=out_scale, act_cubic=act_cubic,
+                  bias_up=bias_up, act_features=act_features)
 
 
 def split_count(runtime, rows: int, w: torch.Tensor) -> int:

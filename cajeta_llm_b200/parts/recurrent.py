@@ -1,8 +1,7 @@
-"""Mixers that keep a state of fixed size per request: the state-space mixer of Mamba-2 and
-the gated delta rule.
+"""Mixers that keep a state of fixed size per request.
 
-Both project the row, pass part of the projection through a short causal convolution over
-time (per channel, ``conv`` taps, then SiLU) and walk the request's tokens in order through a
+The first two, the state-space mixer of Mamba-2 and the gated delta rule, project the row, pass part of
+the projection through a short causal convolution over time (per channel, ``conv`` taps, then SiLU) and walk the request's tokens in order through a
 float32 state ``S`` per head.  The state of a request lives in its slot of the cache
 manager's state tensor (one flat float32 vector per schedule entry: the convolution's last
 ``conv - 1`` inputs, then the heads' ``S`` in the order the scan's threads hold them); it is
@@ -67,6 +66,17 @@ entries, ``z = sigmoid(W_z x + b_z)``, ``u = W_x x + b_x``, ``c = u + 1/2`` wher
 and the result is ``W_o (S_t * silu(W_g x))``.  The state is ``width`` float32 entries a request.  Gates, candidate and
 state are float32.  Parameters: ``hidden_size``, ``width``.  Tensors: ``z``, ``z.b``, ``x``, ``x.b``, ``g``, ``o``.
 
+``lightning`` (linear attention with one constant decay per head).  ``q = silu(W_q x)``, ``k = silu(W_k x)`` (``heads x dim``),
+``v = silu(W_v x)`` (``heads x vdim``)::
+
+    S_t = decay_h S_(t-1) + k_t v_t^T ;  o_t = S_t^T q_t                          (S: dim x vdim)
+
+The heads' ``o`` side by side are RMS-normed together, times ``norm`` (``heads * vdim`` entries), times ``sigmoid(W_g x)``, then
+``W_o``.  Decays and state are float32; the projections' activations are the input product's epilogue.  Portions of a
+prompt run 64 tokens at a time on the tensor cores on the bfloat16 path (``csrc/decay_attention.cu``).  Parameters:
+``hidden_size``, ``heads``, ``dim``, ``vdim``, ``decay`` (a number in [0, 1] per head), ``eps``.  Tensors: ``q``, ``k``, ``v``, ``g``,
+``norm``, ``o``.
+
 A mixer inside another part (a block that keeps state of its own before the mixer's, a mixer that runs two
 side by side) finds its share of the request's state vector at ``entry.state_offset``.
 """
@@ -74,6 +84,7 @@ from __future__ import annotations
 
 from typing import Dict, Optional
 
+import numpy as np
 import torch
 
 from ..csrc import kernels as K
@@ -417,5 +428,78 @@ class MinGRUMixer(_StateMixer):
         parts = project_split(rt, gated, self.w_o, out_scale=self.out_scale) if self.allow_pending else None
         if parts is None:
             project(rt, gated, self.w_o, residual, accumulate=True, out_scale=self.out_scale)
+        K.tag = None
+        return parts
+
+
+@register_part("mixer", "lightning")
+class LightningMixer(_StateMixer):
+    def __init__(self, spec, prefix, runtime):
+        super().__init__(spec, prefix, runtime)
+        self.hidden = int(spec["hidden_size"])
+        self.heads = int(spec["heads"])
+        self.dim = int(spec["dim"])
+        self.vdim = int(spec["vdim"])
+        self.eps = float(spec["eps"])
+        decay = np.asarray([float(d) for d in spec["decay"]], dtype=np.float64)
+        if decay.shape != (self.heads,) or not bool(((decay >= 0.0) & (decay <= 1.0)).all()):
+            raise ValueError(f"decay must give {self.heads} numbers in [0, 1], found {list(spec['decay'])}")
+        if self.dim > 256:
+            raise ValueError(f"dim {self.dim} is larger than the recurrence's kernel takes (256)")
+        self.qk = self.heads * self.dim
+        self.v = self.heads * self.vdim
+        # one product: q | k | v (activated) | g
+        self.n_act = 2 * self.qk + self.v
+        self.n_in = self.n_act + self.v
+        with np.errstate(divide="ignore"):
+            tables = (decay, decay[:, None] ** np.arange(K.DECAY_CHUNK + 1)[None, :], np.log2(decay))
+        self.decay, self.powers, self.log2_decay = (
+            torch.from_numpy(np.ascontiguousarray(t)).to(device=runtime.device, dtype=d)
+            for t, d in zip(tables, (torch.float32, torch.float32, torch.float64)))
+        self.allow_pending = False         # a block that takes partial sums from its mixer sets this True
+        self.w_in = self.w_norm = self.w_o = None
+
+    def state_need(self) -> Optional[StateNeed]:
+        return StateNeed((self.heads * self.dim * self.vdim,), torch.float32)
+
+    def params(self) -> Dict[str, ParamSpec]:
+        return {
+            self.name("q"): ParamSpec((self.qk, self.hidden)),
+            self.name("k"): ParamSpec((self.qk, self.hidden)),
+            self.name("v"): ParamSpec((self.v, self.hidden)),
+            self.name("g"): ParamSpec((self.v, self.hidden)),
+            self.name("norm"): ParamSpec((self.v,), role="vector", init="ones"),
+            self.name("o"): ParamSpec((self.hidden, self.v)),
+        }
+
+    def libraries(self) -> set:
+        return (super().libraries() - {"recurrent"}) | {"decay_attention"}
+
+    def load(self, source) -> None:
+        self.w_in = torch.cat([self.fetch(source, self.name(n)) for n in ("q", "k", "v", "g")], dim=0).contiguous()
+        self.w_norm = self.fetch(source, self.name("norm"))
+        self.w_o = self.fetch(source, self.name("o"))
+
+    def defers(self, rows: int) -> bool:
+        return self.allow_pending and splits_few_rows(self.runtime, rows, self.w_o)
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, entry) -> Optional[torch.Tensor]:
+        rt = self.runtime
+        T = x.shape[0]
+        proj = torch.empty((T, self.n_in), dtype=rt.act_dtype, device=x.device)
+        K.tag = "mixer in"
+        project(rt, x, self.w_in, proj, act="silu", act_features=self.n_act)
+        o = torch.empty((T, self.v), dtype=torch.float32, device=x.device)
+        K.tag = "scan"
+        K.decay_attention(proj, 0, self.qk, 2 * self.qk, self.decay, self.powers, self.log2_decay, entry.state,
+                          getattr(entry, "state_offset", 0), ctx.req_start, ctx.req_slot, ctx.n_requests, o, self.heads, self.dim,
+                          self.vdim, single=getattr(ctx, "all_single", False))
+        gated = torch.empty((T, self.v), dtype=rt.act_dtype, device=x.device)
+        K.tag = "gate + norm"
+        K.gated_row_norm(o, proj, self.n_act, self.w_norm, self.eps, gated)
+        K.tag = "o"
+        parts = project_split(rt, gated, self.w_o) if self.allow_pending else None
+        if parts is None:
+            project(rt, gated, self.w_o, residual, accumulate=True)
         K.tag = None
         return parts
