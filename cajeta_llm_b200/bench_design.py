@@ -1,11 +1,13 @@
-"""Throughput of a Balalorn, a Saropel, a Govuvik, a Dimuvik or a Rugezen model at layer sizes that resemble real models', beside the
+"""Throughput of a Balalorn, a Saropel, a Govuvik, a Dimuvik, a Rugezen or a Zoporax model at layer sizes that resemble real models', beside the
 engine's Qwen2-MoE model at equal width, depth, experts and feed-forward sizes (Govuvik: beside Balalorn, the
 engine's other model with recurrent state, at equal width, depth and experts; Dimuvik: beside Balalorn, the engine's
 other model with attention over a latent and a borrowed cache, at equal width, depth, heads, latent and experts; Rugezen:
 beside a Saropel of dense layers alone, the engine's other model of parallel blocks with capped attention and a looped
-stretch, at equal width, depth, heads and feed-forward, and beside Balalorn for its recurrent layers).
+stretch, at equal width, depth, heads and feed-forward, and beside Balalorn for its recurrent layers; Zoporax: beside Dimuvik,
+the engine's other model whose latent attention has a latent of the queries, and beside Balalorn, whose layers are latent attention and
+recurrences too, at equal width, depth, heads, latent, experts and feed-forward).
 
-``python bench.py --design balalorn|saropel|govuvik|dimuvik|rugezen [--sizes small,medium,large]`` prints one JSON line per
+``python bench.py --design balalorn|saropel|govuvik|dimuvik|rugezen|zoporax [--sizes small,medium,large]`` prints one JSON line per
 (size, model): prefill tokens a second (one prompt of 2,048 tokens), decode tokens a second
 (8 requests of 512 tokens each, steps replayed from CUDA graphs), and where the time of both
 steps goes by class of work (launches serialised, an event behind each), with the bytes or
@@ -103,6 +105,28 @@ def dimuvik_config(s):
             "layers": [kinds[i % 4](i) for i in range(s["layers"])]}
 
 
+ZOPORAX_WINDOW = 1024
+ZOPORAX_KINDS = ("lightning", "latent", "lightning", "latent")
+
+
+def zoporax_config(s):
+    """Four layers: linear attention with a decay per head (H heads of 128) + dense, windowed latent attention (queries through a
+    latent of three times the keys' rank, half rotation with stretched frequencies, a gate per entry) + routed with a shared
+    expert, linear attention + routed, latent attention + dense."""
+    h, H = s["width"], s["heads"]
+    latent = {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": s["rank"], "q_rank": 3 * s["rank"], "scale": (128 + 64) ** -0.5,
+              "mask": {"size": ZOPORAX_WINDOW},
+              "rot": {"base": 50000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    linear = {"heads": H, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-2.0 - 6.0 * i / H) for i in range(H)]}
+    moe = {"kind": "moe", "expert": {"ff": s["eff"]}, "shared": {"ff": s["eff"]},
+           "router": {"experts": s["experts"], "top": s["top"], "scale": 2.0, "groups": {"count": 4, "keep": 2}}}
+    dense = {"kind": "dense", "ff": s["ff"]}
+    mlps = (dense, moe, moe, dense)
+    return {"architecture": "Zoporax", "width": h, "vocab": VOCAB, "norm": {"eps": 1e-6},
+            "layers": [{"type": "lightning", "mixer": linear, "mlp": mlps[i % 4]} if ZOPORAX_KINDS[i % 4] == "lightning"
+                       else {"type": "latent_attention", "mixer": latent, "mlp": mlps[i % 4]} for i in range(s["layers"])]}
+
+
 RUGEZEN_RUNS = ("attention", "mingru", "mingru", "attention")      # three layers of weights; the middle one runs twice
 
 
@@ -138,9 +162,33 @@ def qwen_config(s, shared=0):
             "tie_word_embeddings": False, "use_sliding_window": False}
 
 
+# designs whose feed-forwards are compared by class: (gated experts, gated dense, a shared expert), of two layers each
+WEIGHT_CLASSES = {"zoporax": (False, True, True), "dimuvik": (True, False, True), "balalorn": (True, True, False)}
+
+
+def weight_needs(design, s, rows, prefill):
+    """(bytes, flops) of the feed-forward products of one step: a decode step streams each weight it uses once (of the experts as
+    many as its rows are expected to pick between them), a prompt portion's flops count."""
+    gated_e, gated_d, shared = WEIGHT_CLASSES[design]
+    one, E, top = 2 * s["width"] * s["eff"], s["experts"], s["top"]
+    used = E * (1.0 - (1.0 - top / E) ** rows) + (1 if shared else 0)
+    picks = rows * (top + (1 if shared else 0))
+    out = {}
+    for label, n, w in (("dense gate/up" if gated_d else "dense up", 2 if gated_d else 1, None), ("dense down", 1, None),
+                        ("experts gate/up" if gated_e else "experts up", 2 if gated_e else 1, one), ("experts down", 1, one)):
+        if w is None:
+            by, fl = 2 * n * s["width"] * s["ff"], 2 * n * s["width"] * s["ff"] * rows
+        else:
+            by, fl = n * w * used, n * w * picks
+        out[label] = (0 if prefill else 2 * by, 2 * fl if prefill else 0)          # two layers of each kind
+    return out
+
+
 def needs(design, s, rows, ctx, prefill):
     """(bytes, flops) the attention-like classes of one step must move, over all layers."""
     L, H, out = s["layers"], s["heads"], {}
+    if design in WEIGHT_CLASSES:
+        out.update(weight_needs(design, s, rows, prefill))
     if design == "qwen2_moe":
         kv = ctx * 2 * H * 128 * 2
         out["attention"] = (rows * kv * L if not prefill else 0, 4 * H * 128 * rows * (rows + 1) // 2 * L if prefill else 0)
@@ -182,6 +230,15 @@ def needs(design, s, rows, ctx, prefill):
         out["scan"] = (reqs * 2 * (n_mem * mem + n_par * gla)
                        + rows * 4 * (n_mem * (H // 2) * (2 * 128 + 256 + 2) + n_par * (H // 4) * (3 * 128 + 256)),
                        rows * (n_mem * (H // 2) * 128 * 256 * 6 + n_par * (H // 4) * 128 * 256 * 5))
+        return out
+    if design == "zoporax":
+        kinds = [ZOPORAX_KINDS[i % 4] for i in range(L)]
+        n_lat, n_lin, w = kinds.count("latent"), kinds.count("lightning"), ZOPORAX_WINDOW
+        out["attention"] = (rows * min(ctx, w) * (s["rank"] + 64) * 2 * n_lat if not prefill else 0,
+                            2 * H * (128 + 64 + 128) * n_lat * sum(min(i + 1, w) for i in range(rows)) if prefill else 0)
+        # the states once in, once out; q, k and v in bfloat16 in, a float32 row out; the least work of the recurrence
+        reqs = 1 if prefill else rows
+        out["scan"] = ((reqs * 2 * H * 128 * 128 * 4 + rows * H * 128 * (3 * 2 + 4)) * n_lin, rows * H * 128 * 128 * 5 * n_lin)
         return out
     if design == "dimuvik":
         n_lat, n_diff = (L + 3) // 4 + (L + 1) // 4, (L + 2) // 4 + L // 4
@@ -226,6 +283,8 @@ def run(args, peaks) -> int:
             pair = (("govuvik", govuvik_config(s)), ("balalorn", balalorn_config(s)))
         elif args.design == "dimuvik":
             pair = (("dimuvik", dimuvik_config(s)), ("balalorn", balalorn_config(s)))
+        elif args.design == "zoporax":
+            pair = (("zoporax", zoporax_config(s)), ("dimuvik", dimuvik_config(s)), ("balalorn", balalorn_config(s)))
         elif args.design == "rugezen":
             pair = (("rugezen", rugezen_config(s)), ("saropel_dense", saropel_dense_config(s)), ("balalorn", balalorn_config(s)))
         else:

@@ -77,6 +77,51 @@ __device__ __forceinline__ float plain_act(float v, int act) {
     v = fmaxf(v, 0.0f);
     return v * v;
 }
+// The same for results that are rounded to bfloat16: silu with the fast exponential and division; gelu by the rational
+// approximation of the error function with five terms by C. Hastings (Abramowitz and Stegun, Handbook of Mathematical
+// Functions, 7.1.26; absolute error at most 1.5e-7), erfc(y) = t (a1 + t (a2 + .. a5)) exp(-y^2), t = 1 / (1 + p y), y >= 0.
+__device__ __forceinline__ float plain_act_fast(float v, int act) {
+    if (act == ACT_GELU) {
+        const float y = fabsf(v) * 0.70710678118654752f;
+        const float t = __fdividef(1.0f, fmaf(0.3275911f, y, 1.0f));
+        float a = fmaf(1.061405429f, t, -1.453152027f);
+        a = fmaf(a, t, 1.421413741f);
+        a = fmaf(a, t, -0.284496736f);
+        a = fmaf(a, t, 0.254829592f);
+        const float tail = 0.5f * a * t * __expf(-y * y);        // Phi(-|v|)
+        return v * (v >= 0.0f ? 1.0f - tail : tail);
+    }
+    if (act == ACT_SILU) return __fdividef(v, 1.0f + __expf(-v));
+    v = fmaxf(v, 0.0f);
+    return v * v;
+}
+// N results at once: the choice outside the loop, the values' chains side by side
+template <int N>
+__device__ __forceinline__ void plain_acts_fast(float (&v)[N], int act) {
+    if (act == ACT_GELU) {
+#pragma unroll
+        for (int j = 0; j < N; ++j) v[j] = plain_act_fast(v[j], ACT_GELU);
+    } else if (act == ACT_SILU) {
+#pragma unroll
+        for (int j = 0; j < N; ++j) v[j] = plain_act_fast(v[j], ACT_SILU);
+    } else {
+#pragma unroll
+        for (int j = 0; j < N; ++j) v[j] = plain_act_fast(v[j], ACT_RELU2);
+    }
+}
+// 16 biases of consecutive features from f0 on (zeros without a bias or past the last feature)
+__device__ __forceinline__ void load_bias16(const float* b, int f0, int features, float (&o)[16]) {
+    if (b && f0 + 16 <= features && (((uintptr_t)(b + f0)) & 15) == 0) {
+#pragma unroll
+        for (int j = 0; j < 16; j += 4) {
+            const float4 v = __ldg((const float4*)(b + f0 + j));
+            o[j] = v.x; o[j + 1] = v.y; o[j + 2] = v.z; o[j + 3] = v.w;
+        }
+    } else {
+#pragma unroll
+        for (int j = 0; j < 16; ++j) o[j] = b && f0 + j < features ? b[f0 + j] : 0.0f;
+    }
+}
 
 // Launches overlap their neighbours in the stream (programmatic dependent launch): a kernel
 // may be set up on the SMs while the one before it is still draining.  Every kernel of this

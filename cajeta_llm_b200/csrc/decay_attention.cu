@@ -8,6 +8,7 @@
 //
 //   walk     every token in order: the state's rows dealt to eight warps, its columns to their lanes, all of it in
 //            registers; single decoded tokens, short portions, and everything on the 32-bit path
+//            (the next tokens' inputs are on their way to registers while these are walked)
 //   chunk    (bfloat16 q, k, v) portions of a prompt, 64 tokens at a time on the tensor cores:
 //                O = (Q K^T . L) V + diag(lambda^(i+1)) Q S ,   L_ij = lambda^(i-j) for j <= i, else 0
 //                S <- lambda^n S + K^T diag(lambda^(n-1-j)) V
@@ -69,20 +70,36 @@ __global__ void __launch_bounds__(WALK_WARPS * 32) walk_kernel(WalkArgs p) {
         s[i] = live && d < p.dim ? S[(size_t)d * p.vdim + col] : 0.0f;
     }
     const float decay = p.decay[head];
+    // what this thread brings of WALK_TOK tokens: entries thread + 256 i of their [WALK_TOK][DIM] queries and keys, one value
+    constexpr int MINE = WALK_TOK * DIM / (WALK_WARPS * 32);
+    static_assert(MINE >= 1 && WALK_TOK == WALK_WARPS, "a block's threads share out the tokens' entries evenly");
+    float q_next[MINE], k_next[MINE], v_next;
+    auto fetch = [&](int t0) {
+        const TX* base = (const TX*)p.x + (size_t)(first + t0) * p.ld;
+#pragma unroll
+        for (int i = 0; i < MINE; ++i) {
+            const int e = threadIdx.x + WALK_WARPS * 32 * i, t = e / DIM, d = e % DIM;
+            const bool ok = t0 + t < n && d < p.dim;
+            const TX* row = base + (size_t)(ok ? t : 0) * p.ld + head * p.dim + (ok ? d : 0);
+            q_next[i] = ok ? to_f32(row[p.off_q]) : 0.0f;
+            k_next[i] = ok ? to_f32(row[p.off_k]) : 0.0f;
+        }
+        const bool ok = t0 + warp < n && live;
+        v_next = ok ? to_f32(base[(size_t)warp * p.ld + p.off_v + head * p.vdim + col]) : 0.0f;
+    };
+    fetch(0);
     for (int t0 = 0; t0 < n; t0 += WALK_TOK) {
         const int nt = min(WALK_TOK, n - t0);
-        for (int e = threadIdx.x; e < nt * DIM; e += WALK_WARPS * 32) {
-            const int t = e / DIM, d = e % DIM;
-            const TX* row = (const TX*)p.x + (size_t)(first + t0 + t) * p.ld + head * p.dim;
+#pragma unroll
+        for (int i = 0; i < MINE; ++i) {
+            const int e = threadIdx.x + WALK_WARPS * 32 * i, t = e / DIM, d = e % DIM;
             const int at = (d % WALK_WARPS) * ROWS + d / WALK_WARPS;
-            qs[t][at] = d < p.dim ? to_f32(row[p.off_q + d]) : 0.0f;
-            ks[t][at] = d < p.dim ? to_f32(row[p.off_k + d]) : 0.0f;
+            qs[t][at] = q_next[i];
+            ks[t][at] = k_next[i];
         }
-        for (int e = threadIdx.x; e < nt * 32; e += WALK_WARPS * 32) {
-            const int t = e / 32, c = blockIdx.z * 32 + e % 32;
-            vs[t][e % 32] = c < p.vdim ? to_f32(((const TX*)p.x)[(size_t)(first + t0 + t) * p.ld + p.off_v + head * p.vdim + c]) : 0.0f;
-        }
+        vs[warp][lane] = v_next;
         __syncthreads();
+        if (t0 + WALK_TOK < n) fetch(t0 + WALK_TOK);
         for (int t = 0; t < nt; ++t) {
             const float v = vs[t][lane];
             const float4* k4 = (const float4*)(ks[t] + warp * ROWS);
@@ -174,7 +191,8 @@ struct ChunkArgs {
     const int* req_slot;
     int n_requests;
     float* out;                   // [T, heads * vdim]
-    float* added;                 // [segments][heads][dim][vdim]: what a segment adds to the state; in a request's last one S_0
+    float4* added;                // [segments][heads][column tiles][D / 8][threads]: what a segment adds to the state, in the order the
+                                  // threads hold it; in a request's last one S_0
     int heads, dim, vdim;
     int seg;                      // tokens of a segment (a multiple of CHUNK)
     int most;                     // requests of at most this many rows are left to the walk
@@ -250,29 +268,52 @@ __global__ void __launch_bounds__(32 * WARPS) chunk_kernel(ChunkArgs p) {
     float S[D / 8][4];                                       // S^T: [j][0,1] = (va, 8 j + 2 t4 + 0,1), [2,3] = (vb, ..)
 #pragma unroll
     for (int j = 0; j < D / 8; ++j) S[j][0] = S[j][1] = S[j][2] = S[j][3] = 0.0f;
-    const size_t mat = (size_t)p.dim * p.vdim;
-    auto add_scaled = [&](const float* m, float f) {
+    float* state = p.state + (size_t)p.req_slot[req] * p.slot_stride + (size_t)head * p.dim * p.vdim;
+    auto state_at = [&](int j, int e, bool& ok) {            // where entry e of S[j] lies in a [dim][vdim] matrix
+        const int d = 8 * j + 2 * t4 + (e & 1), v = e < 2 ? va : vb;
+        ok = d < p.dim && v < p.vdim;
+        return ok ? (size_t)d * p.vdim + v : (size_t)0;
+    };
+    auto read_state = [&]() {
 #pragma unroll
         for (int j = 0; j < D / 8; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                const int d = 8 * j + 2 * t4 + (e & 1), v = e < 2 ? va : vb;
-                if (d < p.dim && v < p.vdim) S[j][e] = fmaf(f, m[(size_t)d * p.vdim + v], S[j][e]);
+                bool ok;
+                const float v = state[state_at(j, e, ok)];
+                S[j][e] = ok ? v : 0.0f;
             }
     };
-    const float* before = p.state + (size_t)p.req_slot[req] * p.slot_stride + head * mat;         // S_0
-    float* kept = p.added ? p.added + ((size_t)(blockIdx.x - at + n_segs - 1) * p.heads + head) * mat : nullptr;
+    auto held = [&](int segment) {                           // this thread's part of what the launch's segment left in `added`
+        return p.added + (((size_t)segment * p.heads + head) * gridDim.z + blockIdx.z) * (D / 8) * THREADS + tid;
+    };
+    auto keep_in = [&](float4* m) {
+#pragma unroll
+        for (int j = 0; j < D / 8; ++j) m[(size_t)j * THREADS] = make_float4(S[j][0], S[j][1], S[j][2], S[j][3]);
+    };
     if (ADDED && at == 0) {
-        for (int e = tid; e < p.dim * V; e += THREADS) {
-            const int d = e / V, v = v0 + e % V;
-            if (v < p.vdim) kept[(size_t)d * p.vdim + v] = before[(size_t)d * p.vdim + v];
-        }
+        read_state();
+        keep_in(held(blockIdx.x + n_segs - 1));
+#pragma unroll
+        for (int j = 0; j < D / 8; ++j) S[j][0] = S[j][1] = S[j][2] = S[j][3] = 0.0f;
     }
-    if (!ADDED) {
+    if (!ADDED && n_segs == 1) read_state();
+    if (!ADDED && n_segs > 1) {
         const double l2 = p.log2_decay[head];
-        add_scaled(n_segs > 1 ? kept : before, power_of(l2, s0));
-        for (int s = 0; s < at; ++s)                         // segment s ends (at - 1 - s) whole segments before this one begins
-            add_scaled(p.added + ((size_t)(blockIdx.x - at + s) * p.heads + head) * mat, power_of(l2, (at - 1 - s) * p.seg));
+        const int base = blockIdx.x - at;
+        for (int s = -1; s < at; ++s) {
+            // S_0, then the segments before this one: segment s ends (at - 1 - s) whole segments before this one begins
+            const float4* m = held(s < 0 ? base + n_segs - 1 : base + s);
+            const float f = power_of(l2, s < 0 ? s0 : (at - 1 - s) * p.seg);
+#pragma unroll
+            for (int j = 0; j < D / 8; ++j) {
+                const float4 a = m[(size_t)j * THREADS];
+                S[j][0] = fmaf(f, a.x, S[j][0]);
+                S[j][1] = fmaf(f, a.y, S[j][1]);
+                S[j][2] = fmaf(f, a.z, S[j][2]);
+                S[j][3] = fmaf(f, a.w, S[j][3]);
+            }
+        }
     }
 
     int cur = 0;
@@ -405,15 +446,15 @@ __global__ void __launch_bounds__(32 * WARPS) chunk_kernel(ChunkArgs p) {
         }
         __syncthreads();                                     // this chunk's tiles and scores are read before they are written again
     }
-    if (ADDED || last) {
-        float* m = ADDED ? p.added + ((size_t)blockIdx.x * p.heads + head) * mat
-                         : p.state + (size_t)p.req_slot[req] * p.slot_stride + head * mat;
+    if (ADDED) keep_in(held(blockIdx.x));
+    else if (last) {
 #pragma unroll
         for (int j = 0; j < D / 8; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                const int d = 8 * j + 2 * t4 + (e & 1), v = e < 2 ? va : vb;
-                if (d < p.dim && v < p.vdim) m[(size_t)d * p.vdim + v] = S[j][e];
+                bool ok;
+                const size_t to = state_at(j, e, ok);
+                if (ok) state[to] = S[j][e];
             }
     }
 }
@@ -472,7 +513,8 @@ CJ_EXPORT int cj_decay_walk(const void* x, int x_dtype, int ld, int off_q, int o
 
 // The tensor-core form for requests with more rows than `most`.  x bfloat16, 16-byte aligned rows and columns; dim <= 128, dim and
 // vdim multiples of 8.  seg: tokens of a segment, a multiple of 64; segments: blocks laid out for them, at least
-// rows / seg + requests; added: float32 [segments, heads, dim, vdim] scratch (may be null when every request fits one segment).
+// rows / seg + requests; added: scratch of cj_decay_added_floats float32 a segment, 16-byte aligned (may be null when
+// every request fits one segment).
 CJ_EXPORT int cj_decay_chunk(const void* x, int ld, int off_q, int off_k, int off_v, const float* powers, const double* log2_decay,
                              float* state, long long slot_stride, const int* req_start, const int* req_slot, int requests, float* out,
                              float* added, int segments, int heads, int dim, int vdim, int seg, int most, cudaStream_t stream) {
@@ -480,9 +522,9 @@ CJ_EXPORT int cj_decay_chunk(const void* x, int ld, int off_q, int off_k, int of
     if (!x || !powers || !log2_decay || !state || !req_start || !req_slot || !out) return CJ_ERR_ARG;
     if (heads <= 0 || heads > 65535 || dim <= 0 || dim > 128 || vdim <= 0 || seg <= 0 || seg % CHUNK != 0 || most < 0) return CJ_ERR_SIZE;
     if (slot_stride < (long long)heads * dim * vdim) return CJ_ERR_SIZE;
-    if ((dim | vdim | ld | off_q | off_k | off_v) % 8 != 0 || ((uintptr_t)x & 15)) return CJ_ERR_ALIGN;
+    if ((dim | vdim | ld | off_q | off_k | off_v) % 8 != 0 || (((uintptr_t)x | (uintptr_t)added) & 15)) return CJ_ERR_ALIGN;
     ChunkArgs p{(const __nv_bfloat16*)x, ld, off_q, off_k, off_v, powers, log2_decay, state, slot_stride, req_start, req_slot, requests,
-                out, added, heads, dim, vdim, seg, most};
+                out, (float4*)added, heads, dim, vdim, seg, most};
 #define LAUNCH_ONE(D_, W_, A_)                                                                                          \
     do {                                                                                                                \
         constexpr int bytes = ChunkSmem<D_, W_>::BYTES;                                                                 \
@@ -504,6 +546,12 @@ CJ_EXPORT int cj_decay_chunk(const void* x, int ld, int off_q, int off_k, int of
 #undef LAUNCH
 #undef LAUNCH_ONE
     return launch_status();
+}
+
+// float32 entries of `added` that one segment needs
+CJ_EXPORT long long cj_decay_added_floats(int heads, int dim, int vdim) {
+    const int D = dim <= 64 ? 64 : 128, W = vdim <= 64 ? 4 : 8;
+    return (long long)heads * ((vdim + 16 * W - 1) / (16 * W)) * (D / 8) * 4 * 32 * W;
 }
 
 // z: the gates' columns, rows ld_z apart, in z_dtype; (z, out): (float32, float32) or (bfloat16, bfloat16)

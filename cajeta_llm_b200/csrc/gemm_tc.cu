@@ -375,18 +375,18 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
 #pragma unroll
                     for (int j = 0; j < 16; ++j) v0[j] = v1[j] = 0;
                 }
-                float v[16];
+                float v[16], b0[16], b1[16];
+                if (EPI == EPI_SWIGLU_BF16 && !SWAP) {
+                    cj::load_bias16(p.bias, c.feat0 + c0, p.features, b0);
+                    cj::load_bias16(p.bias2, c.feat0 + c0, p.features, b1);
+                }
 #pragma unroll
                 for (int j = 0; j < 16; ++j) {
                     v[j] = __uint_as_float(v0[j]);
                     // the result is rounded to bfloat16 (8 bits): the fast exponential and division (2 ulp of float32) do not show
                     if (EPI == EPI_SWIGLU_BF16) {
-                        if (!SWAP) {
-                            const int f = min(c.feat0 + c0 + j, p.features - 1);
-                            bg = p.bias ? p.bias[f] : 0.0f;
-                            bu = p.bias2 ? p.bias2[f] : 0.0f;
-                        }
-                        v[j] = cj::gated_act_fast(v[j] + bg, __uint_as_float(v1[j]) + bu, p.act_limit, p.act_alpha, p.act_cubic);
+                        v[j] = cj::gated_act_fast(v[j] + (SWAP ? bg : b0[j]), __uint_as_float(v1[j]) + (SWAP ? bu : b1[j]), p.act_limit,
+                                                  p.act_alpha, p.act_cubic);
                     }
                 }
                 if (!SWAP) {
@@ -400,8 +400,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
                         for (int j = 0; j < 16; ++j) if (whole || feat + j < p.features) v[j] += p.bias[feat + j];
                     }
                     if (EPI == EPI_ACT_BF16) {
+                        if (feat + 16 <= p.act_feats) cj::plain_acts_fast<16>(v, p.act);
+                        else if (feat < p.act_feats) {
 #pragma unroll
-                        for (int j = 0; j < 16; ++j) if (feat + j < p.act_feats) v[j] = cj::plain_act(v[j], p.act);
+                            for (int j = 0; j < 16; ++j) if (feat + j < p.act_feats) v[j] = cj::plain_act_fast(v[j], p.act);
+                        }
                     }
                     if (EPI == EPI_STORE_F32 || EPI == EPI_ACC_F32) {
 #pragma unroll
@@ -445,13 +448,17 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
                     const int feat = c.feat0 + r;
                     if (r >= feat_tile || feat >= p.features) continue;
                     const float b = add_bias ? p.bias[feat] : 0.0f;
+                    if (EPI == EPI_ACT_BF16) {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) v[j] += b;
+                        if (feat < p.act_feats) cj::plain_acts_fast<16>(v, p.act);
+                    }
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
                         int token = c.tok0 + c0 + j;
                         if (token >= c.tok_end) break;
                         long long o = (long long)token * p.ldo + feat;
-                        float val = v[j] + b;
-                        if (EPI == EPI_ACT_BF16 && feat < p.act_feats) val = cj::plain_act(val, p.act);
+                        float val = EPI == EPI_ACT_BF16 ? v[j] : v[j] + b;
                         if (EPI == EPI_STORE_F32 || EPI == EPI_ACC_F32) val *= p.out_scale;
                         if (EPI == EPI_STORE_F32) ((float*)p.out)[o + split_off] = val;
                         else if (EPI == EPI_ACC_F32) ((float*)p.out)[o] += val;

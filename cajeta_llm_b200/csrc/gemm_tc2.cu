@@ -268,11 +268,14 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant
                         for (int j = 0; j < 32; ++j)
                             if (c0 + j < n_cols) ((float*)p.out)[o0 + j * p.ldo] = old[j] + (__uint_as_float(v[j]) + b) * p.out_scale;
                     } else {
+                        float f[32];
+#pragma unroll
+                        for (int j = 0; j < 32; ++j) f[j] = __uint_as_float(v[j]) + b;
+                        if (EPI == EPI_ACT_BF16 && feat < p.act_feats) cj::plain_acts_fast<32>(f, p.act);       // an expert without a gate
 #pragma unroll
                         for (int j = 0; j < 32; ++j) {
                             if (c0 + j >= n_cols) break;
-                            float val = __uint_as_float(v[j]) + b;
-                            if (EPI == EPI_ACT_BF16 && feat < p.act_feats) val = cj::plain_act(val, p.act);       // an expert without a gate
+                            const float val = f[j];
                             if (EPI == EPI_STORE_F32) ((float*)p.out)[o0 + j * p.ldo] = val * p.out_scale;
                             else ((__nv_bfloat16*)p.out)[o0 + j * p.ldo] = __float2bfloat16_rn(val);
                         }
@@ -443,6 +446,9 @@ swiglu_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_const
                 for (int c0 = 0; c0 < SW_FEAT; c0 += 16) {
                     if (c.feat0 + c0 >= p.features) break;
                     uint32_t g[16], u[16];
+                    float bg[16], bu[16];
+                    cj::load_bias16(p.bias, c.feat0 + c0, p.features, bg);
+                    cj::load_bias16(p.bias2, c.feat0 + c0, p.features, bu);
                     tmem_ld16(lane_base + c0, g);
                     tmem_ld16(lane_base + SW_FEAT + c0, u);
                     tmem_ld_wait();
@@ -450,10 +456,8 @@ swiglu_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_const
                     float v[16];
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
-                        const int f = min(c.feat0 + c0 + j, p.features - 1);
-                        const float gv = __uint_as_float(g[j]) + (p.bias ? p.bias[f] : 0.0f);
-                        const float uv = __uint_as_float(u[j]) + (p.bias2 ? p.bias2[f] : 0.0f);
-                        v[j] = cj::gated_act_fast(gv, uv, p.act_limit, p.act_alpha, p.act_cubic);
+                        v[j] = cj::gated_act_fast(__uint_as_float(g[j]) + bg[j], __uint_as_float(u[j]) + bu[j], p.act_limit, p.act_alpha,
+                                                  p.act_cubic);
                     }
                     __nv_bfloat16* dst = dst_row + c0;
                     if (c.feat0 + c0 + 16 <= p.features && (((uintptr_t)dst) & 15) == 0) {

@@ -968,7 +968,10 @@ def decay_attention(x: torch.Tensor, off_q: int, off_k: int, off_v: int, decay: 
         return
     seg = segment or decay_segment(T, heads, vdim)
     segments = T // seg + requests
-    added = torch.empty((segments, heads, dim, vdim), dtype=torch.float32, device=x.device) if T > seg else None
+    added = None
+    if T > seg:
+        lib.cj_decay_added_floats.restype = ctypes.c_longlong
+        added = torch.empty((segments, lib.cj_decay_added_floats(_i(heads), _i(dim), _i(vdim))), dtype=torch.float32, device=x.device)
     st = lib.cj_decay_chunk(_ptr(x), _i(x.stride(0)), _i(off_q), _i(off_k), _i(off_v), _ptr(powers), _ptr(log2_decay), st_ptr,
                             _ll(state.stride(0)), _ptr(req_start), _ptr(req_slot), _i(requests), _ptr(out), _ptr(added), _i(segments),
                             _i(heads), _i(dim), _i(vdim), _i(seg), _i(DECAY_WALK_ROWS), _stream())
