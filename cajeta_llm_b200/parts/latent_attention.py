@@ -250,8 +250,10 @@ class LatentAttention(Part):
             base[:len(totals)] = np.concatenate([[0], np.cumsum(counts)[:-1]]) - np.asarray(firsts)
             tok_req = np.repeat(np.arange(len(totals), dtype=np.int32), counts)
             tok_pos = np.concatenate([np.arange(f, t, dtype=np.int32) for f, t in zip(firsts, totals)])
-            host = torch.from_numpy(np.concatenate([base, tok_req, tok_pos]).astype(np.int32))
-            d = host.to(dev, non_blocking=False)
+            # pinned and not waited for: the step's launches go on while it travels
+            host = torch.empty((base.size + tok_req.size + tok_pos.size,), dtype=torch.int32, pin_memory=True)
+            host.numpy()[:] = np.concatenate([base, tok_req, tok_pos])
+            d = host.to(dev, non_blocking=True)
             R, N = ctx.n_requests, int(tok_req.size)
             layout = layouts[self.window] = (d[:R], d[R:R + N], d[R + N:], N)
         req_base, tok_req, tok_pos, N = layout
